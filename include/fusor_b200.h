@@ -49,7 +49,7 @@ typedef enum fb200_status {
 /* ggml type ids, fusor-ml/gguf/src/lib.rs:35-50 */
 typedef enum fb200_ggml_type {
   FB200_F32 = 0, FB200_F16 = 1, FB200_Q4_0 = 2, FB200_Q5_0 = 6, FB200_Q8_0 = 8,
-  FB200_Q4_K = 12, FB200_Q5_K = 13, FB200_Q6_K = 14
+  FB200_Q4_K = 12, FB200_Q5_K = 13, FB200_Q6_K = 14, FB200_BF16 = 30
 } fb200_ggml_type;
 
 typedef struct fb200_device fb200_device;
@@ -100,7 +100,7 @@ FB200_API int fb200_memset(fb200_device* dev, void* dst_dev, int value, size_t b
  * weight (row-major blocks along K, fusor-ml/cpu/src/quantized.rs:293-294), copied during the
  * call. K must be a multiple of the block size (else FB200_ERR_INVALID_SHAPE, where the
  * reference panics, cpu/src/quantized.rs:54-69); unknown types give
- * FB200_ERR_UNSUPPORTED_DTYPE (GgufReadError::UnsupportedDType). F32/F16 are accepted as dense.
+ * FB200_ERR_UNSUPPORTED_DTYPE (GgufReadError::UnsupportedDType). F32/F16/BF16 are accepted as dense.
  * On the device the blocks are stored in a tile-interleaved order (same bytes, permuted) so
  * that warps read them with coalesced 128-bit loads. Two types are stored otherwise: Q5_0 as Q8_0
  * tiles (the same scale, the 5-bit integer widened to 8 bits: the same values, 34 instead of 22
@@ -300,11 +300,49 @@ typedef struct fb200_llama_config {
 typedef enum fb200_llama_tensor {
   FB200_T_TOKEN_EMBD = 0, FB200_T_OUTPUT = 1, FB200_T_ATTN_Q = 2, FB200_T_ATTN_K = 3,
   FB200_T_ATTN_V = 4, FB200_T_ATTN_OUTPUT = 5, FB200_T_FFN_GATE = 6, FB200_T_FFN_UP = 7,
-  FB200_T_FFN_DOWN = 8, FB200_T_ATTN_NORM = 9, FB200_T_FFN_NORM = 10, FB200_T_OUTPUT_NORM = 11
+  FB200_T_FFN_DOWN = 8, FB200_T_ATTN_NORM = 9, FB200_T_FFN_NORM = 10, FB200_T_OUTPUT_NORM = 11,
+  /* token-mixer layers (fb200_llama_create_layers); FB200_T_ATTN_NORM is the layer's one norm */
+  FB200_T_MIX_Q = 12, FB200_T_MIX_K = 13, FB200_T_MIX_V = 14, FB200_T_MIX_GATE = 15, FB200_T_MIX_OUT = 16,
+  FB200_T_MIX_BETA = 17, FB200_T_MIX_DECAY = 18, FB200_T_MIX_Q_CONV = 19, FB200_T_MIX_K_CONV = 20,
+  FB200_T_MIX_V_CONV = 21, FB200_T_MIX_A_LOG = 22, FB200_T_MIX_DT_BIAS = 23, FB200_T_MIX_OUT_NORM = 24,
+  FB200_T_MIX_DKV = 25, FB200_T_MIX_DKV_NORM = 26, FB200_T_MIX_UK = 27, FB200_T_MIX_UV = 28
 } fb200_llama_tensor;
 
 FB200_API int fb200_llama_create(fb200_device* dev, const fb200_llama_config* cfg, fb200_llama** out);
 FB200_API int fb200_llama_free(fb200_llama* m);
+
+/* ---- decoders made of token-mixer layers (no counterpart in the reference) ----------------------
+ * The same object, entry points and generation loops over another kind of layer: with
+ * h = rms_norm(x) (one norm, FB200_T_ATTN_NORM), x <- x + (mixer(h) + ffn(h)), ffn = down(silu(gate h) *
+ * (up h)) or absent. Weights are dense ([out, in], BF16 or F32 bytes). `compute` selects the precision:
+ * FB200_COMPUTE_BF16 keeps weights, the latent cache and the operands of products of several rows in
+ * bf16 with 32-bit accumulation; the residual stream, norms, positions, attention scores and
+ * weights, convolution sums, decays and recurrent states are f32 in both. FB200_COMPUTE_F32 runs everything in f32.
+ *   FB200_MIX_DELTA   gated delta rule: q, k (kv_heads x dim), v (heads x vdim) pass a causal
+ *                     depthwise convolution of `conv` taps and SiLU, q and k become unit vectors (q
+ *                     x dim^-1/2); per head S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q with
+ *                     g = exp(-exp(A_log) softplus(decay + dt_bias)), beta = sigmoid(beta projection);
+ *                     o is RMS-normalised over vdim, x FB200_T_MIX_OUT_NORM, x silu(gate).
+ *   FB200_MIX_LATENT  latent attention: FB200_T_MIX_DKV gives kv_rank latent rows (RMS-normalised) and rot_dim
+ *                     rows of a key part shared by the heads (rotated); key n = [uk_n c, key part], value n =
+ *                     uv_n c; rotate-half positions on the last rot_dim of every query head; scores
+ *                     x scale over the last `window` positions (0: all); head n x sigmoid(gate_n).
+ *                     kv_from >= 0: the layer reads the cache of that earlier latent layer (same kv_rank,
+ *                     rot_dim and rotation) and has no FB200_T_MIX_DKV of its own.
+ * Recurrent states cannot be rewound: fb200_llama_truncate accepts 0 and the current length. */
+typedef enum fb200_mixer_kind { FB200_MIX_DELTA = 1, FB200_MIX_LATENT = 2 } fb200_mixer_kind;
+typedef enum fb200_compute { FB200_COMPUTE_BF16 = 0, FB200_COMPUTE_F32 = 1 } fb200_compute;
+typedef struct fb200_layer_config {
+  int mixer;                                   /* fb200_mixer_kind */
+  int ffn;                                     /* width of the feed-forward, 0: none */
+  int heads, kv_heads, dim, vdim;              /* kv_heads: delta rule only */
+  int conv;                                    /* delta rule: taps of the short convolution */
+  int kv_rank, rot_dim, window, kv_from;       /* latent attention; kv_from -1: a cache of its own */
+  float rope_base, scale;
+} fb200_layer_config;
+/* cfg: n_layer, hidden, vocab, max_seq_len, max_batch and rms_eps are read; layers[n_layer]. */
+FB200_API int fb200_llama_create_layers(fb200_device* dev, const fb200_llama_config* cfg,
+                                        const fb200_layer_config* layers, int compute, fb200_llama** out);
 /* Tensor names of raw/mod.rs:473-646: blk.{i}.attn_q.weight ... ; norms are f32 vectors
  * (ggml_type FB200_F32), everything else raw GGUF blocks of shape [N, K]. `layer` is ignored
  * for the three model-level tensors. Missing FB200_T_OUTPUT ties it to the embedding
@@ -343,6 +381,10 @@ FB200_API int fb200_llama_generate_sampled(fb200_llama* m, const uint32_t* token
 /* Device pointer of the last forward pass's logits, f32 [batch, vocab] (tensor parallel:
  * [batch, vocab / size], this rank's rows of the output head). */
 FB200_API int fb200_llama_logits_dev(const fb200_llama* m, const float** logits_dev);
+
+/* Logits of chosen rows of the last forward pass (row = batch index * seq + position inside the pass),
+ * f32 [n, vocab] into logits_host: a pass itself forms the logits of its last positions only. */
+FB200_API int fb200_llama_logits_at(fb200_llama* m, const int* rows_host, int n, float* logits_host);
 
 /* ---- tensor parallelism (no counterpart in the reference, which runs one device) ------------
  * One process and one device handle per GPU. Rank 0 makes an id (FB200_COMM_ID_BYTES bytes) and

@@ -20,8 +20,8 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.environ.get("FB200_LIB_PATH") or os.path.join(_HERE, "libfusor_b200.so")
 
 # ggml type ids (fusor-ml/gguf/src/lib.rs:35-50)
-F32, F16, Q4_0, Q5_0, Q8_0, Q4_K, Q5_K, Q6_K = 0, 1, 2, 6, 8, 12, 13, 14
-BLOCK = {F32: (1, 4), F16: (1, 2), Q4_0: (32, 18), Q5_0: (32, 22), Q8_0: (32, 34),
+F32, F16, Q4_0, Q5_0, Q8_0, Q4_K, Q5_K, Q6_K, BF16 = 0, 1, 2, 6, 8, 12, 13, 14, 30
+BLOCK = {F32: (1, 4), F16: (1, 2), BF16: (1, 2), Q4_0: (32, 18), Q5_0: (32, 22), Q8_0: (32, 34),
          Q4_K: (256, 144), Q5_K: (256, 176), Q6_K: (256, 210)}
 
 OK = 0
@@ -72,6 +72,17 @@ class LlamaConfig(C.Structure):
                 ("rope_original_ctx", C.c_int)]
 
 
+class LayerConfig(C.Structure):
+    """fb200_layer_config: one token-mixer layer (fb200_llama_create_layers)."""
+    _fields_ = [("mixer", C.c_int), ("ffn", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int),
+                ("vdim", C.c_int), ("conv", C.c_int), ("kv_rank", C.c_int), ("rot_dim", C.c_int), ("window", C.c_int),
+                ("kv_from", C.c_int), ("rope_base", C.c_float), ("scale", C.c_float)]
+
+
+MIX_DELTA, MIX_LATENT = 1, 2
+COMPUTE = {"bfloat16": 0, "float32": 1}
+
+
 EXPORTS = [
     "fb200_device_create", "fb200_device_destroy", "fb200_device_synchronize", "fb200_last_error",
     "fb200_launch_count", "fb200_device_status", "fb200_device_clear_status",
@@ -86,6 +97,7 @@ EXPORTS = [
     "fb200_kv_cache_buffers", "fb200_flash_attention", "fb200_llama_create", "fb200_llama_free",
     "fb200_llama_set_tensor", "fb200_llama_set_rope_freqs", "fb200_llama_reset", "fb200_llama_truncate", "fb200_llama_position", "fb200_llama_forward",
     "fb200_llama_generate_greedy", "fb200_llama_logits_dev", "fb200_llama_set_tensor_parallel",
+    "fb200_llama_create_layers", "fb200_llama_logits_at",
     "fb200_comm_unique_id", "fb200_comm_create", "fb200_comm_destroy", "fb200_comm_all_reduce_sum",
     "fb200_comm_exchange_handle", "fb200_comm_exchange_attach", "fb200_exchange_wait_check",
 ]
@@ -159,6 +171,8 @@ def load_library():
         "fb200_llama_generate_greedy": (i32, [vp, vp, i32, i32, vp]),
         "fb200_llama_logits_dev": (i32, [vp, pp]),
         "fb200_llama_set_tensor_parallel": (i32, [vp, vp]),
+        "fb200_llama_create_layers": (i32, [vp, C.POINTER(LlamaConfig), C.POINTER(LayerConfig), i32, pp]),
+        "fb200_llama_logits_at": (i32, [vp, vp, i32, vp]),
         "fb200_comm_unique_id": (i32, [vp, sz]),
         "fb200_comm_create": (i32, [vp, i32, i32, vp, sz, pp]),
         "fb200_comm_destroy": (i32, [vp]),
@@ -582,35 +596,17 @@ class Comm:
             self.h = None
 
 
-class Llama:
-    """Llama-architecture decoder (kalosm-llama Model::forward, raw/mod.rs:851-1049).
-
-    With `comm` the model is one rank of a tensor-parallel group: pass the WHOLE model's head and
-    FFN sizes; the local counts (divided by comm.size) go to the library, and `set_tensor` expects
-    this rank's shards (see `kalosm_b200.tp`)."""
+class Decoder:
+    """A decoder on the device: the session (KV caches or recurrent states, position), forward passes and generation
+    loops shared by all architectures. `kalosm_b200.models.load_model` builds one from a checkpoint."""
 
     TENSORS = {"token_embd": 0, "output": 1, "attn_q": 2, "attn_k": 3, "attn_v": 4,
                "attn_output": 5, "ffn_gate": 6, "ffn_up": 7, "ffn_down": 8, "attn_norm": 9,
-               "ffn_norm": 10, "output_norm": 11}
-
-    def __init__(self, device: Device, *, n_layer, hidden, ffn, n_head, n_kv_head, head_dim, vocab,
-                 max_seq_len, max_batch=1, rms_eps=1e-5, rope_theta=500000.0, rope_scaling=None, comm=None):
-        self.device = device
-        self.comm = comm
-        tp = comm.size if comm is not None else 1
-        if n_head % tp or n_kv_head % tp or ffn % tp or vocab % tp:
-            raise FusorError(ERR_INVALID_SHAPE, f"heads {n_head}/{n_kv_head}, ffn {ffn} and vocab {vocab} must be "
-                                                f"divisible by the {tp} tensor-parallel ranks")
-        n_head, n_kv_head, ffn = n_head // tp, n_kv_head // tp, ffn // tp
-        factor, low, high, orig = (0.0, 1.0, 4.0, max_seq_len) if rope_scaling is None else rope_scaling
-        self.cfg = LlamaConfig(n_layer, hidden, ffn, n_head, n_kv_head, head_dim, vocab, max_seq_len,
-                               max_batch, rms_eps, rope_theta, factor, low, high, orig)
-        out = C.c_void_p()
-        device._check(device.lib.fb200_llama_create(device.h, C.byref(self.cfg), C.byref(out)))
-        self.h = out.value
-        self.vocab = vocab // tp  # rows of the output head on this rank = width of the logits it returns
-        if comm is not None:
-            device._check(device.lib.fb200_llama_set_tensor_parallel(self.h, comm.h))
+               "ffn_norm": 10, "output_norm": 11,
+               "mix_q": 12, "mix_k": 13, "mix_v": 14, "mix_gate": 15, "mix_out": 16, "mix_beta": 17, "mix_decay": 18,
+               "mix_q_conv": 19, "mix_k_conv": 20, "mix_v_conv": 21, "mix_a_log": 22, "mix_dt_bias": 23,
+               "mix_out_norm": 24, "mix_dkv": 25, "mix_dkv_norm": 26, "mix_uk": 27, "mix_uv": 28}
+    h = None
 
     def set_tensor(self, name: str, layer: int, ggml_type: int, shape, raw) -> None:
         raw = np.ascontiguousarray(raw)
@@ -620,11 +616,6 @@ class Llama:
         d = self.device
         d._check(d.lib.fb200_llama_set_tensor(self.h, layer, self.TENSORS[name], ggml_type, n, k,
                                               _hp(raw8), raw8.size))
-
-    def set_rope_freqs(self, weights) -> None:
-        """rope_freqs.weight of a checkpoint: per-frequency factors multiplied into the inverse frequencies."""
-        w = np.ascontiguousarray(weights, dtype=np.float32).reshape(-1)
-        self.device._check(self.device.lib.fb200_llama_set_rope_freqs(self.h, _hp(w), w.size))
 
     def reset(self) -> None:
         self.device._check(self.device.lib.fb200_llama_reset(self.h))
@@ -651,6 +642,13 @@ class Llama:
         d._check(d.lib.fb200_llama_forward(self.h, _hp(t), batch, seq, _hp(logits), _hp(nxt)))
         return logits, nxt
 
+    def logits_at(self, rows) -> np.ndarray:
+        """Logits [len(rows), vocab] of chosen rows of the last `forward` (row = batch index * seq + position in the pass)."""
+        r = np.ascontiguousarray(rows, dtype=np.int32).reshape(-1)
+        out = np.empty((r.size, self.vocab), dtype=np.float32)
+        self.device._check(self.device.lib.fb200_llama_logits_at(self.h, _hp(r), r.size, _hp(out)))
+        return out
+
     def generate_greedy(self, tokens, steps: int) -> np.ndarray:
         t = np.ascontiguousarray(tokens, dtype=np.uint32).reshape(-1)
         out = np.empty((t.size, steps), dtype=np.uint32)
@@ -676,3 +674,48 @@ class Llama:
             self.free()
         except Exception:
             pass
+
+
+class Llama(Decoder):
+    """Llama-architecture decoder (kalosm-llama Model::forward, raw/mod.rs:851-1049).
+
+    With `comm` the model is one rank of a tensor-parallel group: pass the WHOLE model's head and
+    FFN sizes; the local counts (divided by comm.size) go to the library, and `set_tensor` expects
+    this rank's shards (see `kalosm_b200.tp`)."""
+
+    def __init__(self, device: Device, *, n_layer, hidden, ffn, n_head, n_kv_head, head_dim, vocab,
+                 max_seq_len, max_batch=1, rms_eps=1e-5, rope_theta=500000.0, rope_scaling=None, comm=None):
+        self.device = device
+        self.comm = comm
+        tp = comm.size if comm is not None else 1
+        if n_head % tp or n_kv_head % tp or ffn % tp or vocab % tp:
+            raise FusorError(ERR_INVALID_SHAPE, f"heads {n_head}/{n_kv_head}, ffn {ffn} and vocab {vocab} must be "
+                                                f"divisible by the {tp} tensor-parallel ranks")
+        n_head, n_kv_head, ffn = n_head // tp, n_kv_head // tp, ffn // tp
+        factor, low, high, orig = (0.0, 1.0, 4.0, max_seq_len) if rope_scaling is None else rope_scaling
+        self.cfg = LlamaConfig(n_layer, hidden, ffn, n_head, n_kv_head, head_dim, vocab, max_seq_len,
+                               max_batch, rms_eps, rope_theta, factor, low, high, orig)
+        out = C.c_void_p()
+        device._check(device.lib.fb200_llama_create(device.h, C.byref(self.cfg), C.byref(out)))
+        self.h = out.value
+        self.vocab = vocab // tp  # rows of the output head on this rank = width of the logits it returns
+        if comm is not None:
+            device._check(device.lib.fb200_llama_set_tensor_parallel(self.h, comm.h))
+
+    def set_rope_freqs(self, weights) -> None:
+        """rope_freqs.weight of a checkpoint: per-frequency factors multiplied into the inverse frequencies."""
+        w = np.ascontiguousarray(weights, dtype=np.float32).reshape(-1)
+        self.device._check(self.device.lib.fb200_llama_set_rope_freqs(self.h, _hp(w), w.size))
+
+
+class HybridDecoder(Decoder):
+    """A decoder of token-mixer layers over dense weights (fb200_llama_create_layers). `layers` is a list of
+    keyword dictionaries with the fields of LayerConfig; `compute` is "bfloat16" or "float32"."""
+
+    def __init__(self, device: Device, *, hidden, vocab, layers, max_seq_len, max_batch=1, rms_eps=1e-5, compute="bfloat16"):
+        self.device, self.comm, self.vocab = device, None, vocab
+        self.cfg = LlamaConfig(n_layer=len(layers), hidden=hidden, vocab=vocab, max_seq_len=max_seq_len, max_batch=max_batch, rms_eps=rms_eps)
+        self.layers = (LayerConfig * len(layers))(*[LayerConfig(**dict({"kv_from": -1}, **kw)) for kw in layers])
+        out = C.c_void_p()
+        device._check(device.lib.fb200_llama_create_layers(device.h, C.byref(self.cfg), self.layers, COMPUTE[compute], C.byref(out)))
+        self.h = out.value

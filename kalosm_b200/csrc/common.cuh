@@ -1,6 +1,7 @@
 // Internal definitions shared by the translation units of libfusor_b200.so.
 #pragma once
 
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 
@@ -73,7 +74,7 @@ struct fb200_qmatrix {
   size_t data_bytes = 0;
   int ntiles = 0;   // ceil(N / 16)
   int ngroups = 0;  // K groups per tile (128 weights for 32-element blocks, 256 for K-quants)
-  bool tiled = false;  // false: `data` holds raw row-major bytes (F32/F16/Q5_0/Q5_K)
+  bool tiled = false;  // false: `data` holds raw row-major bytes (F32/F16/BF16/Q5_0/Q5_K)
 };
 
 int fb200_fail(fb200_device* dev, int code, const char* fmt, ...);
@@ -172,6 +173,7 @@ inline bool block_geom(uint32_t type, int* elems, int* bytes) {
     case FB200_Q6_K: *elems = 256; *bytes = 210; return true;
     case FB200_F32: *elems = 1; *bytes = 4; return true;
     case FB200_F16: *elems = 1; *bytes = 2; return true;
+    case FB200_BF16: *elems = 1; *bytes = 2; return true;
     default: return false;
   }
 }

@@ -214,6 +214,7 @@ __device__ inline float raw_elem(uint32_t type, const uint8_t* raw, uint64_t idx
   switch (type) {
     case FB200_F32: return ((const float*)raw)[idx];
     case FB200_F16: return __half2float(((const __half*)raw)[idx]);
+    case FB200_BF16: return __bfloat162float(((const __nv_bfloat16*)raw)[idx]);
     case FB200_Q5_0: return deq_q5_0(raw + (idx >> 5) * 22, (int)(idx & 31));
     default: return deq_q5k(raw + (idx >> 8) * 176, (int)(idx & 255));
   }

@@ -12,9 +12,7 @@
 #include <cstring>
 #include <memory>
 
-#include "common.cuh"
-#include "fused_step.cuh"
-#include "packed_act.cuh"
+#include "decoder.cuh"
 
 void fb200_rope_tables_host(int head_dim, int ctx, float theta, float factor, float low_ff,
                             float high_ff, int original_ctx, const float* freq_weight,
@@ -44,7 +42,6 @@ int fb200_attention_nsplit(const fb200_device* dev, int b, int hkv, int groups, 
 int fb200_launch_attention_decode_args(fb200_device* dev, const fb200_dec_args& a, int d);
 bool fb200_qgemv1_fits(const fb200_qmatrix* w);
 int fb200_attention_scratch_bytes(int b, int h, int sq, int d, int nsplit, size_t* out);
-struct fb200_comm;
 int fb200_comm_all_reduce(fb200_comm* c, float* buf, size_t n);
 int fb200_comm_all_gather_bytes(fb200_comm* c, const void* in, void* out, size_t bytes);
 int fb200_comm_rank(const fb200_comm* c);
@@ -58,13 +55,6 @@ int fb200_launch_sampler(fb200_device* dev, const float* logits, size_t rows, si
                          uint32_t* ids, uint32_t* also0, size_t stride0, uint32_t* also1, size_t stride1);
 
 namespace {
-
-struct LayerW {
-  fb200_qmatrix *wq = nullptr, *wk = nullptr, *wv = nullptr, *wo = nullptr;
-  fb200_qmatrix *gate = nullptr, *up = nullptr, *down = nullptr, *gate_up = nullptr;
-  float *attn_norm = nullptr, *ffn_norm = nullptr;
-  __half *kc = nullptr, *vc = nullptr;  // [max_batch, Hkv, max_seq, D]
-};
 
 // q [rows, H*D] rotated in place; k rotated and v copied into the fp16 cache at position
 // *pos + s. Row = b * S + s. RoPE pairs are interleaved (2p, 2p+1) as in
@@ -138,63 +128,6 @@ __global__ void advance_kernel(uint32_t* __restrict__ next, uint32_t* __restrict
 
 }  // namespace
 
-struct fb200_llama {
-  fb200_device* dev = nullptr;
-  fb200_llama_config cfg{};
-  fb200_qmatrix *token_embd = nullptr, *output = nullptr;
-  float* output_norm = nullptr;
-  std::vector<LayerW> layers;
-  float *rope_cos = nullptr, *rope_sin = nullptr;
-  bool finalized = false;
-  int pos = 0;
-  // activation buffers, sized for `rows_cap` rows
-  size_t rows_cap = 0;
-  float *x = nullptr, *xn = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *att = nullptr,
-        *attn_out = nullptr, *hbuf = nullptr, *gbuf = nullptr, *last = nullptr, *logits = nullptr;
-  float* att_part = nullptr;
-  size_t att_part_bytes = 0;
-  uint32_t *ids = nullptr, *next = nullptr, *hist = nullptr;
-  int hist_cap = 0;
-  // every token fed to or produced by the model since the last reset, [max_batch, max_seq_len + 1]:
-  // the penalty window of the samplers
-  uint32_t* tok_hist = nullptr;
-  float* mu_dev = nullptr;  // [max_batch] Mirostat 2 state of a sampled decode
-  int *pos_dev = nullptr, *step_dev = nullptr;
-  unsigned long long* argmax_key = nullptr;
-  int* att_done = nullptr;  // arrival counters of the attention splits, one per (batch, kv head)
-  // single-row step: activation rows travel between kernels in the products' operand form
-  fb200_packed_act px, patt, pv, ph;  // residual stream, attention output, attn_out + x, SwiGLU output
-  // the same rows (and q / k / v, the residual stream and the attention projection as f32) as flagged
-  // rows for the barrier-free variants of the persistent kernel: one slab, zero at creation
-  uint8_t* ll_slab = nullptr;
-  fb200_ll_act px_ll, patt_ll, pv_ll, ph_ll;
-  uint2 *q_ll = nullptr, *k_ll = nullptr, *v_ll = nullptr, *x_ll = nullptr, *attn_ll = nullptr;
-  // FB200_FUSED_LL=1 selects the barrier-free variants. Off by default: they are correct (parity
-  // tests run both forms) but measured slower so far (2.2 - 2.6 ms per step of the 8B-shaped model
-  // against 2.03 ms with grid barriers): the trip a flagged row saves at each phase boundary is
-  // outweighed by slower epilogues (8-byte flagged stores), the 86 KB polled row in front of the
-  // down projection and a product loop that gets fewer registers.
-  bool fused_flagged = false;
-  bool fused_is_flagged = false;  // the current program uses the flagged rows
-  bool used_key = false;  // the last forward pass left its greedy id in argmax_key, not in next
-  // CUDA graph of a single-token step, per batch size
-  cudaGraphExec_t graph_exec = nullptr;
-  int graph_batch = 0;
-  uint64_t graph_kernels = 0;  // kernels inside the captured step
-  uint64_t graph_gen = 0;      // the handle's scratch generation the capture recorded addresses of
-  // single-sequence step as one persistent kernel: its program (host and device copies)
-  bool fused_enabled = true;   // FB200_FUSED=0 keeps the multi-kernel step
-  bool fused_valid = false;    // the program matches the current buffers
-  bool fused_usable = false;
-  std::vector<fb200_fused_phase> prog_host;
-  fb200_fused_phase* prog_dev = nullptr;
-  // tensor parallelism: cfg holds the local head / ffn counts; the output head has vocab_local rows
-  fb200_comm* comm = nullptr;
-  int tp_rank = 0, tp_size = 1, vocab_local = 0;
-  float* best_val = nullptr;            // [max_batch] value of the local greedy candidate
-  unsigned long long* best_pair = nullptr;  // [(1 + size) * max_batch] (value, global id) pairs
-};
-
 namespace {
 
 int alloc_f(fb200_device* dev, float** p, size_t n) {
@@ -211,6 +144,14 @@ int ensure_rows(fb200_llama* m, size_t rows) {
   if (m->graph_exec) { cudaGraphExecDestroy(m->graph_exec); m->graph_exec = nullptr; }
   m->fused_valid = false;  // the program holds pointers into these buffers
   int rc;
+  if (m->hybrid) {
+    if ((rc = fb200_hybrid_ensure_rows(m, rows))) return rc;
+    if (m->ids) cudaFree(m->ids);
+    m->ids = nullptr;
+    FB_CUDA(dev, cudaMalloc(&m->ids, rows * sizeof(uint32_t)));
+    m->rows_cap = rows;
+    return FB200_OK;
+  }
   if ((rc = alloc_f(dev, &m->x, rows * c.hidden))) return rc;
   if ((rc = alloc_f(dev, &m->xn, rows * c.hidden))) return rc;
   if ((rc = alloc_f(dev, &m->q, rows * c.n_head * c.head_dim))) return rc;
@@ -232,6 +173,11 @@ int finalize(fb200_llama* m) {
   const auto& c = m->cfg;
   if (!m->token_embd || !m->output_norm)
     return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "llama: token_embd / output_norm not set");
+  if (m->hybrid) {
+    const int rc = fb200_hybrid_finalize(m);
+    if (!rc) m->finalized = true;
+    return rc;
+  }
   if (m->tp_size > 1 && !m->output)
     return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "llama: a tensor-parallel model needs its shard of the output head");
   for (int i = 0; i < c.n_layer; ++i) {
@@ -286,7 +232,7 @@ int build_fused_program(fb200_llama* m) {
   const auto& c = m->cfg;
   m->fused_usable = false;
   m->fused_valid = true;
-  if (!m->fused_enabled || !decode1_supported(m)) return FB200_OK;
+  if (m->hybrid || !m->fused_enabled || !decode1_supported(m)) return FB200_OK;
   if (m->tp_size > 1 && !fb200_comm_exchange_ready(m->comm, m->cfg.hidden)) return FB200_OK;
   if (m->tp_size > 1)  // the exchange variants of the kernel exist for K-quant weights only
     for (const auto& L : m->layers)
@@ -513,7 +459,8 @@ __global__ void pick_candidate_kernel(const unsigned long long* __restrict__ all
   next[b] = best ? (uint32_t)(best & 0xFFFFFFFFu) : 0xFFFFFFFFu;
 }
 
-int run_forward(fb200_llama* m, int batch, int seq) {
+// commit = false: a dry run (a layer with a recurrent state leaves it as it was).
+int run_forward(fb200_llama* m, int batch, int seq, bool commit = true) {
   m->used_key = false;
   fb200_device* dev = m->dev;
   const auto& c = m->cfg;
@@ -521,6 +468,7 @@ int run_forward(fb200_llama* m, int batch, int seq) {
   const int E = c.hidden, H = c.n_head, HK = c.n_kv_head, D = c.head_dim;
   int rc;
   if ((rc = fb200_embedding_lookup(dev, m->token_embd, m->ids, rows, m->x))) return rc;
+  if (m->hybrid) return fb200_hybrid_forward(m, batch, seq, commit);
   const float scale = (float)(1.0 / sqrt((double)D));  // attention_layer.rs:674
   const int nsplit = fb200_attention_nsplit(dev, batch, HK, H / HK, seq, seq > 1 ? seq : c.max_seq_len);
   size_t part_bytes;
@@ -694,7 +642,7 @@ int ensure_graph(fb200_llama* m, int batch) {
   if (m->graph_exec && m->graph_batch == batch && m->graph_gen == dev->scratch_gen) return FB200_OK;
   if (m->graph_exec) { cudaGraphExecDestroy(m->graph_exec); m->graph_exec = nullptr; }
   // make sure every lazily grown scratch buffer already has its final size
-  int rc = run_forward(m, batch, 1);
+  int rc = run_forward(m, batch, 1, false);
   if (rc) return rc;
   FB_CUDA(dev, cudaMemsetAsync(m->argmax_key, 0, 8, dev->stream));  // the warm-up pass left its maximum there
   FB_CUDA(dev, cudaStreamSynchronize(dev->stream));
@@ -729,8 +677,26 @@ int finish_blocking(fb200_llama* m) {
 
 }  // namespace
 
-int fb200_launch_rms_norm(fb200_device* dev, const float* x, const float* res, const float* w,
-                          const float* b, float eps, size_t rows, size_t n, float* y);
+int fb200_decoder_session(fb200_llama* m) {
+  fb200_device* dev = m->dev;
+  const auto& c = m->cfg;
+  m->vocab_local = c.vocab;
+  FB_CUDA(dev, cudaMalloc(&m->last, (size_t)c.max_batch * c.hidden * 4));
+  FB_CUDA(dev, cudaMalloc(&m->logits, (size_t)c.max_batch * c.vocab * 4));
+  FB_CUDA(dev, cudaMalloc(&m->next, (size_t)c.max_batch * 4));
+  FB_CUDA(dev, cudaMalloc(&m->pos_dev, 4));
+  FB_CUDA(dev, cudaMalloc(&m->step_dev, 4));
+  m->hist_cap = c.max_seq_len;
+  FB_CUDA(dev, cudaMalloc(&m->hist, (size_t)c.max_batch * m->hist_cap * 4));
+  FB_CUDA(dev, cudaMemset(m->pos_dev, 0, 4));
+  FB_CUDA(dev, cudaMemset(m->step_dev, 0, 4));
+  FB_CUDA(dev, cudaMalloc(&m->tok_hist, (size_t)c.max_batch * (c.max_seq_len + 1) * 4));
+  FB_CUDA(dev, cudaMemset(m->tok_hist, 0, (size_t)c.max_batch * (c.max_seq_len + 1) * 4));
+  FB_CUDA(dev, cudaMalloc(&m->mu_dev, (size_t)c.max_batch * 4));
+  FB_CUDA(dev, cudaMalloc(&m->argmax_key, 8));
+  FB_CUDA(dev, cudaMemset(m->argmax_key, 0, 8));
+  return FB200_OK;
+}
 
 extern "C" {
 
@@ -748,7 +714,6 @@ int fb200_llama_create(fb200_device* dev, const fb200_llama_config* cfg, fb200_l
   m->dev = dev;
   m->cfg = c;
   m->layers.resize(c.n_layer);
-  m->vocab_local = c.vocab;
   if (const char* e = getenv("FB200_FUSED")) m->fused_enabled = !(e[0] == '0' && e[1] == 0);
   std::vector<float> cs, sn;
   fb200_rope_tables_host(c.head_dim, c.max_seq_len, c.rope_theta, c.rope_factor,
@@ -764,22 +729,9 @@ int fb200_llama_create(fb200_device* dev, const fb200_llama_config* cfg, fb200_l
     FB_CUDA(dev, cudaMemset(L.kc, 0, kv));
     FB_CUDA(dev, cudaMemset(L.vc, 0, kv));
   }
-  FB_CUDA(dev, cudaMalloc(&m->last, (size_t)c.max_batch * c.hidden * 4));
-  FB_CUDA(dev, cudaMalloc(&m->logits, (size_t)c.max_batch * c.vocab * 4));
-  FB_CUDA(dev, cudaMalloc(&m->next, (size_t)c.max_batch * 4));
-  FB_CUDA(dev, cudaMalloc(&m->pos_dev, 4));
-  FB_CUDA(dev, cudaMalloc(&m->step_dev, 4));
-  m->hist_cap = c.max_seq_len;
-  FB_CUDA(dev, cudaMalloc(&m->hist, (size_t)c.max_batch * m->hist_cap * 4));
-  FB_CUDA(dev, cudaMemset(m->pos_dev, 0, 4));
-  FB_CUDA(dev, cudaMemset(m->step_dev, 0, 4));
-  FB_CUDA(dev, cudaMalloc(&m->tok_hist, (size_t)c.max_batch * (c.max_seq_len + 1) * 4));
-  FB_CUDA(dev, cudaMemset(m->tok_hist, 0, (size_t)c.max_batch * (c.max_seq_len + 1) * 4));
-  FB_CUDA(dev, cudaMalloc(&m->mu_dev, (size_t)c.max_batch * 4));
+  if ((rc = fb200_decoder_session(m.get()))) return rc;
   FB_CUDA(dev, cudaMalloc(&m->att_done, (size_t)c.max_batch * c.n_kv_head * sizeof(int)));
   FB_CUDA(dev, cudaMemset(m->att_done, 0, (size_t)c.max_batch * c.n_kv_head * sizeof(int)));
-  FB_CUDA(dev, cudaMalloc(&m->argmax_key, 8));
-  FB_CUDA(dev, cudaMemset(m->argmax_key, 0, 8));
   {
     // packed rows, zero beyond the logical length up to the next multiple of 256 (and one
     // 16-row tile of slack for the producers' last tile)
@@ -836,6 +788,7 @@ int fb200_llama_free(fb200_llama* m) {
   cudaStreamSynchronize(dev->stream);
   if (m->graph_exec) cudaGraphExecDestroy(m->graph_exec);
   if (m->prog_dev) cudaFree(m->prog_dev);
+  fb200_hybrid_free(m);
   for (auto& L : m->layers) {
     fb200_qmatrix* qs[] = {L.wq, L.wk, L.wv, L.wo, L.gate, L.up, L.down, L.gate_up};
     for (auto* q : qs) if (q) fb200_qmatrix_free(q);
@@ -849,7 +802,7 @@ int fb200_llama_free(fb200_llama* m) {
   void* bufs[] = {m->output_norm, m->rope_cos, m->rope_sin, m->x, m->xn, m->q, m->k, m->v, m->att,
                   m->attn_out, m->hbuf, m->gbuf, m->last, m->logits, m->att_part, m->ids, m->next,
                   m->hist, m->pos_dev, m->step_dev, m->argmax_key, m->att_done, m->best_val, m->best_pair,
-                  m->tok_hist, m->mu_dev, m->ll_slab};
+                  m->tok_hist, m->mu_dev, m->ll_slab, m->row_logits};
   for (void* b : bufs) if (b) cudaFree(b);
   for (fb200_packed_act* p : {&m->px, &m->patt, &m->pv, &m->ph}) {
     void* pb[] = {p->limbs, p->xsc, p->xss, p->sumsq};
@@ -867,6 +820,7 @@ int fb200_llama_set_tensor(fb200_llama* m, int layer, int which, uint32_t ggml_t
   if (rc) return rc;
   const auto& c = m->cfg;
   if (m->finalized) return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "llama: tensors are frozen after the first forward pass");
+  if (m->hybrid) return fb200_hybrid_set_tensor(m, layer, which, ggml_type, n, k, bytes_host, nbytes);
   if (which >= FB200_T_ATTN_NORM) {
     const uint64_t len = n * (k ? k : 1);
     if (ggml_type != FB200_F32 || len != (uint64_t)c.hidden || nbytes != len * 4)
@@ -915,6 +869,7 @@ int fb200_llama_set_rope_freqs(fb200_llama* m, const float* weights_host, size_t
   if (rc) return rc;
   const auto& c = m->cfg;
   if (m->finalized) return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "llama: the RoPE tables are frozen after the first forward pass");
+  if (m->hybrid) return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "llama: rope_freqs belong to Llama blocks");
   if (!weights_host || n != (size_t)c.head_dim / 2)
     return fb200_fail(dev, FB200_ERR_INVALID_SHAPE, "llama: rope_freqs needs head_dim / 2 = %d values, got %zu", c.head_dim / 2, n);
   std::vector<float> cs, sn;
@@ -944,6 +899,8 @@ int fb200_llama_truncate(fb200_llama* m, int len) {
   if (rc) return rc;
   if (len < 0 || len > m->pos)
     return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "llama: cannot truncate %d positions to %d", m->pos, len);
+  if (len != 0 && len != m->pos && fb200_hybrid_recurrent(m))
+    return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "llama: a recurrent state cannot be rewound from %d to %d positions (only to 0)", m->pos, len);
   // the caches keep their rows; positions >= len are overwritten as the sequence grows again
   m->pos = len;
   FB_CUDA(dev, cudaMemcpyAsync(m->pos_dev, &m->pos, 4, cudaMemcpyHostToDevice, dev->stream));
@@ -992,6 +949,8 @@ int fb200_llama_forward(fb200_llama* m, const uint32_t* tokens_host, int batch, 
     if ((rc = launch_advance(m, batch, seq, false))) return rc;
   }
   m->pos += seq;
+  m->last_batch = batch;
+  m->last_seq = seq;
   if (logits_host)
     FB_CUDA(dev, cudaMemcpyAsync(logits_host, m->logits, (size_t)batch * m->vocab_local * 4, cudaMemcpyDeviceToHost, dev->stream));
   if (next_host)
@@ -1045,6 +1004,8 @@ int fb200_llama_generate_greedy(fb200_llama* m, const uint32_t* tokens_host, int
   FB_CUDA(dev, cudaMemcpy2DAsync(m->tok_hist + m->pos + 1, (size_t)(c.max_seq_len + 1) * 4, m->hist,
                                  (size_t)m->hist_cap * 4, (size_t)steps * 4, batch, cudaMemcpyDeviceToDevice, dev->stream));
   m->pos += steps;
+  m->last_batch = batch;
+  m->last_seq = 1;
   // hist is [batch, hist_cap]; gather the first `steps` columns
   std::vector<uint32_t> tmp((size_t)batch * m->hist_cap);
   FB_CUDA(dev, cudaMemcpyAsync(tmp.data(), m->hist, tmp.size() * 4, cudaMemcpyDeviceToHost, dev->stream));
@@ -1106,6 +1067,8 @@ int fb200_llama_generate_sampled(fb200_llama* m, const uint32_t* tokens_host, in
       return rc;
   }
   m->pos += steps;
+  m->last_batch = batch;
+  m->last_seq = 1;
   std::vector<uint32_t> tmp((size_t)batch * steps);
   FB_CUDA(dev, cudaMemcpy2DAsync(tmp.data(), (size_t)steps * 4, m->tok_hist + pos0 + 1, hstride * 4, (size_t)steps * 4,
                                  batch, cudaMemcpyDeviceToHost, dev->stream));
@@ -1135,6 +1098,32 @@ int fb200_llama_set_tensor_parallel(fb200_llama* m, fb200_comm* comm) {
     FB_CUDA(dev, cudaMalloc(&m->best_pair, (size_t)(1 + size) * m->cfg.max_batch * 8));
   }
   return FB200_OK;
+}
+
+int fb200_llama_logits_at(fb200_llama* m, const int* rows_host, int n, float* logits_host) {
+  if (!m) return FB200_ERR_INVALID_ARGUMENT;
+  fb200_device* dev = m->dev;
+  int rc = fb200_bind(dev);
+  if (rc) return rc;
+  const auto& c = m->cfg;
+  if (n < 0 || (n && (!rows_host || !logits_host))) return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "logits_at: null argument");
+  const int rows = m->last_batch * m->last_seq;
+  if (!m->row_logits) FB_CUDA(dev, cudaMalloc(&m->row_logits, (size_t)m->vocab_local * 4));
+  for (int i = 0; i < n; ++i) {
+    const int r = rows_host[i];
+    if (r < 0 || r >= rows) return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "logits_at: row %d of a pass of %d rows", r, rows);
+    const float* src = m->logits + (size_t)(r / m->last_seq) * m->vocab_local;
+    if ((r + 1) % m->last_seq) {  // not a last position: its logits were not formed by the pass
+      src = m->row_logits;
+      if (m->hybrid) rc = fb200_hybrid_row_logits(m, (size_t)r, m->row_logits);
+      else rc = fb200_rms_norm_q_mat_mul(dev, m->x + (size_t)r * c.hidden, nullptr, m->output_norm, c.rms_eps, 1,
+                                         m->output ? m->output : m->token_embd, m->row_logits, nullptr);
+      if (rc) return rc;
+    }
+    FB_CUDA(dev, cudaMemcpyAsync(logits_host + (size_t)i * m->vocab_local, src, (size_t)m->vocab_local * 4, cudaMemcpyDeviceToHost, dev->stream));
+    FB_CUDA(dev, cudaStreamSynchronize(dev->stream));  // the next row overwrites the buffer
+  }
+  return finish_blocking(m);
 }
 
 int fb200_llama_logits_dev(const fb200_llama* m, const float** logits_dev) {

@@ -10,7 +10,7 @@ block size). Which tensor splits which way (one all-reduce per pair):
 import numpy as np
 
 # (elements, bytes) per block, fusor-ml/gguf/src/lib.rs:99-121
-BLOCK = {0: (1, 4), 1: (1, 2), 2: (32, 18), 6: (32, 22), 8: (32, 34), 12: (256, 144), 13: (256, 176), 14: (256, 210)}
+BLOCK = {0: (1, 4), 1: (1, 2), 2: (32, 18), 6: (32, 22), 8: (32, 34), 12: (256, 144), 13: (256, 176), 14: (256, 210), 30: (1, 2)}
 
 ROW_SPLIT = ("attn_q", "attn_k", "attn_v", "ffn_gate", "ffn_up", "output")
 COL_SPLIT = ("attn_output", "ffn_down")
