@@ -41,7 +41,7 @@
 #include <cuda.h>
 
 #include "attn_mma.cuh"
-#include "qgemv_common.cuh"
+#include "tcgen05.cuh"
 
 namespace {
 
@@ -69,84 +69,6 @@ struct XArgs {
 // descriptor strides (bytes) of the swizzled operands, and the layout code of the 128-byte swizzle
 constexpr uint32_t X_SW128 = 2;
 constexpr uint32_t X_BOX_BYTES = XK * 64 * 2;  // one TMA box: 64 keys x 64 dims of fp16 = 8 KB
-
-__device__ __forceinline__ bool x_wait(uint32_t bar, uint32_t parity, volatile int* dead, int* status) {
-  for (int it = 0; it < (1 << 22); ++it) {
-    uint32_t ok;
-    asm volatile(
-        "{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n"
-        "selp.u32 %0, 1, 0, p;\n}"
-        : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-    if (ok) return true;
-    if ((it & 255) == 255 && *dead) return false;
-  }
-  *dead = 1;
-  if (status) atomicExch(status, FB200_ERR_TIMEOUT);
-  return false;
-}
-__device__ __forceinline__ void mbar_arrive(uint32_t bar) {
-  asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
-}
-// Shared-memory matrix descriptor without swizzle: start address, leading and stride byte offsets
-// in 16-byte units, descriptor version 1.
-__device__ __forceinline__ uint64_t x_desc(uint32_t saddr, uint32_t lbo, uint32_t sbo, uint32_t layout = 0) {
-  return (uint64_t)((saddr & 0x3FFFFu) >> 4) | ((uint64_t)(lbo >> 4) << 16) | ((uint64_t)(sbo >> 4) << 32) | (1ull << 46) |
-         ((uint64_t)layout << 61);
-}
-// One box of a 3-D tensor map (dims, keys, sequence x KV head) into shared memory; completion is
-// counted in bytes on the mbarrier.
-__device__ __forceinline__ void x_tma_box(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
-  asm volatile(
-      "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
-      ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar) : "memory");
-}
-__device__ __forceinline__ void x_mma(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}"
-      ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
-}
-// The same with the A operand in tensor memory (row i of A in lane i, two fp16 values per column)
-__device__ __forceinline__ void x_mma_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}"
-      ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
-}
-__device__ __forceinline__ void x_commit(uint32_t bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ void x_ld32(uint32_t taddr, uint32_t (&v)[32]) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-      "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-        "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]),
-        "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]),
-        "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
-      : "r"(taddr) : "memory");
-}
-__device__ __forceinline__ void x_st32(uint32_t taddr, const uint32_t (&v)[32]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};"
-      ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]),
-        "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]), "r"(v[16]), "r"(v[17]),
-        "r"(v[18]), "r"(v[19]), "r"(v[20]), "r"(v[21]), "r"(v[22]), "r"(v[23]), "r"(v[24]), "r"(v[25]), "r"(v[26]),
-        "r"(v[27]), "r"(v[28]), "r"(v[29]), "r"(v[30]), "r"(v[31])
-      : "memory");
-}
-// 2^x, flushing denormals (2^-inf = 0)
-__device__ __forceinline__ float x_ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-// Byte offset of the 16-byte chunk `chunk` (8 K elements) of row `row` in a K-major operand whose K
-// extent is `kchunks` chunks: core matrices of a row group side by side along K, row groups behind.
-__device__ __forceinline__ uint32_t x_kmajor(int row, int chunk, int kchunks) {
-  return (uint32_t)((row >> 3) * (kchunks * 128) + chunk * 128 + (row & 7) * 16);
-}
 
 __global__ void __launch_bounds__(X_BLOCK, 2)
 attn_prefill_tc_kernel(const XArgs a, const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap) {
@@ -331,6 +253,9 @@ attn_prefill_tc_kernel(const XArgs a, const __grid_constant__ CUtensorMap kmap, 
 
     // ---- the last product, then normalise and store (nothing is stored after a wait has given up)
     if (ntiles > 0) {
+      // S of the last tile being complete says that O is complete up to the product two tiles back: the last two
+      // are waited for in turn (a parity wait must not start two phases behind)
+      if (ntiles > 1) x_wait(bar_o, (uint32_t)((ntiles - 2) & 1), dead, a.status);
       x_wait(bar_o, (uint32_t)((ntiles - 1) & 1), dead, a.status);
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     }

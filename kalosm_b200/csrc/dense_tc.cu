@@ -12,12 +12,10 @@
 //    output are the two halves of the same CTA, so they sit in the same TMEM lane BM columns apart.
 // Every wait is bounded (2^22 polls): a wait that gives up sets the device status word and a flag that makes the
 // other roles leave; TMEM is released on every path.
-#include <cuda.h>
-
 #include <algorithm>
 
 #include "dense.cuh"
-#include "qgemv_common.cuh"
+#include "tcgen05.cuh"
 
 namespace {
 
@@ -47,55 +45,10 @@ struct DenseTcArgs {
   int* status;
 };
 
-__device__ __forceinline__ bool dt_wait(uint32_t bar, uint32_t parity, volatile int* dead, int* status) {
-  for (int it = 0; it < (1 << 22); ++it) {
-    uint32_t ok;
-    asm volatile(
-        "{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n"
-        "selp.u32 %0, 1, 0, p;\n}"
-        : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-    if (ok) return true;
-    if ((it & 255) == 255 && *dead) return false;
-  }
-  *dead = 1;
-  if (status) atomicExch(status, FB200_ERR_TIMEOUT);
-  return false;
-}
-// The way out after a give-up: waits (bounded, whatever the flag says) for work this CTA has in flight, so that
-// neither copies into its shared memory nor products into its TMEM outlive it.
-__device__ __forceinline__ void dt_drain(uint32_t bar, uint32_t parity) {
-  for (int it = 0; it < (1 << 20); ++it) {
-    uint32_t ok;
-    asm volatile(
-        "{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n"
-        "selp.u32 %0, 1, 0, p;\n}"
-        : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-    if (ok) return;
-  }
-}
 // K-major operand with 128-byte swizzle: rows of 128 bytes, groups of 8 rows 1024 bytes apart, descriptor version 1
 __device__ __forceinline__ uint64_t dt_desc(uint32_t saddr) {
   return (uint64_t)((saddr & 0x3FFFFu) >> 4) | ((uint64_t)1 << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
 }
-__device__ __forceinline__ void dt_mma(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\n"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}"
-      ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
-}
-__device__ __forceinline__ void dt_box(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-      ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
-}
-__device__ __forceinline__ void dt_ld16(uint32_t taddr, uint32_t (&v)[16]) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-        "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
-      : "r"(taddr) : "memory");
-}
-
 template <int BM, int NH>
 __global__ void __launch_bounds__(TC_THREADS, BM <= 64 ? 2 : 1)
 dense_tc_kernel(const DenseTcArgs a, const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap) {
@@ -133,22 +86,22 @@ dense_tc_kernel(const DenseTcArgs a, const __grid_constant__ CUtensorMap wmap, c
       int issued = 0;
       for (int kb = 0; kb < a.kblocks; ++kb, ++issued) {
         const int s = kb % S::STAGES;
-        if (kb >= S::STAGES && !dt_wait(empty + 8 * s, (uint32_t)((kb / S::STAGES - 1) & 1), dead, a.status)) break;
+        if (kb >= S::STAGES && !x_wait(empty + 8 * s, (uint32_t)((kb / S::STAGES - 1) & 1), dead, a.status)) break;
         const uint32_t dst = smem_u32(sm + s * S::STAGE), bar = full + 8 * s;
         mbar_expect_tx(bar, S::STAGE);
-        dt_box(dst, &wmap, kb * TC_BK, r0, bar);
-        if (NH == 2) dt_box(dst + TC_BN * TC_BK * 2, &wmap, kb * TC_BK, r1, bar);
-        dt_box(dst + S::A_BYTES, &xmap, kb * TC_BK, m0, bar);
+        x_tma_box2(dst, &wmap, kb * TC_BK, r0, bar);
+        if (NH == 2) x_tma_box2(dst + TC_BN * TC_BK * 2, &wmap, kb * TC_BK, r1, bar);
+        x_tma_box2(dst + S::A_BYTES, &xmap, kb * TC_BK, m0, bar);
       }
       if (*dead)
-        for (int kb = max(0, issued - S::STAGES); kb < issued; ++kb) dt_drain(full + 8 * (kb % S::STAGES), (uint32_t)((kb / S::STAGES) & 1));
+        for (int kb = max(0, issued - S::STAGES); kb < issued; ++kb) x_drain(full + 8 * (kb % S::STAGES), (uint32_t)((kb / S::STAGES) & 1));
     }
   } else if (warp == TC_EPI_WARPS + 1) {
     if (lane == 0) {
       bool ok = true;
       for (int kb = 0; kb < a.kblocks && ok; ++kb) {
         const int s = kb % S::STAGES;
-        ok = dt_wait(full + 8 * s, (uint32_t)((kb / S::STAGES) & 1), dead, a.status);
+        ok = x_wait(full + 8 * s, (uint32_t)((kb / S::STAGES) & 1), dead, a.status);
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const uint32_t st = smem_u32(sm + s * S::STAGE);
@@ -156,17 +109,17 @@ dense_tc_kernel(const DenseTcArgs a, const __grid_constant__ CUtensorMap wmap, c
         for (int k = 0; k < TC_BK / 16; ++k)  // 32 bytes further inside the 128-byte rows per K step
 #pragma unroll
           for (int h = 0; h < NH; ++h)
-            dt_mma(tmem + (uint32_t)(h * BM), dt_desc(st + h * TC_BN * TC_BK * 2 + k * 32), dt_desc(st + S::A_BYTES + k * 32), S::IDESC,
+            x_mma(tmem + (uint32_t)(h * BM), dt_desc(st + h * TC_BN * TC_BK * 2 + k * 32), dt_desc(st + S::A_BYTES + k * 32), S::IDESC,
                    (kb | k) ? 1u : 0u);
-        asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(empty + 8 * s) : "memory");
+        x_commit(empty + 8 * s);
       }
-      asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(done) : "memory");
+      x_commit(done);
     }
   } else {
     // ---- epilogue: warp w reads TMEM lanes 32 (w % 4) .., columns of one half of the activation rows
     const int quad = warp & 3, ch = warp >> 2;
-    dt_wait(done, 0, dead, a.status);
-    if (*dead) dt_drain(done, 0);
+    x_wait(done, 0, dead, a.status);
+    if (*dead) x_drain(done, 0);
     else {
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const uint32_t tl = tmem + ((uint32_t)(32 * quad) << 16);
@@ -176,8 +129,8 @@ dense_tc_kernel(const DenseTcArgs a, const __grid_constant__ CUtensorMap wmap, c
         if (m0 + c >= a.m) break;
         const int lim = min(16, a.m - (m0 + c));
         uint32_t v0[16], v1[16];
-        dt_ld16(tl + (uint32_t)c, v0);
-        if (NH == 2) dt_ld16(tl + (uint32_t)(BM + c), v1);
+        x_ld16(tl + (uint32_t)c, v0);
+        if (NH == 2) x_ld16(tl + (uint32_t)(BM + c), v1);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         if (pair) {
           if (n0 + r < a.ff) {

@@ -53,6 +53,8 @@ struct fb200_hybrid {
   __nv_bfloat16 *hb = nullptr, *zb = nullptr;
   float *qn = nullptr, *kn = nullptr, *vn = nullptr, *gb = nullptr, *kq = nullptr, *o = nullptr;
   float *qa = nullptr, *part = nullptr;
+  __nv_bfloat16* kvx = nullptr;
+  size_t kvx_elems = 0;
 };
 
 namespace {
@@ -209,6 +211,11 @@ int make_layer(fb200_llama* m, int i) {
   return FB200_OK;
 }
 
+// A prompt pass long enough for the expansion of keys and values to pay (tensor-core attention over them)
+bool expanded(const fb200_hybrid* hy, const fb200_layer_config& c, int seq) {
+  return !hy->f32 && seq >= 16 && fb200_latent_prefill_covers(c.heads, c.dim, c.rot_dim, c.vdim, c.kv_rank, c.scale);
+}
+
 int run_layer(fb200_llama* m, MixerLayer& L, int batch, int seq, bool commit) {
   fb200_device* dev = m->dev;
   fb200_hybrid* hy = m->hybrid;
@@ -248,8 +255,13 @@ int run_layer(fb200_llama* m, MixerLayer& L, int batch, int seq, bool commit) {
     a.rope_cos = L.rope_cos; a.rope_sin = L.rope_sin; a.b = batch; a.s = seq; a.h = c.heads; a.d = c.dim; a.r = c.rot_dim; a.v = c.vdim;
     a.rk = c.kv_rank; a.rkp = L.rkp; a.window = c.window; a.scale = c.scale; a.pos_dev = m->pos_dev; a.pos = m->pos;
     a.z = z; a.ldz = hy->ldz; a.z_bf16 = !wide; a.qa = hy->qa; a.part = hy->part;
-    a.nsplit = fb200_latent_nsplit(dev, rows, c.heads, c.window, m->cfg.max_seq_len);
-    if ((rc = fb200_latent_rows(dev, a))) return rc;
+    if (expanded(hy, c, seq)) {
+      a.kvx = hy->kvx;
+      if ((rc = fb200_latent_append(dev, a)) || (rc = fb200_latent_prefill(dev, a, L.w_ukv))) return rc;
+    } else {
+      a.nsplit = fb200_latent_nsplit(dev, rows, c.heads, c.window, m->cfg.max_seq_len);
+      if ((rc = fb200_latent_rows(dev, a))) return rc;
+    }
   }
 
   fb200_dense_job out;
@@ -273,8 +285,11 @@ int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows) {
       heads = std::max(heads, (size_t)c.heads);
       kvh = std::max(kvh, (size_t)c.kv_heads);
     } else {
-      qa = std::max(qa, rows * c.heads * (size_t)(c.kv_rank + c.rot_dim));
-      part = std::max(part, std::max(rows * c.heads, (size_t)4 * dev->sm_count) * (size_t)(c.kv_rank + 2));
+      // rows of the latent-space path: all of them, or fewer where longer passes expand keys and values
+      const bool exp = expanded(hy, c, 16);
+      const size_t r = exp ? std::min(rows, (size_t)16 * m->cfg.max_batch) : rows;
+      qa = std::max(qa, r * c.heads * (size_t)(c.kv_rank + c.rot_dim));
+      part = std::max(part, std::max(r * c.heads, (size_t)4 * dev->sm_count) * (size_t)(c.kv_rank + 2));
     }
   }
   struct { void** p; size_t bytes; } bufs[] = {
@@ -311,6 +326,20 @@ int fb200_hybrid_forward(fb200_llama* m, int batch, int seq, bool commit) {
   fb200_device* dev = m->dev;
   fb200_hybrid* hy = m->hybrid;
   int rc;
+  size_t kvx = 0;
+  for (const auto& L : hy->layers)
+    if (L.c.mixer == FB200_MIX_LATENT && expanded(hy, L.c, seq)) {
+      const int before = L.c.window && L.c.window - 1 < m->pos ? L.c.window - 1 : m->pos;
+      kvx = std::max(kvx, (size_t)batch * (before + seq) * L.c.heads * (L.c.dim + L.c.vdim));
+    }
+  if (kvx > hy->kvx_elems) {
+    FB_CUDA(dev, cudaStreamSynchronize(dev->stream));
+    if (hy->kvx) cudaFree(hy->kvx);
+    hy->kvx = nullptr;
+    hy->kvx_elems = 0;
+    FB_CUDA(dev, cudaMalloc(&hy->kvx, kvx * 2));
+    hy->kvx_elems = kvx;
+  }
   for (auto& L : hy->layers)
     if ((rc = run_layer(m, L, batch, seq, commit))) return rc;
   // final norm and output head on the last position of every sequence
@@ -350,7 +379,7 @@ void fb200_hybrid_free(fb200_llama* m) {
                     L.own_rope ? L.rope_cos : nullptr, L.own_rope ? L.rope_sin : nullptr};
     for (void* b : bufs) if (b) cudaFree(b);
   }
-  void* bufs[] = {hy->proj, hy->zf, hy->hb, hy->zb, hy->qn, hy->kn, hy->vn, hy->gb, hy->kq, hy->o, hy->qa, hy->part};
+  void* bufs[] = {hy->proj, hy->zf, hy->hb, hy->zb, hy->qn, hy->kn, hy->vn, hy->gb, hy->kq, hy->o, hy->qa, hy->part, hy->kvx};
   for (void* b : bufs) if (b) cudaFree(b);
   delete hy;
   m->hybrid = nullptr;

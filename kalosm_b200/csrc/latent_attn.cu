@@ -38,9 +38,9 @@ __device__ __forceinline__ void unpack(const uint4& u, float (&f)[4], float) {
 __device__ __forceinline__ void store_elem(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ void store_elem(float* p, float v) { *p = v; }
 
-// T: element type of the expansion matrices and of the cache
+// T: element type of the expansion matrices and of the cache. CTAs 0 .. heads - 1 of a row take a query head each.
 template <typename T>
-__global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(const fb200_latent_args a) {
+__global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(const fb200_latent_args a, int heads) {
   constexpr int E = 16 / (int)sizeof(T);
   extern __shared__ __align__(16) float lsm[];  // query head [d + r], or partial sums [LQ_THREADS][E]
   __shared__ float red[LQ_THREADS / 32];
@@ -51,7 +51,7 @@ __global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(const fb200_la
   const float* yr = a.y + (size_t)row * a.ldy;
   const int half = a.r / 2;
   const float *cs = a.rope_cos + (size_t)pos * half, *sn = a.rope_sin + (size_t)pos * half;
-  if ((int)blockIdx.x == a.h) {  // the new position of a layer with a cache of its own
+  if ((int)blockIdx.x == heads) {  // the new position of a layer with a cache of its own
     const float* src = yr + a.off_dkv;
     T* dst = reinterpret_cast<T*>(a.cache) + ((size_t)b * a.cap + pos) * a.ldc;
     float ss = 0.f;
@@ -255,7 +255,7 @@ int latent_rows(fb200_device* dev, const fb200_latent_args& a) {
   constexpr int E = 16 / (int)sizeof(T);
   int rc;
   const size_t smem_q = (size_t)(((a.d + 3) & ~3) + LQ_THREADS * E) * 4;
-  if ((rc = fb200_launch(dev, latent_query_kernel<T>, dim3((unsigned)(a.h + (a.off_dkv >= 0 ? 1 : 0)), rows), dim3(LQ_THREADS), smem_q, true, a)))
+  if ((rc = fb200_launch(dev, latent_query_kernel<T>, dim3((unsigned)(a.h + (a.off_dkv >= 0 ? 1 : 0)), rows), dim3(LQ_THREADS), smem_q, true, a, a.h)))
     return rc;
   const int n = (a.ldc + 63) / 64;
   const dim3 grid((unsigned)a.nsplit, (unsigned)a.h, rows);
@@ -281,6 +281,14 @@ int fb200_latent_nsplit(const fb200_device* dev, int b, int h, int window, int c
   const int keys = window && window < cap ? window : cap;
   const int ns = std::min((keys + 31) / 32, 4 * dev->sm_count / std::max(1, b * h));
   return std::max(1, std::min(ns, 32));
+}
+
+int fb200_latent_append(fb200_device* dev, const fb200_latent_args& a) {
+  if (a.off_dkv < 0) return FB200_OK;
+  const dim3 grid(1, (unsigned)(a.b * a.s));
+  if (a.b * a.s > 65535) return fb200_fail(dev, FB200_ERR_CAPACITY, "latent attention: at most 65535 rows per pass");
+  if (a.cache_f32) return fb200_launch(dev, latent_query_kernel<float>, grid, dim3(LQ_THREADS), 16, true, a, 0);
+  return fb200_launch(dev, latent_query_kernel<__nv_bfloat16>, grid, dim3(LQ_THREADS), 16, true, a, 0);
 }
 
 int fb200_latent_rows(fb200_device* dev, const fb200_latent_args& a) {

@@ -58,9 +58,11 @@ struct fb200_latent_args {
   int z_bf16;
   float *qa, *part;  // [rows][h][rk + r]; [rows][h][nsplit][rk + 2]
   int nsplit;
-  // prompt pass with expanded keys and values (bf16): queries [rows][h][qd], expansions [keys][h d | h v]
-  __nv_bfloat16 *qx, *kvx;
+  __nv_bfloat16* kvx;  // prompt pass with expanded keys and values: [b * keys][h d | h v]
 };
 bool fb200_latent_covers(int d, int r, int v, int rk);
 int fb200_latent_nsplit(const fb200_device* dev, int b, int h, int window, int cap);
-int fb200_latent_rows(fb200_device* dev, const fb200_latent_args& a);  // any s: latent-space attention, row by row
+int fb200_latent_append(fb200_device* dev, const fb200_latent_args& a);  // the new positions' latents into the cache only
+int fb200_latent_rows(fb200_device* dev, const fb200_latent_args& a);    // any s: append, latent-space attention row by row
+bool fb200_latent_prefill_covers(int h, int d, int r, int v, int rk, float scale);
+int fb200_latent_prefill(fb200_device* dev, const fb200_latent_args& a, const fb200_qmatrix* w_ukv);  // after the append

@@ -5,10 +5,24 @@ token from the equations, with no chunking, no caches and no code shared with th
 
 A model is a dict {"width", "vocab", "eps", "layers": [...], "tensors": {name: array}} whose layers
 are the entries of a checkpoint's config.json ("type", "mixer", "mlp").
+
+`rnd` is the rounding of the operands of matrix products (identity by default): with a 16-bit rounding the
+functions show how far rounding alone moves the logits, which is what the tests measure a 16-bit run against.
 """
 from __future__ import annotations
 
 import numpy as np
+
+
+def exact(x):
+    return x
+
+
+def round_bf16(x):
+    """To the nearest bf16 (ties to even), in the type of x."""
+    u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
+    u = (u + 0x7FFF + ((u >> 16) & 1)) & np.uint32(0xFFFF0000)
+    return u.view(np.float32).astype(x.dtype)
 
 
 def rms_norm(x, w, eps):
@@ -59,8 +73,9 @@ def delta_rule(q, k, v, g, beta, state=None):
     return out, S
 
 
-def delta_mixer(h, mx, W, eps):
+def delta_mixer(h, mx, W, eps, rnd=exact):
     """The 'delta' mixer over a whole sequence: h [T, width] -> [T, width]. W(name) gives a tensor."""
+    h = rnd(h)
     T = h.shape[0]
     H, HK, D, V = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
     q, k, v = (silu(causal_conv(h @ W(n).T, W(n + ".conv"))) for n in ("q", "k", "v"))
@@ -71,7 +86,7 @@ def delta_mixer(h, mx, W, eps):
     g = np.exp(-np.exp(W("A_log")) * softplus(h @ W("a").T + W("dt_bias")))
     o, _ = delta_rule(q[:, group], k[:, group], v.reshape(T, H, V), g, beta)
     o = rms_norm(o, W("norm"), eps) * silu((h @ W("g").T).reshape(T, H, V))
-    return o.reshape(T, H * V) @ W("o").T
+    return rnd(o.reshape(T, H * V)) @ W("o").T
 
 
 def rotate_half(x, pos, base, dims):
@@ -85,13 +100,13 @@ def rotate_half(x, pos, base, dims):
     return np.concatenate([u * c - w * s, w * c + u * s, x[..., dims:]], axis=-1)
 
 
-def latent_rows(h, mx, W, eps):
+def latent_rows(h, mx, W, eps, rnd=exact):
     """What a latent-attention layer caches per token: (c [T, kv_rank], rotated key part [T, rot_dim])."""
     r = mx["kv_rank"]
     y = h @ W("dkv").T
     c = rms_norm(y[:, :r], W("dkv.norm"), eps)
     kr = rotate_half(y[:, r:], np.arange(h.shape[0]), mx["rot"]["base"], mx["rot"]["dims"])
-    return c, kr
+    return rnd(c), rnd(kr)
 
 
 def window_softmax(s, window):
@@ -104,30 +119,33 @@ def window_softmax(s, window):
     return p / p.sum(-1, keepdims=True)
 
 
-def latent_mixer(h, mx, W, eps, rows=None):
+def latent_mixer(h, mx, W, eps, rows=None, rnd=exact):
     """The 'latent_attention' mixer. `rows` = another layer's (c, rotated key part); returns
     ([T, width], the rows used)."""
+    h = rnd(h)
     T = h.shape[0]
     H, D, R, V = mx["heads"], mx["dim"], mx["rot_dim"], mx["vdim"]
-    c, kr = rows if rows is not None else latent_rows(h, mx, W, eps)
+    c, kr = rows if rows is not None else latent_rows(h, mx, W, eps, rnd)
     q = (h @ W("q").T).reshape(T, H, D + R)
     qr = rotate_half(q[..., D:], np.arange(T), mx["rot"]["base"], mx["rot"]["dims"])
-    k = (c @ W("uk").T).reshape(T, H, D)
-    v = (c @ W("uv").T).reshape(T, H, V)
+    q, qr = rnd(q), rnd(qr)
+    k = rnd(c @ W("uk").T).reshape(T, H, D)
+    v = rnd(c @ W("uv").T).reshape(T, H, V)
     gate = sigmoid(h @ W("g").T)
     out = np.zeros((T, H, V), dtype=h.dtype)
     window = (mx.get("mask") or {}).get("size", 0)
     for n in range(H):
         s = (q[:, n, :D] @ k[:, n].T + qr[:, n] @ kr.T) * mx["scale"]
-        out[:, n] = (window_softmax(s, window) @ v[:, n]) * gate[:, n, None]
-    return out.reshape(T, H * V) @ W("o").T, (c, kr)
+        out[:, n] = (rnd(window_softmax(s, window)) @ v[:, n]) * gate[:, n, None]
+    return rnd(out.reshape(T, H * V)) @ W("o").T, (c, kr)
 
 
-def dense_ff(h, W):
-    return (silu(h @ W("gate").T) * (h @ W("up").T)) @ W("down").T
+def dense_ff(h, W, rnd=exact):
+    h = rnd(h)
+    return rnd(silu(h @ W("gate").T) * (h @ W("up").T)) @ W("down").T
 
 
-def forward(model, tokens, dtype=np.float64, layers_out=None):
+def forward(model, tokens, dtype=np.float64, layers_out=None, rnd=exact):
     """Logits [T, vocab] of a whole sequence; `layers_out` collects the residual stream per layer."""
     t = model["tensors"]
 
@@ -142,14 +160,14 @@ def forward(model, tokens, dtype=np.float64, layers_out=None):
         def W(n, i=i):
             return get(f"l{i}.mix.{n}")
         if kind == "delta":
-            y = delta_mixer(h, mx, W, model["eps"])
+            y = delta_mixer(h, mx, W, model["eps"], rnd)
         elif kind == "latent_attention":
-            y, rows[i] = latent_mixer(h, mx, W, model["eps"], rows[mx["kv_from"]] if "kv_from" in mx else None)
+            y, rows[i] = latent_mixer(h, mx, W, model["eps"], rows[mx["kv_from"]] if "kv_from" in mx else None, rnd)
         else:
             raise ValueError(kind)
         if L.get("mlp"):
-            y = y + dense_ff(h, lambda n, i=i: get(f"l{i}.mlp.{n}"))
+            y = y + dense_ff(h, lambda n, i=i: get(f"l{i}.mlp.{n}"), rnd)
         x = x + y
         if layers_out is not None:
             layers_out.append(x.copy())
-    return rms_norm(x, get("final.norm"), model["eps"]) @ get("head").T
+    return rnd(rms_norm(x, get("final.norm"), model["eps"])) @ get("head").T
