@@ -248,14 +248,14 @@ attn_prefill_tc_kernel(const XArgs a, const __grid_constant__ CUtensorMap kmap, 
       }
       asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+      // before the last product can start, the one before it is seen complete: the final wait below then is for the
+      // phase in progress (a parity wait must be neither two phases early nor two late)
+      if (tile > 0 && tile == ntiles - 1) x_wait(bar_o, (uint32_t)((tile - 1) & 1), dead, a.status);
       mbar_arrive(bar_pfull);  // phase t
     }
 
     // ---- the last product, then normalise and store (nothing is stored after a wait has given up)
     if (ntiles > 0) {
-      // S of the last tile being complete says that O is complete up to the product two tiles back: the last two
-      // are waited for in turn (a parity wait must not start two phases behind)
-      if (ntiles > 1) x_wait(bar_o, (uint32_t)((ntiles - 2) & 1), dead, a.status);
       x_wait(bar_o, (uint32_t)((ntiles - 1) & 1), dead, a.status);
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     }

@@ -237,11 +237,11 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
       }
       asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+      // before the last product can start, the one before it is seen complete: the final wait below then is for the
+      // phase in progress (a parity wait must be neither two phases early nor two late)
+      if (t > 0 && t == ntiles - 1) x_wait(bar_o, (uint32_t)((t - 1) & 1), dead, a.status);
       mbar_arrive(bar_pfull);
     }
-    // S of the last tile being complete says that O is complete up to the product two tiles back: the last two are
-    // waited for in turn (a parity wait must not start two phases behind)
-    if (ntiles > 1) x_wait(bar_o, (uint32_t)((ntiles - 2) & 1), dead, a.status);
     x_wait(bar_o, (uint32_t)((ntiles - 1) & 1), dead, a.status);
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const bool store = row < a.s && !*dead;
