@@ -3,16 +3,19 @@
 //   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //
 // per head, with S [d, v] in 32-bit floats. The columns of S are independent, so a column (or a few) is
-// what a group of lanes owns for the whole sequence: it stays in registers, k and q of a token come from shared
-// memory, and both sums over d are formed in one pass from the state BEFORE the token,
+// what a group of lanes owns for the whole sequence: it stays in registers, k and q come from shared memory.
+// Both sums over d are formed in one pass from the state BEFORE the token,
 //   S^T k -> g (S^T k),   o = g (S^T q) + u (k . q),
-// which leaves one reduction over the lanes per token. Everything is f32, and a token is always processed the
-// same way, so a sequence gives the same state however it is cut.
+// and in a prompt four tokens share a pass: with a_i = S^T k_i, c_i = S^T q_i from the state before the four,
+// G_i = g_0 .. g_i and w_j = (g_(j+1) .. g_i) u_j,
+//   u_i = beta_i (v_i - G_i a_i - sum_(j<i) (k_j . k_i) w_j),   o_i = G_i c_i + sum_(j<=i) (k_j . q_i) w_j,
+//   S <- G_3 S + sum_j k_j w_j,
+// the same recurrence with one reduction over the lanes per four tokens. Everything is f32.
 //
 //  * delta_step_kernel: one new token per sequence. One CTA per (head, sequence): convolution, unit vectors,
 //    decay, state update, read-out, RMSNorm and gate. Bound: HBM on the state (read and written once).
-//  * prompts: delta_prep_kernel (convolution, SiLU, unit vectors, decay and write strength), delta_scan_kernel (the
-//    recurrence; bound: f32 FMA issue, packed two-wide), delta_out_kernel (RMSNorm, gate) and
+//  * prompts: delta_prep_kernel (convolution, SiLU, unit vectors, products of the four tokens' k and q, decay and
+//    write strength), delta_scan_kernel (the recurrence; bound: f32 FMA issue, packed two-wide), delta_out_kernel (RMSNorm, gate) and
 //    conv_ring_kernel (the convolution's memory).
 #include "mixers.cuh"
 #include "qgemv_common.cuh"
@@ -55,9 +58,8 @@ __device__ __forceinline__ float conv_in(const fb200_delta_args& a, int b, int c
   return a.ring[((size_t)b * a.taps + p % a.taps) * a.channels + c];
 }
 __device__ __forceinline__ float conv_silu(const fb200_delta_args& a, int b, int c, int t, int pos) {
-  const float* w = a.conv_w + (size_t)c * a.taps;
   float acc = 0.f;
-  for (int j = 0; j < a.taps; ++j) acc = fmaf(w[j], conv_in(a, b, c, t - (a.taps - 1) + j, pos), acc);
+  for (int j = 0; j < a.taps; ++j) acc = fmaf(a.conv_w[(size_t)j * a.channels + c], conv_in(a, b, c, t - (a.taps - 1) + j, pos), acc);
   return dr_silu(acc);
 }
 
@@ -209,61 +211,120 @@ __global__ void __launch_bounds__(ST_MAX_THREADS) delta_step_kernel(const fb200_
 }
 
 // ---- prompts ---------------------------------------------------------------------------------------------
-constexpr int PREP_T = 16, PREP_WARPS = 4, PREP_VCH = 128;
+constexpr int CH = 4;  // tokens per pass of the recurrence
+constexpr int PREP_WARPS = 4, PREP_VCH = 128;
+constexpr int PAIRS = 16;  // k_j . k_i (j < i): 6 values, then k_j . q_i (j <= i): 10 values, i-major
+// (j, i) of pair p, two bits each
+constexpr uint32_t PAIR_J = 0u | 0u << 2 | 1u << 4 | 0u << 6 | 1u << 8 | 2u << 10 | 0u << 12 | 0u << 14 | 1u << 16 | 0u << 18 | 1u << 20 |
+                            2u << 22 | 0u << 24 | 1u << 26 | 2u << 28 | 3u << 30;
+constexpr uint32_t PAIR_I = 1u | 2u << 2 | 2u << 4 | 3u << 6 | 3u << 8 | 3u << 10 | 0u << 12 | 1u << 14 | 1u << 16 | 2u << 18 | 2u << 20 |
+                            2u << 22 | 3u << 24 | 3u << 26 | 3u << 28 | 3u << 30;
 
-// A warp per (unit, 16 tokens): units 0 .. hk are the q and k vectors of a q/k head, then blocks of 128 v channels, then
+// convolution + SiLU of channel c for the CH tokens from t0 (zeros from token s on)
+__device__ __forceinline__ void conv_chunk(const fb200_delta_args& a, int b, int c, int t0, int pos, float (&out)[CH]) {
+#pragma unroll
+  for (int i = 0; i < CH; ++i) out[i] = 0.f;
+  if (t0 >= a.taps - 1 && t0 + CH <= a.s) {  // every input is a row of this pass
+    const float* y = a.y + ((size_t)b * a.s + t0 - (a.taps - 1)) * a.ldy + c;
+    for (int j = 0; j < a.taps; ++j) {
+      const float w = a.conv_w[(size_t)j * a.channels + c];
+#pragma unroll
+      for (int i = 0; i < CH; ++i) out[i] = fmaf(w, y[(size_t)(i + j) * a.ldy], out[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < CH; ++i) out[i] = dr_silu(out[i]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < CH; ++i)
+      if (t0 + i < a.s) out[i] = conv_silu(a, b, c, t0 + i, pos);
+  }
+}
+
+// Sums v[0..31] over the lanes of a warp; lane l returns the total of v[l].
+__device__ __forceinline__ float warp_sum32(float (&v)[32]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float send = up ? v[i] : v[i + o], keep = up ? v[i + o] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, o);
+    }
+  }
+  return v[0];
+}
+
+// A warp per (unit, CH tokens): units 0 .. hk are the q and k vectors of a q/k head, then blocks of 128 v channels, then
 // the decays and write strengths of all heads. NE = channels of a q/k head per lane.
 template <int NE>
 __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prep_kernel(const fb200_delta_args a) {
-  const int lane = threadIdx.x & 31, b = blockIdx.z, t0 = blockIdx.x * PREP_T, t1 = min(a.s, t0 + PREP_T);
+  const int lane = threadIdx.x & 31, b = blockIdx.z, t0 = blockIdx.x * CH, n = min(CH, a.s - t0);
   const int hv = a.h * a.v, vblocks = (hv + PREP_VCH - 1) / PREP_VCH;
   int unit = blockIdx.y * PREP_WARPS + (threadIdx.x >> 5);
   const int pos = *a.pos_dev;
   if (unit < a.hk) {
-    const float qscale = 1.0f / sqrtf((float)a.d);
-    for (int t = t0; t < t1; ++t) {
-      float q[NE], k[NE], skk = 0.f, sqq = 0.f, skq = 0.f;
+    float q[NE][CH], k[NE][CH], sum[32];
 #pragma unroll
-      for (int i = 0; i < NE; ++i) {
-        const int c = lane + 32 * i;
-        q[i] = k[i] = 0.f;
-        if (c < a.d) {
-          q[i] = conv_silu(a, b, unit * a.d + c, t, pos);
-          k[i] = conv_silu(a, b, (a.hk + unit) * a.d + c, t, pos);
-        }
-        skk = fmaf(k[i], k[i], skk);
-        sqq = fmaf(q[i], q[i], sqq);
-        skq = fmaf(k[i], q[i], skq);
+    for (int i = 0; i < 32; ++i) sum[i] = 0.f;
+#pragma unroll
+    for (int e = 0; e < NE; ++e) {
+      const int c = lane + 32 * e;
+#pragma unroll
+      for (int i = 0; i < CH; ++i) q[e][i] = k[e][i] = 0.f;
+      if (c < a.d) {
+        conv_chunk(a, b, unit * a.d + c, t0, pos, q[e]);
+        conv_chunk(a, b, (a.hk + unit) * a.d + c, t0, pos, k[e]);
       }
-      skk = warp_sum(skk);
-      sqq = warp_sum(sqq);
-      skq = warp_sum(skq);
-      const float ik = 1.0f / sqrtf(skk + UNIT_EPS), iq = (1.0f / sqrtf(sqq + UNIT_EPS)) * qscale;
-      const size_t row = ((size_t)b * a.s + t) * a.hk + unit;
 #pragma unroll
-      for (int i = 0; i < NE; ++i) {
-        const int c = lane + 32 * i;
+      for (int i = 0; i < CH; ++i) {
+        sum[i] = fmaf(k[e][i], k[e][i], sum[i]);
+        sum[4 + i] = fmaf(q[e][i], q[e][i], sum[4 + i]);
+      }
+#pragma unroll
+      for (int p = 0; p < PAIRS; ++p) {
+        const int j = (PAIR_J >> (2 * p)) & 3, i = (PAIR_I >> (2 * p)) & 3;
+        sum[8 + p] = fmaf(k[e][j], p < 6 ? k[e][i] : q[e][i], sum[8 + p]);
+      }
+    }
+    const float total = warp_sum32(sum);
+    const float inv = (1.0f / sqrtf(total + UNIT_EPS)) * (lane >= 4 ? 1.0f / sqrtf((float)a.d) : 1.0f);  // lanes 0..3: k, 4..7: q
+    const int p = lane - 8;
+    const float sj = __shfl_sync(0xFFFFFFFFu, inv, (PAIR_J >> (2 * (p & 15))) & 3);
+    const float si = __shfl_sync(0xFFFFFFFFu, inv, ((PAIR_I >> (2 * (p & 15))) & 3) + (p < 6 ? 0 : 4));
+    if (p >= 0 && p < PAIRS) a.kq[(((size_t)b * gridDim.x + blockIdx.x) * a.hk + unit) * PAIRS + p] = total * sj * si;
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {
+      const float ik = __shfl_sync(0xFFFFFFFFu, inv, i), iq = __shfl_sync(0xFFFFFFFFu, inv, 4 + i);
+      if (i >= n) continue;
+      const size_t row = ((size_t)b * a.s + t0 + i) * a.hk + unit;
+#pragma unroll
+      for (int e = 0; e < NE; ++e) {
+        const int c = lane + 32 * e;
         if (c < a.dp) {
-          a.qn[row * a.dp + c] = q[i] * iq;
-          a.kn[row * a.dp + c] = k[i] * ik;
+          a.qn[row * a.dp + c] = q[e][i] * iq;
+          a.kn[row * a.dp + c] = k[e][i] * ik;
         }
       }
-      if (lane == 0) a.kq[row] = skq * ik * iq;
     }
     return;
   }
   unit -= a.hk;
   if (unit < vblocks) {
-    for (int t = t0; t < t1; ++t)
 #pragma unroll
-      for (int i = 0; i < PREP_VCH / 32; ++i) {
-        const int c = unit * PREP_VCH + lane + 32 * i;
-        if (c < hv) a.vn[((size_t)b * a.s + t) * hv + c] = conv_silu(a, b, a.off_v + c, t, pos);
-      }
+    for (int e = 0; e < PREP_VCH / 32; ++e) {
+      const int c = unit * PREP_VCH + lane + 32 * e;
+      if (c >= hv) continue;
+      float v[CH];
+      conv_chunk(a, b, a.off_v + c, t0, pos, v);
+#pragma unroll
+      for (int i = 0; i < CH; ++i)
+        if (i < n) a.vn[((size_t)b * a.s + t0 + i) * hv + c] = v[i];
+    }
     return;
   }
   if (unit > vblocks) return;
-  for (int i = lane; i < (t1 - t0) * a.h; i += 32) {
+  for (int i = lane; i < n * a.h; i += 32) {
     const int t = t0 + i / a.h, h = i % a.h;
     const size_t row = (size_t)b * a.s + t;
     const float* yr = a.y + row * a.ldy;
@@ -272,38 +333,50 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prep_kernel(const fb200
   }
 }
 
-constexpr int SC_WARPS = 4;
+constexpr int SC_WARPS = 8;
 
+// TOK tokens per shared-memory stage (a multiple of CH)
 template <int EPT, int LPC, int TOK>
 __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_delta_args a) {
-  constexpr int DP = EPT * LPC, COLS = SC_WARPS * 32 / LPC, THREADS = SC_WARPS * 32;
-  constexpr int STAGE = TOK * (2 * DP + COLS + 4);  // floats: k, q [TOK][DP], v [TOK][COLS], (g, beta, kq, -) [TOK][4]
+  constexpr int DP = EPT * LPC, COLS = SC_WARPS * 32 / LPC, THREADS = SC_WARPS * 32, NC = TOK / CH;
+  // floats of a stage: k, q [TOK][DP], v [COLS][TOK], pairs [NC][PAIRS], g [TOK], beta [TOK]
+  constexpr int OV = 2 * TOK * DP, OP = OV + COLS * TOK, OG = OP + NC * PAIRS, STAGE = OG + 2 * TOK;
+  constexpr bool KEEP = EPT <= 16;  // k of the four tokens stays in registers for the update
   extern __shared__ __align__(16) float dsm[];
-  const int tid = threadIdx.x, h = blockIdx.y, b = blockIdx.z, group = a.h / a.hk, hk = h / group, hv = a.h * a.v;
+  const int tid = threadIdx.x, lane = tid & 31, h = blockIdx.y, b = blockIdx.z, group = a.h / a.hk, hk = h / group, hv = a.h * a.v;
   const int p = tid % LPC, cl = tid / LPC, c = blockIdx.x * COLS + cl;
-  const int pos = *a.pos_dev;
+  const int pos = *a.pos_dev, nchunks = (a.s + CH - 1) / CH;
   const size_t row0 = (size_t)b * a.s;
-  auto cp4 = [](uint32_t dst, const void* src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory"); };
-  auto cp16 = [](uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); };
+  auto cp4 = [](const float* dst, const float* src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory"); };
+  auto cp16 = [](const float* dst, const float* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory"); };
   auto fetch = [&](int t0, int stage) {
     float* sb = dsm + stage * STAGE;
     const int n = min(TOK, a.s - t0);
-    for (int i = tid; i < n * (DP / 4); i += THREADS) {
+    for (int i = tid; i < TOK * (DP / 4); i += THREADS) {
       const int t = i / (DP / 4), e = (i % (DP / 4)) * 4;
-      const size_t src = ((row0 + t0 + t) * a.hk + hk) * (size_t)DP + e;
-      cp16(smem_u32(sb + t * DP + e), a.kn + src);
-      cp16(smem_u32(sb + (TOK + t) * DP + e), a.qn + src);
+      if (t < n) {
+        const size_t src = ((row0 + t0 + t) * a.hk + hk) * (size_t)DP + e;
+        cp16(sb + t * DP + e, a.kn + src);
+        cp16(sb + (TOK + t) * DP + e, a.qn + src);
+      } else {  // beyond the last token: k = q = v = 0, g = 1, beta = 0 change nothing
+        *reinterpret_cast<float4*>(sb + t * DP + e) = make_float4(0.f, 0.f, 0.f, 0.f);
+        *reinterpret_cast<float4*>(sb + (TOK + t) * DP + e) = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
     }
-    float* vb = sb + 2 * TOK * DP;
-    for (int i = tid; i < n * COLS; i += THREADS) {
+    for (int i = tid; i < TOK * COLS; i += THREADS) {
       const int t = i / COLS, cc = i % COLS, col = blockIdx.x * COLS + cc;
-      if (col < a.v) cp4(smem_u32(vb + i), a.vn + (row0 + t0 + t) * hv + h * a.v + col);
+      if (t < n && col < a.v) cp4(sb + OV + cc * TOK + t, a.vn + (row0 + t0 + t) * hv + h * a.v + col);
+      else sb[OV + cc * TOK + t] = 0.f;
     }
-    float* gs = vb + TOK * COLS;
-    for (int i = tid; i < n * 3; i += THREADS) {
-      const int t = i / 3, f = i % 3;
-      const size_t r = row0 + t0 + t;
-      cp4(smem_u32(gs + t * 4 + f), f < 2 ? a.gb + (r * a.h + h) * 2 + f : a.kq + r * a.hk + hk);
+    for (int i = tid; i < NC * (PAIRS / 4); i += THREADS) {
+      const int ch = t0 / CH + i / (PAIRS / 4), e = (i % (PAIRS / 4)) * 4;
+      if (ch < nchunks) cp16(sb + OP + (i / (PAIRS / 4)) * PAIRS + e, a.kq + (((size_t)b * nchunks + ch) * a.hk + hk) * PAIRS + e);
+      else *reinterpret_cast<float4*>(sb + OP + (i / (PAIRS / 4)) * PAIRS + e) = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    for (int i = tid; i < 2 * TOK; i += THREADS) {
+      const int t = i % TOK, f = i / TOK;
+      if (t < n) cp4(sb + OG + i, a.gb + ((row0 + t0 + t) * a.h + h) * 2 + f);
+      else sb[OG + i] = f ? 0.f : 1.f;
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -316,29 +389,111 @@ __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_d
 #pragma unroll
     for (int i = 0; i < EPT / 2; ++i) s[i] = make_float2(0.f, 0.f);
   }
-  const int chunks = (a.s + TOK - 1) / TOK;
-  for (int ch = 0; ch < chunks; ++ch) {
-    if (ch + 1 < chunks) {
-      fetch((ch + 1) * TOK, (ch + 1) & 1);
+  const int stages = (a.s + TOK - 1) / TOK;
+  for (int st = 0; st < stages; ++st) {
+    if (st + 1 < stages) {
+      fetch((st + 1) * TOK, (st + 1) & 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
-    const float* sb = dsm + (ch & 1) * STAGE;
-    const float *vb = sb + 2 * TOK * DP, *gs = vb + TOK * COLS;
-    const int n = min(TOK, a.s - ch * TOK);
-    float* orow = a.o + (row0 + ch * TOK) * hv + h * a.v + c;
-    for (int t = 0; t < n; ++t) {
-      const float *ks = sb + t * DP, *qs = sb + (TOK + t) * DP;
-      const float4 gk = *reinterpret_cast<const float4*>(gs + t * 4);
-      float dk, dq;
-      column_dots<EPT, LPC>(s, ks, qs, p, dk, dq);
-      const float u = gk.y * (vb[t * COLS + cl] - gk.x * dk);
-      column_update<EPT, LPC>(s, ks, p, gk.x, u);
-      if (p == 0 && c < a.v) orow[(size_t)t * hv] = fmaf(gk.x, dq, u * gk.z);
+    const float* sb = dsm + (st & 1) * STAGE;
+#pragma unroll 1
+    for (int ch = 0; ch < NC; ++ch) {
+      const int t0 = st * TOK + ch * CH;
+      if (t0 >= a.s) break;
+      const float *kb = sb + ch * CH * DP, *qb = sb + (TOK + ch * CH) * DP;
+      // ---- a_i = S^T k_i, c_i = S^T q_i over this lane's elements
+      float2 kf[KEEP ? CH : 1][EPT / 2];
+      float val[2 * CH];
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        float2 k0 = make_float2(0.f, 0.f), k1 = k0, q0 = k0, q1 = k0;
+#pragma unroll
+        for (int e = 0; e < EPT / 4; ++e) {
+          const float4 k = *reinterpret_cast<const float4*>(kb + i * DP + 4 * (e * LPC + p));
+          const float4 q = *reinterpret_cast<const float4*>(qb + i * DP + 4 * (e * LPC + p));
+          k0 = fma2(s[2 * e], make_float2(k.x, k.y), k0);
+          k1 = fma2(s[2 * e + 1], make_float2(k.z, k.w), k1);
+          q0 = fma2(s[2 * e], make_float2(q.x, q.y), q0);
+          q1 = fma2(s[2 * e + 1], make_float2(q.z, q.w), q1);
+          if (KEEP) {
+            kf[KEEP ? i : 0][2 * e] = make_float2(k.x, k.y);
+            kf[KEEP ? i : 0][2 * e + 1] = make_float2(k.z, k.w);
+          }
+        }
+        val[i] = (k0.x + k0.y) + (k1.x + k1.y);
+        val[CH + i] = (q0.x + q0.y) + (q1.x + q1.y);
+      }
+      // ---- totals over the LPC lanes: eight values over eight lanes by halving, then the rest of the lanes
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int i = 0; i < o; ++i) {
+          const float send = up ? val[i] : val[i + o], keep = up ? val[i + o] : val[i];
+          val[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, o);
+        }
+      }
+      float mine = val[0];  // lane l: value l % 8
+#pragma unroll
+      for (int o = 8; o < LPC; o <<= 1) mine += __shfl_xor_sync(0xFFFFFFFFu, mine, o);
+      float av[CH], cv[CH];
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        av[i] = __shfl_sync(0xFFFFFFFFu, mine, (lane & ~7) | i);
+        cv[i] = __shfl_sync(0xFFFFFFFFu, mine, (lane & ~7) | (CH + i));
+      }
+      // ---- the four tokens in order
+      float pr[PAIRS];
+#pragma unroll
+      for (int i = 0; i < PAIRS / 4; ++i) {
+        const float4 x = *reinterpret_cast<const float4*>(sb + OP + ch * PAIRS + 4 * i);
+        pr[4 * i] = x.x; pr[4 * i + 1] = x.y; pr[4 * i + 2] = x.z; pr[4 * i + 3] = x.w;
+      }
+      const float4 g4 = *reinterpret_cast<const float4*>(sb + OG + ch * CH), b4 = *reinterpret_cast<const float4*>(sb + OG + TOK + ch * CH);
+      const float4 v4 = *reinterpret_cast<const float4*>(sb + OV + cl * TOK + ch * CH);
+      const float gi[CH] = {g4.x, g4.y, g4.z, g4.w}, bi[CH] = {b4.x, b4.y, b4.z, b4.w}, vi[CH] = {v4.x, v4.y, v4.z, v4.w};
+      float w[CH], out = 0.f, G = 1.f;
+      int pk = 0, pq = 6;
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        G *= gi[i];
+        float uk = G * av[i], o = G * cv[i];
+#pragma unroll
+        for (int j = 0; j < CH; ++j)
+          if (j < i) {
+            w[j] *= gi[i];
+            uk = fmaf(pr[pk++], w[j], uk);
+            o = fmaf(pr[pq++], w[j], o);
+          }
+        w[i] = bi[i] * (vi[i] - uk);
+        o = fmaf(pr[pq++], w[i], o);
+        if (p == i) out = o;
+      }
+      if (p < CH && c < a.v && t0 + p < a.s) a.o[(row0 + t0 + p) * hv + h * a.v + c] = out;
+      // ---- S <- G S + sum_j k_j w_j
+      const float2 G2 = make_float2(G, G);
+#pragma unroll
+      for (int e = 0; e < EPT / 2; ++e) s[e] = mul2(s[e], G2);
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        const float2 w2 = make_float2(w[i], w[i]);
+#pragma unroll
+        for (int e = 0; e < EPT / 4; ++e) {
+          if (KEEP) {
+            s[2 * e] = fma2(kf[KEEP ? i : 0][2 * e], w2, s[2 * e]);
+            s[2 * e + 1] = fma2(kf[KEEP ? i : 0][2 * e + 1], w2, s[2 * e + 1]);
+          } else {
+            const float4 k = *reinterpret_cast<const float4*>(kb + i * DP + 4 * (e * LPC + p));
+            s[2 * e] = fma2(make_float2(k.x, k.y), w2, s[2 * e]);
+            s[2 * e + 1] = fma2(make_float2(k.z, k.w), w2, s[2 * e + 1]);
+          }
+        }
+      }
     }
-    __syncthreads();  // the stage is free before the chunk after next lands in it
+    __syncthreads();  // the stage is free before the one after next lands in it
   }
   if (c < a.v) store_column<EPT, LPC>(col, p, s);
 }
@@ -384,7 +539,7 @@ int launch_step(fb200_device* dev, const fb200_delta_args& a) {
 template <int EPT, int LPC, int TOK>
 int launch_scan(fb200_device* dev, const fb200_delta_args& a) {
   constexpr int DP = EPT * LPC, COLS = SC_WARPS * 32 / LPC;
-  constexpr size_t smem = (size_t)2 * TOK * (2 * DP + COLS + 4) * 4;
+  constexpr size_t smem = (size_t)2 * (2 * TOK * DP + COLS * TOK + TOK / CH * PAIRS + 2 * TOK) * 4;
   static bool configured[64] = {false};
   if (!configured[dev->ordinal & 63]) {
     FB_CUDA(dev, cudaFuncSetAttribute(delta_scan_kernel<EPT, LPC, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -398,7 +553,7 @@ int launch_scan(fb200_device* dev, const fb200_delta_args& a) {
 template <int NE>
 int launch_prep(fb200_device* dev, const fb200_delta_args& a) {
   const int units = a.hk + (a.h * a.v + PREP_VCH - 1) / PREP_VCH + 1;
-  delta_prep_kernel<NE><<<dim3((unsigned)((a.s + PREP_T - 1) / PREP_T), (unsigned)((units + PREP_WARPS - 1) / PREP_WARPS), (unsigned)a.b),
+  delta_prep_kernel<NE><<<dim3((unsigned)((a.s + CH - 1) / CH), (unsigned)((units + PREP_WARPS - 1) / PREP_WARPS), (unsigned)a.b),
                           PREP_WARPS * 32, 0, dev->stream>>>(a);
   FB_LAUNCH_CHECK(dev);
   return FB200_OK;
@@ -437,11 +592,11 @@ int fb200_delta_prompt(fb200_device* dev, const fb200_delta_args& a) {
   }
   if (rc) return rc;
   switch (a.dp) {
-    case 32: rc = launch_scan<8, 4, 16>(dev, a); break;
-    case 64: rc = launch_scan<16, 4, 16>(dev, a); break;
-    case 128: rc = launch_scan<32, 4, 16>(dev, a); break;
+    case 32: rc = launch_scan<4, 8, 16>(dev, a); break;
+    case 64: rc = launch_scan<8, 8, 16>(dev, a); break;
+    case 128: rc = launch_scan<16, 8, 16>(dev, a); break;
     case 256: rc = launch_scan<32, 8, 16>(dev, a); break;
-    case 512: rc = launch_scan<32, 16, 4>(dev, a); break;
+    case 512: rc = launch_scan<32, 16, 8>(dev, a); break;
     default: rc = launch_scan<32, 32, 4>(dev, a); break;
   }
   if (rc) return rc;

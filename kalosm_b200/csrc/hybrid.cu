@@ -295,7 +295,7 @@ int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows) {
   struct { void** p; size_t bytes; } bufs[] = {
       {(void**)&m->x, rows * E * 4}, {(void**)&m->xn, rows * E * 4}, {(void**)&hy->proj, rows * hy->ldy * 4}, {(void**)&hy->zf, rows * hy->ldz * 4},
       {(void**)&hy->hb, rows * up_to(E, 64) * 2}, {(void**)&hy->zb, rows * hy->ldz * 2}, {(void**)&hy->qn, rows * qk * 4},
-      {(void**)&hy->kn, rows * qk * 4}, {(void**)&hy->vn, rows * hv * 4}, {(void**)&hy->gb, rows * heads * 8}, {(void**)&hy->kq, rows * kvh * 4},
+      {(void**)&hy->kn, rows * qk * 4}, {(void**)&hy->vn, rows * hv * 4}, {(void**)&hy->gb, rows * heads * 8}, {(void**)&hy->kq, (rows + 3 * (size_t)m->cfg.max_batch) / 4 * kvh * 64 + 64},
       {(void**)&hy->o, rows * hv * 4}, {(void**)&hy->qa, qa * 4}, {(void**)&hy->part, part * 4}};
   for (auto& b : bufs) {
     if (*b.p) { cudaFree(*b.p); *b.p = nullptr; }
@@ -432,6 +432,7 @@ int fb200_hybrid_set_tensor(fb200_llama* m, int layer, int which, uint32_t type,
   const uint64_t qk = (uint64_t)c.kv_heads * c.dim, hv = (uint64_t)c.heads * c.vdim;
   fb200_qmatrix* w = L.w_in;
   float* vd = nullptr;
+  bool conv = false;
   uint64_t row0 = 0, col0 = 0;
   ek = E;
   switch (which) {
@@ -449,9 +450,9 @@ int fb200_hybrid_set_tensor(fb200_llama* m, int layer, int which, uint32_t type,
     case FB200_T_MIX_DKV: en = (uint64_t)c.kv_rank + c.rot_dim; row0 = L.off_dkv; break;
     case FB200_T_MIX_UK: en = (uint64_t)c.heads * c.dim; ek = c.kv_rank; w = L.w_ukv; break;
     case FB200_T_MIX_UV: en = hv; ek = c.kv_rank; w = L.w_ukv; row0 = (uint64_t)c.heads * c.dim; break;
-    case FB200_T_MIX_Q_CONV: en = qk; ek = c.conv; vd = L.conv_w; break;
-    case FB200_T_MIX_K_CONV: en = qk; ek = c.conv; vd = L.conv_w + qk * c.conv; break;
-    case FB200_T_MIX_V_CONV: en = hv; ek = c.conv; vd = L.conv_w + 2 * qk * c.conv; break;
+    case FB200_T_MIX_Q_CONV: en = qk; ek = c.conv; conv = true; break;
+    case FB200_T_MIX_K_CONV: en = qk; ek = c.conv; col0 = qk; conv = true; break;
+    case FB200_T_MIX_V_CONV: en = hv; ek = c.conv; col0 = 2 * qk; conv = true; break;
     case FB200_T_MIX_A_LOG: en = c.heads; ek = 1; vd = L.a_log; break;
     case FB200_T_MIX_DT_BIAS: en = c.heads; ek = 1; vd = L.dt_bias; break;
     case FB200_T_MIX_OUT_NORM: en = c.vdim; ek = 1; vd = L.out_norm; break;
@@ -459,6 +460,16 @@ int fb200_hybrid_set_tensor(fb200_llama* m, int layer, int which, uint32_t type,
     default: return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "tensor id %d", which);
   }
   if ((rc = shape_ok())) return rc;
+  if (conv) {  // convolution taps [channels, taps] -> columns col0 .. of [taps][channels]
+    std::vector<float> f;
+    if ((rc = to_f32(dev, type, src, n * k, f))) return rc;
+    std::vector<float> t(f.size());
+    for (uint64_t i = 0; i < n; ++i)
+      for (uint64_t j = 0; j < k; ++j) t[j * n + i] = f[i * k + j];
+    FB_CUDA(dev, cudaMemcpy2D(L.conv_w + col0, (size_t)L.channels * 4, t.data(), n * 4, n * 4, k, cudaMemcpyHostToDevice));
+    L.have |= 1u << which;
+    return FB200_OK;
+  }
   rc = vd ? vec(vd) : put_block(dev, w, row0, col0, type, n, k, src);
   if (!rc) L.have |= 1u << which;
   return rc;

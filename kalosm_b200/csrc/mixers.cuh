@@ -15,7 +15,7 @@ struct fb200_delta_args {
   const float* y;
   size_t ldy;
   int off_v, off_g, off_b, off_a;
-  const float *conv_w, *a_log, *dt_bias, *out_norm;
+  const float *conv_w, *a_log, *dt_bias, *out_norm;  // conv_w [taps][channels]
   float eps;
   float *state, *ring;
   int b, s, h, hk, d, v, dp, taps, channels;
@@ -25,7 +25,7 @@ struct fb200_delta_args {
   int z_bf16;
   int commit;  // 0: a dry run of a decode step, the state stays as it is
   // prompt pass scratch: unit q and k [rows][hk][dp], v [rows][h v], (decay, write strength) [rows][h][2],
-  // k . q [rows][hk], read-out [rows][h v]
+  // products of four tokens' k and q [b][ceil(s / 4)][hk][16], read-out [rows][h v]
   float *qn, *kn, *vn, *gb, *kq, *o;
 };
 int fb200_delta_dp(int d);                                         // padded head size, 0 when d is not covered
