@@ -600,6 +600,208 @@ def run_tensor_parallel(args):
         sys.exit(3)
 
 
+# ---- --hybrid: a Koludra decoder (delta rule + latent attention, dense bf16) beside a Llama decoder of equal size --------
+
+def hybrid_layers(width, ffn, window, n_layer):
+    """Layer list with the sizes of real layers: 128-wide heads, 512-wide latents, 3 delta rules to 2 attentions."""
+    h, mlp = width // 128, {"kind": "dense", "ff": ffn}
+    d = {"type": "delta", "mixer": dict(heads=h, kv_heads=h // 2, dim=128, vdim=128, conv=4), "mlp": mlp}
+    d2 = {"type": "delta_2", "mixer": dict(heads=h, kv_heads=h, dim=128, vdim=128, conv=4), "mlp": mlp}
+    a = {"type": "latent_attention", "mlp": mlp,
+         "mixer": dict(heads=h, dim=128, rot_dim=64, vdim=128, kv_rank=512, mask={"size": window}, rot={"base": 500000.0, "dims": 64},
+                       scale=192 ** -0.5)}
+    shared = dict(a, mixer=dict(a["mixer"], kv_from=1))
+    return [(d, a, d2, d, shared)[i % 5] for i in range(n_layer)]
+
+
+def build_hybrid_model(dev, torch, width, ffn, window, n_layer, vocab, ctx, seed=0):
+    """Random weights made on the GPU, handed over as bf16 bytes. Returns (model, layers, parameters of the streamed matrices)."""
+    import kalosm_b200 as kb
+    from kalosm_b200 import koludra
+    layers = hybrid_layers(width, ffn, window, n_layer)
+    cfg = {"architecture": "Koludra", "layers": layers, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    params = [0]
+
+    def shape_of(name):
+        if name in ("embed", "head"):
+            return (vocab, width)
+        if name == "final.norm" or name.endswith("norm1"):
+            return (width,)
+        i, part, rest = name.split(".", 2)
+        L = layers[int(i[1:])]
+        mx, ff = L["mixer"], L["mlp"]["ff"]
+        H, hv = mx["heads"], mx["heads"] * mx["vdim"]
+        if part == "mlp":
+            return (width, ff) if rest == "down" else (ff, width)
+        if L["type"].startswith("delta"):
+            qk = mx["kv_heads"] * mx["dim"]
+            rows = {"q": qk, "k": qk, "v": hv, "g": hv, "b": H, "a": H}
+            if rest.endswith(".conv"):
+                return (rows[rest[0]], mx["conv"])
+            return {"o": (width, hv), "A_log": (H,), "dt_bias": (H,), "norm": (mx["vdim"],)}.get(rest) or (rows[rest], width)
+        r = mx["kv_rank"]
+        return {"q": (H * (mx["dim"] + mx["rot_dim"]), width), "g": (H, width), "o": (width, hv), "uk": (H * mx["dim"], r), "uv": (hv, r),
+                "dkv": (r + mx["rot_dim"], width), "dkv.norm": (r,)}[rest]
+
+    def tensor(name):
+        shape = shape_of(name)
+        w = torch.randn(shape, generator=g, device="cuda", dtype=torch.float32)
+        if len(shape) == 1:
+            w = 1.0 + 0.1 * w if "norm" in name else 0.5 * w - 1.0
+        else:
+            w *= 0.3 if name.endswith(".conv") else shape[1] ** -0.5
+            if name != "embed" and not name.endswith(".conv"):
+                params[0] += shape[0] * shape[1]
+        return kb.BF16, shape, w.to(torch.bfloat16).view(torch.int16).cpu().numpy()
+    return koludra.build(dev, cfg, tensor, ctx, 1), layers, params[0]
+
+
+def device_table(torch, fn, reps):
+    """Device time per kernel of `reps` calls of fn (CUPTI): {short kernel name: (us per call, launches per call)}."""
+    from torch.profiler import ProfilerActivity, profile
+    with profile(activities=[ProfilerActivity.CUDA]) as prof:
+        for _ in range(reps):
+            fn()
+        torch.cuda.synchronize()
+    out = {}
+    for ev in prof.key_averages():
+        t = getattr(ev, "device_time_total", None)
+        t = ev.cuda_time_total if t is None else t
+        name = ev.key.replace("void ", "").replace("(anonymous namespace)::", "").split("(")[0].split("<")[0]
+        if t > 0 and "mem" not in name.lower():
+            us, n = out.get(name, (0.0, 0.0))
+            out[name] = (us + t / reps, n + ev.count / reps)
+    return out
+
+
+def hybrid_work(layers, width, vocab, rows, ctx, n_sm):
+    """Roofline work of one pass of `rows` new positions behind `ctx` cached ones: {kernel: (kind, amount, peak)}; kind "hbm"
+    in bytes, "tensor" and "f32" in flops."""
+    peak = {"hbm": peaks()[0] * 1e9, "tensor": tensor_peak()[0] * 1e12, "f32": n_sm * 128 * 2 * 1.965e9}  # f32: nominal FMA rate
+    w = {}
+
+    def add(name, kind, amount):
+        w[name] = (kind, w.get(name, (kind, 0.0))[1] + amount)
+    for L in layers:
+        mx, ff = L["mixer"], L["mlp"]["ff"]
+        H, V = mx["heads"], mx["vdim"]
+        delta = L["type"].startswith("delta")
+        n_in = 2 * ff + (2 * mx["kv_heads"] * mx["dim"] + 2 * H * V + 2 * H if delta else
+                         H * (mx["dim"] + mx["rot_dim"]) + H + (0 if "kv_from" in mx else mx["kv_rank"] + mx["rot_dim"]))
+        mats = n_in * width + width * (H * V + ff)
+        add(*(("dense_gemv_kernel", "hbm", 2.0 * mats) if rows == 1 else ("dense_tc_kernel", "tensor", 2.0 * mats * rows)))
+        if delta and rows == 1:
+            add("delta_step_kernel", "hbm", 8.0 * H * V * mx["dim"])
+        elif delta:
+            add("delta_prep_kernel", "hbm", 8.0 * rows * (2 * mx["kv_heads"] * mx["dim"] + H * V))
+            add("delta_scan_kernel", "f32", 6.0 * rows * H * V * mx["dim"])  # two sums over d and one update
+            add("delta_out_kernel", "hbm", 10.0 * rows * H * V)
+        elif rows == 1:
+            add("latent_query_kernel", "hbm", 2.0 * H * mx["dim"] * mx["kv_rank"])
+            add("latent_attn_kernel", "hbm", 2.0 * min(mx["mask"]["size"], ctx + 1) * (mx["kv_rank"] + mx["rot_dim"]))
+            add("latent_out_kernel", "hbm", 2.0 * H * V * mx["kv_rank"])
+        else:
+            win = mx["mask"]["size"]
+            add("dense_tc_kernel", "tensor", 2.0 * (rows + min(win - 1, ctx)) * H * (mx["dim"] + V) * mx["kv_rank"])
+            pairs = float(sum(min(win, ctx + i + 1) for i in range(rows)))
+            add("latent_prefill_kernel", "tensor", 2.0 * pairs * H * (mx["dim"] + mx["rot_dim"] + V))
+    if rows == 1:
+        add("dense_gemv_kernel", "hbm", 2.0 * vocab * width)
+    return {n: (k, a, peak[k]) for n, (k, a) in w.items()}
+
+
+def llama_work(cfg, rows, ctx):
+    tf = tensor_peak()[0] * 1e12
+    mats = sum(n * k for name, l, _t, (n, k) in tensor_plan(cfg) if l >= 0)
+    pairs = rows * (rows + 1) / 2 + rows * ctx
+    return {"qgemm_tc_kernel": ("tensor", 2.0 * mats * rows, tf),
+            "attn_prefill_tc_kernel": ("tensor", 4.0 * pairs * cfg["n_head"] * cfg["head_dim"] * cfg["n_layer"], tf)}
+
+
+def kernel_rows(table, work):
+    rows = []
+    for name, (us, n) in sorted(table.items(), key=lambda kv: -kv[1][0]):
+        r = {"kernel": name, "us": round(us, 2), "launches": round(n, 2)}
+        if name in work:
+            kind, amount, peak = work[name]
+            r.update(bound=kind, frac=round(amount / (us * 1e-6) / peak, 4))
+        rows.append(r)
+    return rows
+
+
+def run_hybrid(args):
+    """Prefill and decode of a Koludra decoder with layers of real-model sizes (random bf16 weights) beside a Llama decoder
+    (Q4_K / Q6_K weights, the closest existing model) of the same width, feed-forward, layers and vocabulary; one JSON line per size
+    with the device time and roofline fraction of every kernel. Kernels of a decode step overlap their predecessors' tails (programmatic
+    dependent launch), so their times in the table contain waiting; FB200_PDL=0 gives stand-alone times. Not the bench line."""
+    import torch
+    import kalosm_b200 as kb
+    torch.cuda.set_device(0)
+    stream = torch.cuda.Stream()
+    torch.cuda.set_stream(stream)
+    n_sm = torch.cuda.get_device_properties(0).multi_processor_count
+
+    def timed(fn, reps):
+        fn()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(stream)
+        for _ in range(reps):
+            fn()
+        e1.record(stream)
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / reps
+
+    vocab, steps, lens = 32768, 64, (512, 2048, 8192)
+    for width, ffn, window, n_layer in ((2048, 8192, 1024, 10), (4096, 14336, 2048, 10)):
+        if args.hybrid_only not in (0, width):
+            continue
+        ctx = max(lens) + 4 * steps + 64
+        line = {"bench": "hybrid", "width": width, "ffn": ffn, "window": window, "layers": n_layer, "vocab": vocab,
+                "data": "synthetic (random weights, random token ids)", "peaks": {"hbm_gbs": peaks()[0], "bf16_tflops": tensor_peak()[0]},
+                "pdl": os.environ.get("FB200_PDL", "1"), "l2": "every pass streams more weights than the L2 holds"}
+        for kind in ("koludra",) if args.no_llama else ("koludra", "llama"):
+            dev = kb.Device(0, stream.cuda_stream)
+            layers = None
+            if kind == "koludra":
+                m, layers, params = build_hybrid_model(dev, torch, width, ffn, window, n_layer, vocab, ctx)
+                wbytes = 2.0 * params
+            else:
+                cfg = dict(n_layer=n_layer, hidden=width, ffn=ffn, n_head=width // 128, n_kv_head=width // 512, head_dim=128, vocab=vocab)
+                m = build_gpu_model(dev, torch, cfg, 1, ctx, seed=1)
+                wbytes = float(weight_bytes_per_step(cfg))
+            sampler = ClockSampler(0)
+            sampler.start()
+            time.sleep(0.3)
+            t0 = time.time()
+            out = {"weight_bytes_per_step": wbytes, "prefill": [], "decode": []}
+            last = np.array([1], dtype=np.uint32)
+            for n in lens:
+                prompt = np.random.default_rng(n).integers(0, vocab, size=(1, n), dtype=np.uint32)
+
+                def prefill():
+                    m.reset()
+                    m.forward(prompt, want_logits=False)
+                ms = timed(prefill, 3 if n > 4096 else 5)
+                table = device_table(torch, prefill, 2)
+                work = hybrid_work(layers, width, vocab, n, 0, n_sm) if layers else llama_work(cfg, n, 0)
+                out["prefill"].append({"tokens": n, "ms": ms, "tok_s": n / ms * 1e3, "kernels": kernel_rows(table, work)})
+                m.generate_greedy(last, 8)
+                ms = timed(lambda: m.generate_greedy(last, steps), 1) / steps
+                kv = 0 if layers else 4.0 * n_layer * (width // 512) * 128 * (n + 8 + steps * 1.5)
+                table = {k: (us / 16, c / 16) for k, (us, c) in device_table(torch, lambda: m.generate_greedy(last, 16), 1).items()}
+                work = hybrid_work(layers, width, vocab, 1, n, n_sm) if layers else {"fused_step_kernel": ("hbm", wbytes + kv, peaks()[0] * 1e9)}
+                out["decode"].append({"context": n, "ms": ms, "tok_s": 1e3 / ms, "hbm_frac": (wbytes + kv) / (ms * 1e-3) / (peaks()[0] * 1e9),
+                                      "kernels": kernel_rows(table, work)})
+            out["clocks"] = sampler.stop(t0, time.time())
+            out["device_status"] = dev.status()
+            line[kind] = out
+            m.free()
+            dev.close()
+        print(json.dumps(line), flush=True)
+
+
 def run_sweep(args):
     """Per-kernel table of the other configurations of the path, one JSON line each (not the bench
     line): single-row and small-batch quantised products over the Llama-3-8B matrix shapes, and
@@ -931,6 +1133,10 @@ def main():
     ap.add_argument("--tp-prompt", type=int, default=2048)
     ap.add_argument("--tp-nccl", action="store_true", help="with --tp: keep the decode step on NCCL all-reduces")
     ap.add_argument("--no-tp", action="store_true", help="with --gpus N > 1: skip the tensor-parallel leg after the replicas")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="prefill and decode of a Koludra decoder at two layer sizes beside a Llama decoder of equal size")
+    ap.add_argument("--hybrid-only", type=int, default=0, help="with --hybrid: only this width (2048 or 4096)")
+    ap.add_argument("--no-llama", action="store_true", help="with --hybrid: skip the Llama side")
     ap.add_argument("--gemv-reps", type=int, default=8)
     ap.add_argument("--kernel-table", action="store_true",
                     help="add the device time per kernel of 8 extra decode steps (torch.profiler) as `kernel_table`")
@@ -942,6 +1148,8 @@ def main():
         run_reference(args)
     elif args.sweep:
         run_sweep(args)
+    elif args.hybrid:
+        run_hybrid(args)
     elif args.gemv_only:
         run_gemv_only(args)
     elif args.q5_only:

@@ -63,6 +63,17 @@ __device__ __forceinline__ float conv_silu(const fb200_delta_args& a, int b, int
   return dr_silu(acc);
 }
 
+// what the cached inputs contribute to the convolution of channel c at position pos
+__device__ __forceinline__ float conv_past(const fb200_delta_args& a, int b, int c, int pos) {
+  float acc = 0.f;
+#pragma unroll 4
+  for (int j = 0; j < a.taps - 1; ++j) {
+    const int p = pos - (a.taps - 1) + j;
+    if (p >= 0) acc = fmaf(a.conv_w[(size_t)j * a.channels + c], a.ring[((size_t)b * a.taps + p % a.taps) * a.channels + c], acc);
+  }
+  return acc;
+}
+
 // A column's d elements lie over LPC lanes, EPT per lane: element 4 (i LPC + p) + j is float j of piece i of lane p.
 template <int EPT, int LPC>
 __device__ __forceinline__ void load_column(const float* col, int p, float2 (&s)[EPT / 2]) {
@@ -129,18 +140,31 @@ __global__ void __launch_bounds__(ST_MAX_THREADS) delta_step_kernel(const fb200_
   float2 s[EPT / 2];
   const bool has0 = c0 < a.v && pos > 0;
   if (has0) load_column<EPT, LPC>(st + (size_t)c0 * a.dp, p, s);
+  // so were the convolution's older inputs: threads take q [dp] | k [dp], and a lane per column its v channel
+  auto qk_channel = [&](int i) { return i < a.dp ? (i < a.d ? hk * a.d + i : -1) : (i - a.dp < a.d ? (a.hk + hk) * a.d + i - a.dp : -1); };
+  const int ch0 = tid < 2 * a.dp ? qk_channel(tid) : -1;
+  const float past0 = ch0 >= 0 ? conv_past(a, b, ch0, pos) : 0.f, w0 = ch0 >= 0 ? a.conv_w[(size_t)(a.taps - 1) * a.channels + ch0] : 0.f;
+  float vpast = 0.f, vw = 0.f;
+  if (p == 0 && c0 < a.v) {
+    vpast = conv_past(a, b, a.off_v + h * a.v + c0, pos);
+    vw = a.conv_w[(size_t)(a.taps - 1) * a.channels + a.off_v + h * a.v + c0];
+  }
   pdl_launch_dependents();
   pdl_wait();
   const float* yr = a.y + (size_t)b * a.ldy;
+  float v0 = 0.f;
+  if (p == 0 && c0 < a.v) v0 = dr_silu(fmaf(vw, yr[a.off_v + h * a.v + c0], vpast));
+  v0 = __shfl_sync(0xFFFFFFFFu, v0, lane & ~(LPC - 1));
+  for (int i = tid; i < 2 * a.dp; i += nt) {
+    const int ch = i == tid ? ch0 : qk_channel(i);
+    float x = 0.f;
+    if (ch >= 0) x = i == tid ? dr_silu(fmaf(w0, yr[ch], past0)) : conv_silu(a, b, ch, 0, pos);
+    (i < a.dp ? qs : ks - a.dp)[i] = x;
+  }
+  __syncthreads();
   float skk = 0.f, sqq = 0.f, skq = 0.f;
   for (int i = tid; i < a.dp; i += nt) {
-    float k = 0.f, q = 0.f;
-    if (i < a.d) {
-      q = conv_silu(a, b, hk * a.d + i, 0, pos);
-      k = conv_silu(a, b, (a.hk + hk) * a.d + i, 0, pos);
-    }
-    ks[i] = k;
-    qs[i] = q;
+    const float k = ks[i], q = qs[i];
     skk = fmaf(k, k, skk);
     sqq = fmaf(q, q, sqq);
     skq = fmaf(k, q, skq);
@@ -171,7 +195,7 @@ __global__ void __launch_bounds__(ST_MAX_THREADS) delta_step_kernel(const fb200_
         for (int i = 0; i < EPT / 2; ++i) s[i] = make_float2(0.f, 0.f);
       }
     }
-    const float v = in ? conv_silu(a, b, a.off_v + h * a.v + c, 0, pos) : 0.f;
+    const float v = it == 0 ? v0 : in ? conv_silu(a, b, a.off_v + h * a.v + c, 0, pos) : 0.f;
     float dk, dq;
     column_dots<EPT, LPC>(s, ks, qs, p, dk, dq);
     const float u = beta * (v - g * (dk * ik));
@@ -335,16 +359,17 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prep_kernel(const fb200
 
 constexpr int SC_WARPS = 8;
 
-// TOK tokens per shared-memory stage (a multiple of CH)
-template <int EPT, int LPC, int TOK>
+// A group of LPC lanes owns CPT columns of S (k and q read from shared memory serve all of them), TOK tokens make a
+// shared-memory stage (a multiple of CH).
+template <int EPT, int LPC, int CPT, int TOK>
 __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_delta_args a) {
-  constexpr int DP = EPT * LPC, COLS = SC_WARPS * 32 / LPC, THREADS = SC_WARPS * 32, NC = TOK / CH;
+  constexpr int DP = EPT * LPC, GROUPS = SC_WARPS * 32 / LPC, COLS = GROUPS * CPT, THREADS = SC_WARPS * 32, NC = TOK / CH;
   // floats of a stage: k, q [TOK][DP], v [COLS][TOK], pairs [NC][PAIRS], g [TOK], beta [TOK]
   constexpr int OV = 2 * TOK * DP, OP = OV + COLS * TOK, OG = OP + NC * PAIRS, STAGE = OG + 2 * TOK;
   constexpr bool KEEP = EPT <= 16;  // k of the four tokens stays in registers for the update
   extern __shared__ __align__(16) float dsm[];
   const int tid = threadIdx.x, lane = tid & 31, h = blockIdx.y, b = blockIdx.z, group = a.h / a.hk, hk = h / group, hv = a.h * a.v;
-  const int p = tid % LPC, cl = tid / LPC, c = blockIdx.x * COLS + cl;
+  const int p = tid % LPC, cl = tid / LPC, c = blockIdx.x * COLS + cl;  // columns c, c + GROUPS, ..
   const int pos = *a.pos_dev, nchunks = (a.s + CH - 1) / CH;
   const size_t row0 = (size_t)b * a.s;
   auto cp4 = [](const float* dst, const float* src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory"); };
@@ -381,13 +406,16 @@ __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_d
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   fetch(0, 0);
-  float2 s[EPT / 2];
-  float* col = a.state + (((size_t)b * a.h + h) * a.v + c) * a.dp;
-  if (c < a.v && pos > 0) {
-    load_column<EPT, LPC>(col, p, s);
-  } else {
+  float2 s[CPT][EPT / 2];
+  float* state = a.state + ((size_t)b * a.h + h) * (size_t)a.v * a.dp;
 #pragma unroll
-    for (int i = 0; i < EPT / 2; ++i) s[i] = make_float2(0.f, 0.f);
+  for (int cc = 0; cc < CPT; ++cc) {
+    if (c + cc * GROUPS < a.v && pos > 0) {
+      load_column<EPT, LPC>(state + (size_t)(c + cc * GROUPS) * a.dp, p, s[cc]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < EPT / 2; ++i) s[cc][i] = make_float2(0.f, 0.f);
+    }
   }
   const int stages = (a.s + TOK - 1) / TOK;
   for (int st = 0; st < stages; ++st) {
@@ -406,44 +434,57 @@ __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_d
       const float *kb = sb + ch * CH * DP, *qb = sb + (TOK + ch * CH) * DP;
       // ---- a_i = S^T k_i, c_i = S^T q_i over this lane's elements
       float2 kf[KEEP ? CH : 1][EPT / 2];
-      float val[2 * CH];
+      float val[CPT][2 * CH];
 #pragma unroll
       for (int i = 0; i < CH; ++i) {
-        float2 k0 = make_float2(0.f, 0.f), k1 = k0, q0 = k0, q1 = k0;
+        float2 ka[CPT], qa[CPT];
+#pragma unroll
+        for (int cc = 0; cc < CPT; ++cc) ka[cc] = qa[cc] = make_float2(0.f, 0.f);
 #pragma unroll
         for (int e = 0; e < EPT / 4; ++e) {
           const float4 k = *reinterpret_cast<const float4*>(kb + i * DP + 4 * (e * LPC + p));
           const float4 q = *reinterpret_cast<const float4*>(qb + i * DP + 4 * (e * LPC + p));
-          k0 = fma2(s[2 * e], make_float2(k.x, k.y), k0);
-          k1 = fma2(s[2 * e + 1], make_float2(k.z, k.w), k1);
-          q0 = fma2(s[2 * e], make_float2(q.x, q.y), q0);
-          q1 = fma2(s[2 * e + 1], make_float2(q.z, q.w), q1);
+#pragma unroll
+          for (int cc = 0; cc < CPT; ++cc) {
+            ka[cc] = fma2(s[cc][2 * e], make_float2(k.x, k.y), ka[cc]);
+            qa[cc] = fma2(s[cc][2 * e], make_float2(q.x, q.y), qa[cc]);
+            ka[cc] = fma2(s[cc][2 * e + 1], make_float2(k.z, k.w), ka[cc]);
+            qa[cc] = fma2(s[cc][2 * e + 1], make_float2(q.z, q.w), qa[cc]);
+          }
           if (KEEP) {
             kf[KEEP ? i : 0][2 * e] = make_float2(k.x, k.y);
             kf[KEEP ? i : 0][2 * e + 1] = make_float2(k.z, k.w);
           }
         }
-        val[i] = (k0.x + k0.y) + (k1.x + k1.y);
-        val[CH + i] = (q0.x + q0.y) + (q1.x + q1.y);
+#pragma unroll
+        for (int cc = 0; cc < CPT; ++cc) {
+          val[cc][i] = ka[cc].x + ka[cc].y;
+          val[cc][CH + i] = qa[cc].x + qa[cc].y;
+        }
       }
       // ---- totals over the LPC lanes: eight values over eight lanes by halving, then the rest of the lanes
 #pragma unroll
       for (int o = 4; o > 0; o >>= 1) {
         const bool up = lane & o;
 #pragma unroll
-        for (int i = 0; i < o; ++i) {
-          const float send = up ? val[i] : val[i + o], keep = up ? val[i + o] : val[i];
-          val[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, o);
-        }
+        for (int i = 0; i < o; ++i)
+#pragma unroll
+          for (int cc = 0; cc < CPT; ++cc) {
+            const float send = up ? val[cc][i] : val[cc][i + o], keep = up ? val[cc][i + o] : val[cc][i];
+            val[cc][i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, o);
+          }
       }
-      float mine = val[0];  // lane l: value l % 8
+      float av[CPT][CH], cv[CPT][CH];
 #pragma unroll
-      for (int o = 8; o < LPC; o <<= 1) mine += __shfl_xor_sync(0xFFFFFFFFu, mine, o);
-      float av[CH], cv[CH];
+      for (int cc = 0; cc < CPT; ++cc) {
+        float mine = val[cc][0];  // lane l: value l % 8
 #pragma unroll
-      for (int i = 0; i < CH; ++i) {
-        av[i] = __shfl_sync(0xFFFFFFFFu, mine, (lane & ~7) | i);
-        cv[i] = __shfl_sync(0xFFFFFFFFu, mine, (lane & ~7) | (CH + i));
+        for (int o = 8; o < LPC; o <<= 1) mine += __shfl_xor_sync(0xFFFFFFFFu, mine, o);
+#pragma unroll
+        for (int i = 0; i < CH; ++i) {
+          av[cc][i] = __shfl_sync(0xFFFFFFFFu, mine, (lane & ~7) | i);
+          cv[cc][i] = __shfl_sync(0xFFFFFFFFu, mine, (lane & ~7) | (CH + i));
+        }
       }
       // ---- the four tokens in order
       float pr[PAIRS];
@@ -453,49 +494,65 @@ __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_d
         pr[4 * i] = x.x; pr[4 * i + 1] = x.y; pr[4 * i + 2] = x.z; pr[4 * i + 3] = x.w;
       }
       const float4 g4 = *reinterpret_cast<const float4*>(sb + OG + ch * CH), b4 = *reinterpret_cast<const float4*>(sb + OG + TOK + ch * CH);
-      const float4 v4 = *reinterpret_cast<const float4*>(sb + OV + cl * TOK + ch * CH);
-      const float gi[CH] = {g4.x, g4.y, g4.z, g4.w}, bi[CH] = {b4.x, b4.y, b4.z, b4.w}, vi[CH] = {v4.x, v4.y, v4.z, v4.w};
-      float w[CH], out = 0.f, G = 1.f;
-      int pk = 0, pq = 6;
+      const float gi[CH] = {g4.x, g4.y, g4.z, g4.w}, bi[CH] = {b4.x, b4.y, b4.z, b4.w};
+      const float2 G2 = make_float2(((g4.x * g4.y) * g4.z) * g4.w, ((g4.x * g4.y) * g4.z) * g4.w);
+      float w[CPT][CH];
 #pragma unroll
-      for (int i = 0; i < CH; ++i) {
-        G *= gi[i];
-        float uk = G * av[i], o = G * cv[i];
+      for (int cc = 0; cc < CPT; ++cc) {
+        const float4 v4 = *reinterpret_cast<const float4*>(sb + OV + (cl + cc * GROUPS) * TOK + ch * CH);
+        const float vi[CH] = {v4.x, v4.y, v4.z, v4.w};
+        float out = 0.f, G = 1.f;
+        int pk = 0, pq = 6;
 #pragma unroll
-        for (int j = 0; j < CH; ++j)
-          if (j < i) {
-            w[j] *= gi[i];
-            uk = fmaf(pr[pk++], w[j], uk);
-            o = fmaf(pr[pq++], w[j], o);
-          }
-        w[i] = bi[i] * (vi[i] - uk);
-        o = fmaf(pr[pq++], w[i], o);
-        if (p == i) out = o;
+        for (int i = 0; i < CH; ++i) {
+          G *= gi[i];
+          float uk = G * av[cc][i], o = G * cv[cc][i];
+#pragma unroll
+          for (int j = 0; j < CH; ++j)
+            if (j < i) {
+              w[cc][j] *= gi[i];
+              uk = fmaf(pr[pk++], w[cc][j], uk);
+              o = fmaf(pr[pq++], w[cc][j], o);
+            }
+          w[cc][i] = bi[i] * (vi[i] - uk);
+          o = fmaf(pr[pq++], w[cc][i], o);
+          if (p == i) out = o;
+        }
+        const int col = c + cc * GROUPS;
+        if (p < CH && col < a.v && t0 + p < a.s) a.o[(row0 + t0 + p) * hv + h * a.v + col] = out;
       }
-      if (p < CH && c < a.v && t0 + p < a.s) a.o[(row0 + t0 + p) * hv + h * a.v + c] = out;
       // ---- S <- G S + sum_j k_j w_j
-      const float2 G2 = make_float2(G, G);
 #pragma unroll
-      for (int e = 0; e < EPT / 2; ++e) s[e] = mul2(s[e], G2);
+      for (int cc = 0; cc < CPT; ++cc)
+#pragma unroll
+        for (int e = 0; e < EPT / 2; ++e) s[cc][e] = mul2(s[cc][e], G2);
 #pragma unroll
       for (int i = 0; i < CH; ++i) {
-        const float2 w2 = make_float2(w[i], w[i]);
 #pragma unroll
         for (int e = 0; e < EPT / 4; ++e) {
+          float2 k0, k1;
           if (KEEP) {
-            s[2 * e] = fma2(kf[KEEP ? i : 0][2 * e], w2, s[2 * e]);
-            s[2 * e + 1] = fma2(kf[KEEP ? i : 0][2 * e + 1], w2, s[2 * e + 1]);
+            k0 = kf[KEEP ? i : 0][2 * e];
+            k1 = kf[KEEP ? i : 0][2 * e + 1];
           } else {
             const float4 k = *reinterpret_cast<const float4*>(kb + i * DP + 4 * (e * LPC + p));
-            s[2 * e] = fma2(make_float2(k.x, k.y), w2, s[2 * e]);
-            s[2 * e + 1] = fma2(make_float2(k.z, k.w), w2, s[2 * e + 1]);
+            k0 = make_float2(k.x, k.y);
+            k1 = make_float2(k.z, k.w);
+          }
+#pragma unroll
+          for (int cc = 0; cc < CPT; ++cc) {
+            const float2 w2 = make_float2(w[cc][i], w[cc][i]);
+            s[cc][2 * e] = fma2(k0, w2, s[cc][2 * e]);
+            s[cc][2 * e + 1] = fma2(k1, w2, s[cc][2 * e + 1]);
           }
         }
       }
     }
     __syncthreads();  // the stage is free before the one after next lands in it
   }
-  if (c < a.v) store_column<EPT, LPC>(col, p, s);
+#pragma unroll
+  for (int cc = 0; cc < CPT; ++cc)
+    if (c + cc * GROUPS < a.v) store_column<EPT, LPC>(state + (size_t)(c + cc * GROUPS) * a.dp, p, s[cc]);
 }
 
 // A warp per (row, head): RMSNorm over v, the plain weight, the SiLU gate.
@@ -536,16 +593,16 @@ int launch_step(fb200_device* dev, const fb200_delta_args& a) {
   return fb200_launch(dev, delta_step_kernel<EPT, LPC>, dim3((unsigned)a.h, (unsigned)a.b), dim3((unsigned)threads), smem, true, a);
 }
 
-template <int EPT, int LPC, int TOK>
+template <int EPT, int LPC, int CPT, int TOK>
 int launch_scan(fb200_device* dev, const fb200_delta_args& a) {
-  constexpr int DP = EPT * LPC, COLS = SC_WARPS * 32 / LPC;
+  constexpr int DP = EPT * LPC, COLS = SC_WARPS * 32 / LPC * CPT;
   constexpr size_t smem = (size_t)2 * (2 * TOK * DP + COLS * TOK + TOK / CH * PAIRS + 2 * TOK) * 4;
   static bool configured[64] = {false};
   if (!configured[dev->ordinal & 63]) {
-    FB_CUDA(dev, cudaFuncSetAttribute(delta_scan_kernel<EPT, LPC, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    FB_CUDA(dev, cudaFuncSetAttribute(delta_scan_kernel<EPT, LPC, CPT, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured[dev->ordinal & 63] = true;
   }
-  delta_scan_kernel<EPT, LPC, TOK><<<dim3((unsigned)((a.v + COLS - 1) / COLS), (unsigned)a.h, (unsigned)a.b), SC_WARPS * 32, smem, dev->stream>>>(a);
+  delta_scan_kernel<EPT, LPC, CPT, TOK><<<dim3((unsigned)((a.v + COLS - 1) / COLS), (unsigned)a.h, (unsigned)a.b), SC_WARPS * 32, smem, dev->stream>>>(a);
   FB_LAUNCH_CHECK(dev);
   return FB200_OK;
 }
@@ -592,12 +649,12 @@ int fb200_delta_prompt(fb200_device* dev, const fb200_delta_args& a) {
   }
   if (rc) return rc;
   switch (a.dp) {
-    case 32: rc = launch_scan<4, 8, 16>(dev, a); break;
-    case 64: rc = launch_scan<8, 8, 16>(dev, a); break;
-    case 128: rc = launch_scan<16, 8, 16>(dev, a); break;
-    case 256: rc = launch_scan<32, 8, 16>(dev, a); break;
-    case 512: rc = launch_scan<32, 16, 8>(dev, a); break;
-    default: rc = launch_scan<32, 32, 4>(dev, a); break;
+    case 32: rc = launch_scan<4, 8, 2, 16>(dev, a); break;
+    case 64: rc = launch_scan<8, 8, 2, 16>(dev, a); break;
+    case 128: rc = launch_scan<8, 16, 2, 16>(dev, a); break;
+    case 256: rc = launch_scan<16, 16, 2, 16>(dev, a); break;
+    case 512: rc = launch_scan<16, 32, 2, 8>(dev, a); break;
+    default: rc = launch_scan<32, 32, 1, 4>(dev, a); break;
   }
   if (rc) return rc;
   const size_t warps = (size_t)a.b * a.s * a.h;

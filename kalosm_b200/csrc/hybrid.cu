@@ -289,7 +289,7 @@ int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows) {
       const bool exp = expanded(hy, c, 16);
       const size_t r = exp ? std::min(rows, (size_t)16 * m->cfg.max_batch) : rows;
       qa = std::max(qa, r * c.heads * (size_t)(c.kv_rank + c.rot_dim));
-      part = std::max(part, std::max(r * c.heads, (size_t)4 * dev->sm_count) * (size_t)(c.kv_rank + 2));
+      part = std::max(part, std::max(r * c.heads, (size_t)8 * dev->sm_count) * (size_t)(c.kv_rank + 2));
     }
   }
   struct { void** p; size_t bytes; } bufs[] = {
