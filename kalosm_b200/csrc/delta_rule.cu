@@ -357,11 +357,12 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prep_kernel(const fb200
   }
 }
 
-constexpr int SC_WARPS = 8;
+constexpr int SC_WARPS = 8, CPT = 4;  // columns per group of lanes
 
-// A group of LPC lanes owns CPT columns of S (k and q read from shared memory serve all of them), TOK tokens make a
-// shared-memory stage (a multiple of CH).
-template <int EPT, int LPC, int CPT, int TOK>
+// A group of LPC lanes owns CPT columns of S: k and q read from shared memory serve all of them, and the sums are
+// reduced so that lane p ends up with those of column p % 4, so one pass over the four tokens does all columns.
+// TOK tokens make a shared-memory stage (a multiple of CH).
+template <int EPT, int LPC, int TOK>
 __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_delta_args a) {
   constexpr int DP = EPT * LPC, GROUPS = SC_WARPS * 32 / LPC, COLS = GROUPS * CPT, THREADS = SC_WARPS * 32, NC = TOK / CH;
   // floats of a stage: k, q [TOK][DP], v [COLS][TOK], pairs [NC][PAIRS], g [TOK], beta [TOK]
@@ -462,29 +463,17 @@ __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_d
           val[cc][CH + i] = qa[cc].x + qa[cc].y;
         }
       }
-      // ---- totals over the LPC lanes: eight values over eight lanes by halving, then the rest of the lanes
+      // ---- totals over the LPC lanes: two halving steps leave lane p with column p % 4, the rest adds up its lanes
 #pragma unroll
-      for (int o = 4; o > 0; o >>= 1) {
-        const bool up = lane & o;
+      for (int x = 0; x < 2 * CH; ++x) {
+        const bool odd = lane & 1, high = lane & 2;
+        const float s01 = odd ? val[0][x] : val[1][x], k01 = odd ? val[1][x] : val[0][x];
+        const float s23 = odd ? val[2][x] : val[3][x], k23 = odd ? val[3][x] : val[2][x];
+        const float c01 = k01 + __shfl_xor_sync(0xFFFFFFFFu, s01, 1), c23 = k23 + __shfl_xor_sync(0xFFFFFFFFu, s23, 1);
+        float t = (high ? c23 : c01) + __shfl_xor_sync(0xFFFFFFFFu, high ? c01 : c23, 2);
 #pragma unroll
-        for (int i = 0; i < o; ++i)
-#pragma unroll
-          for (int cc = 0; cc < CPT; ++cc) {
-            const float send = up ? val[cc][i] : val[cc][i + o], keep = up ? val[cc][i + o] : val[cc][i];
-            val[cc][i] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, o);
-          }
-      }
-      float av[CPT][CH], cv[CPT][CH];
-#pragma unroll
-      for (int cc = 0; cc < CPT; ++cc) {
-        float mine = val[cc][0];  // lane l: value l % 8
-#pragma unroll
-        for (int o = 8; o < LPC; o <<= 1) mine += __shfl_xor_sync(0xFFFFFFFFu, mine, o);
-#pragma unroll
-        for (int i = 0; i < CH; ++i) {
-          av[cc][i] = __shfl_sync(0xFFFFFFFFu, mine, (lane & ~7) | i);
-          cv[cc][i] = __shfl_sync(0xFFFFFFFFu, mine, (lane & ~7) | (CH + i));
-        }
+        for (int o = 4; o < LPC; o <<= 1) t += __shfl_xor_sync(0xFFFFFFFFu, t, o);
+        val[0][x] = t;
       }
       // ---- the four tokens in order
       float pr[PAIRS];
@@ -496,31 +485,36 @@ __global__ void __launch_bounds__(SC_WARPS * 32) delta_scan_kernel(const fb200_d
       const float4 g4 = *reinterpret_cast<const float4*>(sb + OG + ch * CH), b4 = *reinterpret_cast<const float4*>(sb + OG + TOK + ch * CH);
       const float gi[CH] = {g4.x, g4.y, g4.z, g4.w}, bi[CH] = {b4.x, b4.y, b4.z, b4.w};
       const float2 G2 = make_float2(((g4.x * g4.y) * g4.z) * g4.w, ((g4.x * g4.y) * g4.z) * g4.w);
+      const int mycol = cl + (p & 3) * GROUPS;
+      const float4 v4 = *reinterpret_cast<const float4*>(sb + OV + mycol * TOK + ch * CH);
+      const float vi[CH] = {v4.x, v4.y, v4.z, v4.w};
+      float u[CH], out[CH], G = 1.f;
+      int pk = 0, pq = 6;
+#pragma unroll
+      for (int i = 0; i < CH; ++i) {
+        G *= gi[i];
+        float uk = G * val[0][i], o = G * val[0][CH + i];
+#pragma unroll
+        for (int j = 0; j < CH; ++j)
+          if (j < i) {
+            u[j] *= gi[i];
+            uk = fmaf(pr[pk++], u[j], uk);
+            o = fmaf(pr[pq++], u[j], o);
+          }
+        u[i] = bi[i] * (vi[i] - uk);
+        out[i] = fmaf(pr[pq++], u[i], o);
+      }
+      if (p < 8 && blockIdx.x * COLS + mycol < a.v) {  // lanes 0..3 store tokens 0 and 1, lanes 4..7 tokens 2 and 3
+        const int i0 = p < 4 ? 0 : 2;
+        float* dst = a.o + (row0 + t0 + i0) * hv + h * a.v + blockIdx.x * COLS + mycol;
+        if (t0 + i0 < a.s) dst[0] = p < 4 ? out[0] : out[2];
+        if (t0 + i0 + 1 < a.s) dst[hv] = p < 4 ? out[1] : out[3];
+      }
       float w[CPT][CH];
 #pragma unroll
-      for (int cc = 0; cc < CPT; ++cc) {
-        const float4 v4 = *reinterpret_cast<const float4*>(sb + OV + (cl + cc * GROUPS) * TOK + ch * CH);
-        const float vi[CH] = {v4.x, v4.y, v4.z, v4.w};
-        float out = 0.f, G = 1.f;
-        int pk = 0, pq = 6;
+      for (int cc = 0; cc < CPT; ++cc)
 #pragma unroll
-        for (int i = 0; i < CH; ++i) {
-          G *= gi[i];
-          float uk = G * av[cc][i], o = G * cv[cc][i];
-#pragma unroll
-          for (int j = 0; j < CH; ++j)
-            if (j < i) {
-              w[cc][j] *= gi[i];
-              uk = fmaf(pr[pk++], w[cc][j], uk);
-              o = fmaf(pr[pq++], w[cc][j], o);
-            }
-          w[cc][i] = bi[i] * (vi[i] - uk);
-          o = fmaf(pr[pq++], w[cc][i], o);
-          if (p == i) out = o;
-        }
-        const int col = c + cc * GROUPS;
-        if (p < CH && col < a.v && t0 + p < a.s) a.o[(row0 + t0 + p) * hv + h * a.v + col] = out;
-      }
+        for (int i = 0; i < CH; ++i) w[cc][i] = __shfl_sync(0xFFFFFFFFu, u[i], (lane & ~3) | cc);
       // ---- S <- G S + sum_j k_j w_j
 #pragma unroll
       for (int cc = 0; cc < CPT; ++cc)
@@ -593,16 +587,16 @@ int launch_step(fb200_device* dev, const fb200_delta_args& a) {
   return fb200_launch(dev, delta_step_kernel<EPT, LPC>, dim3((unsigned)a.h, (unsigned)a.b), dim3((unsigned)threads), smem, true, a);
 }
 
-template <int EPT, int LPC, int CPT, int TOK>
+template <int EPT, int LPC, int TOK>
 int launch_scan(fb200_device* dev, const fb200_delta_args& a) {
   constexpr int DP = EPT * LPC, COLS = SC_WARPS * 32 / LPC * CPT;
   constexpr size_t smem = (size_t)2 * (2 * TOK * DP + COLS * TOK + TOK / CH * PAIRS + 2 * TOK) * 4;
   static bool configured[64] = {false};
   if (!configured[dev->ordinal & 63]) {
-    FB_CUDA(dev, cudaFuncSetAttribute(delta_scan_kernel<EPT, LPC, CPT, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    FB_CUDA(dev, cudaFuncSetAttribute(delta_scan_kernel<EPT, LPC, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured[dev->ordinal & 63] = true;
   }
-  delta_scan_kernel<EPT, LPC, CPT, TOK><<<dim3((unsigned)((a.v + COLS - 1) / COLS), (unsigned)a.h, (unsigned)a.b), SC_WARPS * 32, smem, dev->stream>>>(a);
+  delta_scan_kernel<EPT, LPC, TOK><<<dim3((unsigned)((a.v + COLS - 1) / COLS), (unsigned)a.h, (unsigned)a.b), SC_WARPS * 32, smem, dev->stream>>>(a);
   FB_LAUNCH_CHECK(dev);
   return FB200_OK;
 }
@@ -649,12 +643,12 @@ int fb200_delta_prompt(fb200_device* dev, const fb200_delta_args& a) {
   }
   if (rc) return rc;
   switch (a.dp) {
-    case 32: rc = launch_scan<4, 8, 2, 16>(dev, a); break;
-    case 64: rc = launch_scan<8, 8, 2, 16>(dev, a); break;
-    case 128: rc = launch_scan<8, 16, 2, 16>(dev, a); break;
-    case 256: rc = launch_scan<16, 16, 2, 16>(dev, a); break;
-    case 512: rc = launch_scan<16, 32, 2, 8>(dev, a); break;
-    default: rc = launch_scan<32, 32, 1, 4>(dev, a); break;
+    case 32: rc = launch_scan<4, 8, 16>(dev, a); break;
+    case 64: rc = launch_scan<4, 16, 16>(dev, a); break;
+    case 128: rc = launch_scan<4, 32, 16>(dev, a); break;
+    case 256: rc = launch_scan<8, 32, 16>(dev, a); break;
+    case 512: rc = launch_scan<16, 32, 8>(dev, a); break;
+    default: rc = launch_scan<32, 32, 4>(dev, a); break;
   }
   if (rc) return rc;
   const size_t warps = (size_t)a.b * a.s * a.h;

@@ -4,9 +4,11 @@
 // product, dense_tc.cu), and the attention runs over them; the rotated key part, shared by the heads, is read
 // from the cache as it is. Bound: tensor cores, 2 (d + r + v) flops per head and visible (query, key) pair.
 //
-// latent_prefill_kernel: the scheme of attn_prefill_tc.cu (one CTA = 128 query rows of one head; a softmax thread per
-// row, a warp that issues the MMAs, a warp that requests the tiles; S = Q K^T double-buffered in TMEM, P written back
+// latent_prefill_kernel: the scheme of attn_prefill_tc.cu (128 query rows of one head: a softmax thread per row; a
+// warp that issues the MMAs, a warp that requests the tiles; S = Q K^T double-buffered in TMEM, P written back
 // over S, O accumulated in TMEM and rescaled lazily), with
+//  * one or two groups of 128 rows per CTA (G): two groups share every key and value tile and take turns, one group's
+//    products run under the other's softmax; each group visits only its own range of tiles,
 //  * keys of two parts: NK boxes of 64 columns per 64-key tile, the first na from the expanded keys (columns h d ..; a
 //    box may run into the next head's columns, which meet zero columns of Q), the rest from the cache's key part,
 //  * a sliding window: tiles in front of the first visible key are never visited, and only tiles that touch the
@@ -21,7 +23,7 @@
 
 namespace {
 
-constexpr int LP_Q = 128, LP_K = 64, LP_THREADS = 128, LP_BLOCK = LP_THREADS + 64;
+constexpr int LP_Q = 128, LP_K = 64, LP_THREADS = 128;
 constexpr uint32_t LP_BOX = LP_K * 64 * 2;  // bytes of one box: 64 keys x 64 columns of bf16
 constexpr int LP_TAIL = 256;
 constexpr float LP_RESCALE = 8.0f;  // log2 of the growth of a row maximum that triggers a rescale of O
@@ -43,39 +45,54 @@ __device__ __forceinline__ uint32_t lp_pack(float lo, float hi) {
   return *reinterpret_cast<const uint32_t*>(&t);
 }
 
-// NV: 64-column boxes of a value tile; KB, VB: key and value tiles in shared memory
-template <int NV, int KB, int VB>
-__global__ void __launch_bounds__(LP_BLOCK)
+// NV: 64-column boxes of a value tile; KB, VB: key and value tiles in shared memory; G: groups of 128 query rows
+template <int NV, int KB, int VB, int G>
+__global__ void __launch_bounds__(G * LP_THREADS + 64)
 latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, const __grid_constant__ CUtensorMap cmap) {
-  constexpr int COLS = NV <= 2 ? 256 : 512;  // S buffers: columns 0..63 and 64..127; O from 128
+  // TMEM of a group: S buffers in columns 0..63 and 64..127, O from 128
+  constexpr int GCOLS = NV <= 2 ? 256 : 512, COLS = G * GCOLS;
+  static_assert(COLS <= 512, "two groups need values of at most 128 columns");
+  constexpr int SOFT = G * LP_THREADS;  // softmax threads
   extern __shared__ uint8_t sm_raw[];
   uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(sm_raw) + 1023) & ~(uintptr_t)1023);
-  const int kbytes = a.nk * (int)LP_BOX, kchunks = a.nk * 8;
+  const int kbytes = a.nk * (int)LP_BOX, kchunks = a.nk * 8, qbytes = LP_Q * a.nk * 128;
   uint8_t* Ks = sm;                             // [KB][nk boxes]
   uint8_t* Vs = Ks + KB * kbytes;               // [VB][NV boxes]
-  uint8_t* Qs = Vs + VB * NV * (int)LP_BOX;     // [128][64 nk], core-matrix layout
-  uint64_t* bars = reinterpret_cast<uint64_t*>(Qs + LP_Q * a.nk * 128);
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 12);
+  uint8_t* Qs = Vs + VB * NV * (int)LP_BOX;     // [G][128][64 nk], core-matrix layout
+  uint64_t* bars = reinterpret_cast<uint64_t*>(Qs + G * qbytes);
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
   volatile int* dead = reinterpret_cast<volatile int*>(tmem_slot + 1);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const uint32_t bar_s = smem_u32(bars), bar_o = smem_u32(bars + 2), bar_kfull = smem_u32(bars + 3), bar_vfull = smem_u32(bars + 7),
-                 bar_pfull = smem_u32(bars + 10);
+  // per group: S done (one per S buffer), O += P V done, P written; per tile buffer: keys landed, values landed
+  const uint32_t bar_s = smem_u32(bars), bar_o = smem_u32(bars + 4), bar_pfull = smem_u32(bars + 6), bar_kfull = smem_u32(bars + 8),
+                 bar_vfull = smem_u32(bars + 11);
   const int qt = gridDim.x - 1 - blockIdx.x;  // longest key ranges first
   const int head = blockIdx.y, b = blockIdx.z;
-  const int q0 = qt * LP_Q, p0 = a.pos + q0;  // first query row of the pass, its position
-  // keys are counted from kbase: key j is row j - kbase of the expansions
-  const int last = min(a.s, q0 + LP_Q) - 1 + a.pos - a.kbase;
-  const int first = max(0, (a.window ? p0 - a.window + 1 : 0) - a.kbase);
-  const int t_first = first / LP_K, ntiles = last / LP_K + 1 - t_first;
+  const int q0 = qt * LP_Q * G;
+  // keys are counted from kbase: key j is row j - kbase of the expansions. Tiles tf[g] .. tl[g] hold the visible keys of
+  // group g; the groups' ranges start and end in order and leave no tile between them out.
+  int tf[G], tl[G];
+  const int t_first = max(0, (a.window ? a.pos + q0 - a.window + 1 : 0) - a.kbase) / LP_K;
+  int t_last = t_first;
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    const int qg = q0 + g * LP_Q;
+    tf[g] = max(0, (a.window ? a.pos + qg - a.window + 1 : 0) - a.kbase) / LP_K;
+    tl[g] = qg < a.s ? (min(a.s, qg + LP_Q) - 1 + a.pos - a.kbase) / LP_K : tf[g] - 1;
+    t_last = max(t_last, tl[g]);
+  }
+  const int ntiles = t_last - t_first + 1;
 
   if (tid == 0) {
     *dead = 0;
-    mbar_init(bar_s, 1);
-    mbar_init(bar_s + 8, 1);
-    mbar_init(bar_o, 1);
+    for (int g = 0; g < G; ++g) {
+      mbar_init(bar_s + 16 * g, 1);
+      mbar_init(bar_s + 16 * g + 8, 1);
+      mbar_init(bar_o + 8 * g, 1);
+      mbar_init(bar_pfull + 8 * g, LP_THREADS);
+    }
     for (int i = 0; i < KB; ++i) mbar_init(bar_kfull + 8 * i, 1);
     for (int i = 0; i < VB; ++i) mbar_init(bar_vfull + 8 * i, 1);
-    mbar_init(bar_pfull, LP_THREADS);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 0) {
@@ -83,9 +100,10 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
   // ---- Q: rotary positions, bf16, K-major operand layout: [d, zeros to 64 na | r, zeros]
-  if (warp < LP_THREADS / 32) {
+  if (tid < SOFT) {
     const int half = a.r / 2;
-    for (int id = tid; id < LP_Q * kchunks; id += LP_THREADS) {
+    const bool vec = ((a.d + a.r) & 3) == 0;
+    for (int id = tid; id < G * LP_Q * kchunks; id += SOFT) {
       const int row = (id & 7) + ((id / (8 * kchunks)) << 3), c = (id >> 3) % kchunks;
       float x[8];
 #pragma unroll
@@ -93,12 +111,18 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
       if (q0 + row < a.s) {
         const float* q = a.y + ((size_t)b * a.s + q0 + row) * a.ldy + (size_t)head * (a.d + a.r);
         if (c < a.na * 8) {
+          if (vec && c * 8 < a.d) {  // d is a multiple of 8
+            const float4 x0 = *reinterpret_cast<const float4*>(q + c * 8), x1 = *reinterpret_cast<const float4*>(q + c * 8 + 4);
+            x[0] = x0.x; x[1] = x0.y; x[2] = x0.z; x[3] = x0.w;
+            x[4] = x1.x; x[5] = x1.y; x[6] = x1.z; x[7] = x1.w;
+          } else {
 #pragma unroll
-          for (int e = 0; e < 8; ++e)
-            if (c * 8 + e < a.d) x[e] = q[c * 8 + e];
+            for (int e = 0; e < 8; ++e)
+              if (c * 8 + e < a.d) x[e] = q[c * 8 + e];
+          }
         } else {
           const int i0 = (c - a.na * 8) * 8;
-          const float *cs = a.rope_cos + (size_t)(p0 + row) * half, *sn = a.rope_sin + (size_t)(p0 + row) * half;
+          const float *cs = a.rope_cos + (size_t)(a.pos + q0 + row) * half, *sn = a.rope_sin + (size_t)(a.pos + q0 + row) * half;
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
             const int i = i0 + e;
@@ -107,7 +131,7 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
           }
         }
       }
-      *reinterpret_cast<uint4*>(Qs + x_kmajor(row, c, kchunks)) =
+      *reinterpret_cast<uint4*>(Qs + (row >> 7) * qbytes + x_kmajor(row & 127, c, kchunks)) =
           make_uint4(lp_pack(x[0], x[1]), lp_pack(x[2], x[3]), lp_pack(x[4], x[5]), lp_pack(x[6], x[7]));
     }
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // these stores -> tensor-core reads
@@ -119,84 +143,103 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
   // instruction descriptors: fp32 accumulator, bf16 operands, M = 128; S: N = 64, both K-major; O: N = 64 NV, B MN-major
   constexpr uint32_t IDESC_S = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LP_K >> 3) << 17) | ((uint32_t)(LP_Q >> 4) << 24);
   constexpr uint32_t IDESC_O = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(NV * 8) << 17) | ((uint32_t)(LP_Q >> 4) << 24);
+  auto in_range = [&](int g, int t) { return t >= tf[g] && t <= tl[g]; };
 
-  if (warp == LP_THREADS / 32 + 1) {
-    // ---- copy requester
+  if (warp == SOFT / 32 + 1) {
+    // ---- copy requester; tile u of the CTA is tile t_first + u
     if (lane == 0) {
       const int ky = b * a.keys, cy = b * a.cap;
-      auto fetch_k = [&](int t) {
-        const uint32_t dst = smem_u32(Ks) + (uint32_t)((t % KB) * kbytes), bar = bar_kfull + 8 * (t % KB);
-        const int j0 = (t_first + t) * LP_K;
+      auto fetch_k = [&](int u) {
+        const uint32_t dst = smem_u32(Ks) + (uint32_t)((u % KB) * kbytes), bar = bar_kfull + 8 * (u % KB);
+        const int j0 = (t_first + u) * LP_K;
         mbar_expect_tx(bar, (uint32_t)kbytes);
         for (int i = 0; i < a.na; ++i) x_tma_box2(dst + i * LP_BOX, &kvmap, head * a.d + 64 * i, ky + j0, bar);
         for (int i = a.na; i < a.nk; ++i) x_tma_box2(dst + i * LP_BOX, &cmap, a.rk + 64 * (i - a.na), cy + j0, bar);
       };
-      auto fetch_v = [&](int t) {
-        const uint32_t dst = smem_u32(Vs) + (uint32_t)((t % VB) * NV) * LP_BOX, bar = bar_vfull + 8 * (t % VB);
-        const int j0 = (t_first + t) * LP_K;
+      auto fetch_v = [&](int u) {
+        const uint32_t dst = smem_u32(Vs) + (uint32_t)((u % VB) * NV) * LP_BOX, bar = bar_vfull + 8 * (u % VB);
+        const int j0 = (t_first + u) * LP_K;
         mbar_expect_tx(bar, NV * LP_BOX);
         for (int i = 0; i < NV; ++i) x_tma_box2(dst + i * LP_BOX, &kvmap, a.v_col + head * a.v + 64 * i, ky + j0, bar);
       };
       int nkt = 0, nvt = 0;  // tiles requested
       while (nkt < KB && nkt < ntiles) fetch_k(nkt++);
       while (nvt < VB && nvt < ntiles) fetch_v(nvt++);
-      for (int t = 0; t + VB < ntiles; ++t) {
-        // S_t is done: its key tile is free; O += P V_t is done: its value tile is free
-        if (!x_wait(bar_s + 8 * (t & 1), (uint32_t)((t >> 1) & 1), dead, a.status)) break;
-        if (t + KB < ntiles) fetch_k(nkt++);
-        if (!x_wait(bar_o, (uint32_t)(t & 1), dead, a.status)) break;
-        fetch_v(nvt++);
+      bool ok = true;
+      for (int u = 0; u + VB < ntiles && ok; ++u) {
+        const int t = t_first + u;
+#pragma unroll
+        for (int g = 0; g < G; ++g)  // S of every group that uses the tile is done: its key buffer is free
+          if (in_range(g, t)) ok = ok && x_wait(bar_s + 16 * g + 8 * ((t - tf[g]) & 1), (uint32_t)(((t - tf[g]) >> 1) & 1), dead, a.status);
+        if (ok && u + KB < ntiles) fetch_k(nkt++);
+#pragma unroll
+        for (int g = 0; g < G; ++g)  // and O: its value buffer is free
+          if (in_range(g, t)) ok = ok && x_wait(bar_o + 8 * g, (uint32_t)((t - tf[g]) & 1), dead, a.status);
+        if (ok) fetch_v(nvt++);
       }
       if (*dead) {
-        for (int t = max(0, nkt - KB); t < nkt; ++t) x_drain(bar_kfull + 8 * (t % KB), (uint32_t)((t / KB) & 1));
-        for (int t = max(0, nvt - VB); t < nvt; ++t) x_drain(bar_vfull + 8 * (t % VB), (uint32_t)((t / VB) & 1));
+        for (int u = max(0, nkt - KB); u < nkt; ++u) x_drain(bar_kfull + 8 * (u % KB), (uint32_t)((u / KB) & 1));
+        for (int u = max(0, nvt - VB); u < nvt; ++u) x_drain(bar_vfull + 8 * (u % VB), (uint32_t)((u / VB) & 1));
       }
     }
-  } else if (warp == LP_THREADS / 32) {
-    // ---- MMA issuer: S_0, then per tile S_(t+1) (under the softmax of tile t) and O += P V_t
+  } else if (warp == SOFT / 32) {
+    // ---- MMA issuer: per tile and group, S of the next tile (under the softmax of this one), then O += P V
     if (lane == 0) {
       const int steps_d = (a.d + 15) / 16, steps_r = (a.r + 15) / 16;
       const uint32_t q_sbo = (uint32_t)kchunks * 128;
-      auto issue_s = [&](int t) {
-        x_wait(bar_kfull + 8 * (t % KB), (uint32_t)((t / KB) & 1), dead, a.status);
+      auto issue_s = [&](int g, int u) {
+        const int tg = t_first + u - tf[g];
+        x_wait(bar_kfull + 8 * (u % KB), (uint32_t)((u / KB) & 1), dead, a.status);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const uint32_t ks = smem_u32(Ks) + (uint32_t)((t % KB) * kbytes), qs = smem_u32(Qs);
+        const uint32_t ks = smem_u32(Ks) + (uint32_t)((u % KB) * kbytes), qs = smem_u32(Qs) + (uint32_t)(g * qbytes);
         for (int i = 0; i < steps_d + steps_r; ++i) {
           const int s = i < steps_d ? i : a.na * 4 + i - steps_d;  // 16-column step of the padded layout
-          x_mma(tmem + (uint32_t)((t & 1) * LP_K), x_desc(qs + s * 256, 128, q_sbo),
+          x_mma(tmem + (uint32_t)(g * GCOLS + (tg & 1) * LP_K), x_desc(qs + s * 256, 128, q_sbo),
                 x_desc(ks + (s >> 2) * LP_BOX + (s & 3) * 32, 16, 1024, LP_SW128), IDESC_S, i ? 1u : 0u);
         }
-        x_commit(bar_s + 8 * (t & 1));
+        x_commit(bar_s + 16 * g + 8 * (tg & 1));
       };
-      issue_s(0);
-      for (int t = 0; t < ntiles; ++t) {
-        if (t + 1 < ntiles) issue_s(t + 1);
-        x_wait(bar_pfull, (uint32_t)(t & 1), dead, a.status);
-        x_wait(bar_vfull + 8 * (t % VB), (uint32_t)((t / VB) & 1), dead, a.status);
-        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const uint32_t vs = smem_u32(Vs) + (uint32_t)((t % VB) * NV) * LP_BOX;
 #pragma unroll
-        for (int s = 0; s < LP_K / 16; ++s)  // 16 keys = 16 rows of 128 bytes further
-          x_mma_ta(tmem + 2 * LP_K, tmem + (uint32_t)((t & 1) * LP_K + s * 8), x_desc(vs + s * 2048, LP_BOX, 1024, LP_SW128), IDESC_O,
-                   (t | s) ? 1u : 0u);
-        x_commit(bar_o);
+      for (int g = 0; g < G; ++g)
+        if (in_range(g, t_first)) issue_s(g, 0);
+      for (int u = 0; u < ntiles; ++u) {
+        const int t = t_first + u;
+#pragma unroll
+        for (int g = 0; g < G; ++g) {
+          if (u + 1 < ntiles && in_range(g, t + 1)) issue_s(g, u + 1);
+          if (!in_range(g, t)) continue;
+          const int tg = t - tf[g];
+          x_wait(bar_pfull + 8 * g, (uint32_t)(tg & 1), dead, a.status);
+          x_wait(bar_vfull + 8 * (u % VB), (uint32_t)((u / VB) & 1), dead, a.status);
+          asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+          const uint32_t vs = smem_u32(Vs) + (uint32_t)((u % VB) * NV) * LP_BOX, tm = tmem + (uint32_t)(g * GCOLS);
+#pragma unroll
+          for (int s = 0; s < LP_K / 16; ++s)  // 16 keys = 16 rows of 128 bytes further
+            x_mma_ta(tm + 2 * LP_K, tm + (uint32_t)((tg & 1) * LP_K + s * 8), x_desc(vs + s * 2048, LP_BOX, 1024, LP_SW128), IDESC_O,
+                     (tg | s) ? 1u : 0u);
+          x_commit(bar_o + 8 * g);
+        }
       }
     }
   } else {
-    // ---- softmax threads: thread r owns query row r = TMEM lane r
-    const uint32_t tl = tmem + ((uint32_t)(32 * warp) << 16);
+    // ---- softmax threads: thread r of group g owns query row q0 + 128 g + r = TMEM lane r
+    const int g = G > 1 ? warp >> 2 : 0, r = tid & 127;
+    const int t0 = G > 1 && g ? tf[G - 1] : tf[0], n = (G > 1 && g ? tl[G - 1] : tl[0]) - t0 + 1;
+    const uint32_t tl_base = tmem + (uint32_t)(g * GCOLS) + ((uint32_t)(32 * (warp & 3)) << 16);
+    const uint32_t my_s = bar_s + 16 * g, my_o = bar_o + 8 * g, my_p = bar_pfull + 8 * g;
     float m_ref = -INFINITY, l_run = 0.f;
-    const int row = q0 + tid;
-    const int hi = a.pos + row - a.kbase;                          // last visible key of this row
-    const int lo = a.window ? hi - a.window + 1 : -(1 << 30);      // first visible key
-    const int hi_min = p0 - a.kbase, lo_max = a.window ? last - a.window + 1 : -(1 << 30);
-    for (int t = 0; t < ntiles; ++t) {
-      const int sb = t & 1, kt = (t_first + t) * LP_K;
-      x_wait(bar_s + 8 * sb, (uint32_t)((t >> 1) & 1), dead, a.status);
+    const int qg = q0 + g * LP_Q, row = qg + r;
+    const int hi = a.pos + row - a.kbase;                      // last visible key of this row
+    const int lo = a.window ? hi - a.window + 1 : -(1 << 30);  // first visible key
+    const int hi_min = a.pos + qg - a.kbase;                   // of the group's rows
+    const int lo_max = a.window ? min(a.s, qg + LP_Q) - 1 + a.pos - a.kbase - a.window + 1 : -(1 << 30);
+    for (int t = 0; t < n; ++t) {
+      const int sb = t & 1, kt = (t0 + t) * LP_K;
+      x_wait(my_s + 8 * sb, (uint32_t)((t >> 1) & 1), dead, a.status);
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       uint32_t sv[2][32];
-      x_ld32(tl + (uint32_t)(sb * LP_K), sv[0]);
-      x_ld32(tl + (uint32_t)(sb * LP_K + 32), sv[1]);
+      x_ld32(tl_base + (uint32_t)(sb * LP_K), sv[0]);
+      x_ld32(tl_base + (uint32_t)(sb * LP_K + 32), sv[1]);
       asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       if (kt + LP_K - 1 > hi_min || kt < lo_max) {  // the tile touches the diagonal or the window's edge of some row
 #pragma unroll
@@ -221,51 +264,53 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
         pk[j] = lp_pack(e0, e1);
       }
       l_run = l_run * alpha + psum;
-      x_st32(tl + (uint32_t)(sb * LP_K), pk);
+      x_st32(tl_base + (uint32_t)(sb * LP_K), pk);
       if (t > 0 && __any_sync(0xFFFFFFFFu, grow)) {  // O is rescaled behind the previous tile's product
-        x_wait(bar_o, (uint32_t)((t - 1) & 1), dead, a.status);
+        x_wait(my_o, (uint32_t)((t - 1) & 1), dead, a.status);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
         for (int c = 0; c < NV * 2; ++c) {
           uint32_t ov[32];
-          x_ld32(tl + 2 * LP_K + 32 * c, ov);
+          x_ld32(tl_base + 2 * LP_K + 32 * c, ov);
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
           for (int i = 0; i < 32; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * alpha);
-          x_st32(tl + 2 * LP_K + 32 * c, ov);
+          x_st32(tl_base + 2 * LP_K + 32 * c, ov);
         }
       }
       asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       // before the last product can start, the one before it is seen complete: the final wait below then is for the
       // phase in progress (a parity wait must be neither two phases early nor two late)
-      if (t > 0 && t == ntiles - 1) x_wait(bar_o, (uint32_t)((t - 1) & 1), dead, a.status);
-      mbar_arrive(bar_pfull);
+      if (t > 0 && t == n - 1) x_wait(my_o, (uint32_t)((t - 1) & 1), dead, a.status);
+      mbar_arrive(my_p);
     }
-    x_wait(bar_o, (uint32_t)((ntiles - 1) & 1), dead, a.status);
-    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    const bool store = row < a.s && !*dead;
-    float scale = 0.f;
-    if (store) {
-      const float g = a.y[((size_t)b * a.s + row) * a.ldy + a.off_g + head];
-      scale = (1.0f / l_run) / (1.0f + expf(-g));
-    }
-    __nv_bfloat16* dst = a.z + ((size_t)b * a.s + row) * a.ldz + (size_t)head * a.v;
-#pragma unroll
-    for (int c = 0; c < NV * 2; ++c) {
-      uint32_t ov[32];
-      x_ld32(tl + 2 * LP_K + 32 * c, ov);
-      asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+    if (n > 0) {
+      x_wait(my_o, (uint32_t)((n - 1) & 1), dead, a.status);
+      asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      const bool store = row < a.s && !*dead;
+      float scale = 0.f;
       if (store) {
+        const float gate = a.y[((size_t)b * a.s + row) * a.ldy + a.off_g + head];
+        scale = (1.0f / l_run) / (1.0f + expf(-gate));
+      }
+      __nv_bfloat16* dst = a.z + ((size_t)b * a.s + row) * a.ldz + (size_t)head * a.v;
 #pragma unroll
-        for (int i = 0; i < 4; ++i)  // v is a multiple of 8: whole 16-byte pieces
-          if (32 * c + 8 * i < a.v) {
-            uint32_t w[4];
+      for (int c = 0; c < NV * 2; ++c) {
+        uint32_t ov[32];
+        x_ld32(tl_base + 2 * LP_K + 32 * c, ov);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        if (store) {
 #pragma unroll
-            for (int e = 0; e < 4; ++e)
-              w[e] = lp_pack(__uint_as_float(ov[8 * i + 2 * e]) * scale, __uint_as_float(ov[8 * i + 2 * e + 1]) * scale);
-            *reinterpret_cast<uint4*>(dst + 32 * c + 8 * i) = make_uint4(w[0], w[1], w[2], w[3]);
-          }
+          for (int i = 0; i < 4; ++i)  // v is a multiple of 8: whole 16-byte pieces
+            if (32 * c + 8 * i < a.v) {
+              uint32_t w[4];
+#pragma unroll
+              for (int e = 0; e < 4; ++e)
+                w[e] = lp_pack(__uint_as_float(ov[8 * i + 2 * e]) * scale, __uint_as_float(ov[8 * i + 2 * e + 1]) * scale);
+              *reinterpret_cast<uint4*>(dst + 32 * c + 8 * i) = make_uint4(w[0], w[1], w[2], w[3]);
+            }
+        }
       }
     }
   }
@@ -275,21 +320,22 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "n"(COLS) : "memory");
 }
 
-template <int NV, int KB, int VB>
-int launch_lp(fb200_device* dev, const LpArgs& a, int b, const CUtensorMap& kvmap, const CUtensorMap& cmap, size_t smem) {
-  static size_t configured[64] = {0};
-  if (configured[dev->ordinal & 63] < smem) {
-    FB_CUDA(dev, cudaFuncSetAttribute(latent_prefill_kernel<NV, KB, VB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    configured[dev->ordinal & 63] = smem;
-  }
-  return fb200_launch(dev, latent_prefill_kernel<NV, KB, VB>, dim3((unsigned)((a.s + LP_Q - 1) / LP_Q), (unsigned)a.h, (unsigned)b), dim3(LP_BLOCK),
-                      smem, false, a, kvmap, cmap);
+size_t lp_smem(int nk, int nv, int kb, int vb, int g) {
+  size_t n = (size_t)kb * nk * LP_BOX + (size_t)vb * nv * LP_BOX + (size_t)g * LP_Q * nk * 128 + LP_TAIL + 1024;
+  if (nv > 2 || g > 1) n = std::max(n, (size_t)120 * 1024);  // all 512 TMEM columns: one CTA per SM
+  return n;
 }
 
-size_t lp_smem(int nk, int nv, int kb, int vb) {
-  size_t n = (size_t)kb * nk * LP_BOX + (size_t)vb * nv * LP_BOX + (size_t)LP_Q * nk * 128 + LP_TAIL + 1024;
-  if (nv > 2) n = std::max(n, (size_t)120 * 1024);  // all 512 TMEM columns: one CTA per SM
-  return n;
+template <int NV, int KB, int VB, int G>
+int launch_lp(fb200_device* dev, const LpArgs& a, int b, const CUtensorMap& kvmap, const CUtensorMap& cmap) {
+  const size_t smem = lp_smem(a.nk, NV, KB, VB, G);
+  static size_t configured[64] = {0};
+  if (configured[dev->ordinal & 63] < smem) {
+    FB_CUDA(dev, cudaFuncSetAttribute(latent_prefill_kernel<NV, KB, VB, G>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    configured[dev->ordinal & 63] = smem;
+  }
+  return fb200_launch(dev, latent_prefill_kernel<NV, KB, VB, G>, dim3((unsigned)((a.s + LP_Q * G - 1) / (LP_Q * G)), (unsigned)a.h, (unsigned)b),
+                      dim3(G * LP_THREADS + 64), smem, false, a, kvmap, cmap);
 }
 
 }  // namespace
@@ -297,7 +343,7 @@ size_t lp_smem(int nk, int nv, int kb, int vb) {
 // Shapes the tensor-core path covers: 16-byte aligned columns and a tile that fits shared memory.
 bool fb200_latent_prefill_covers(int h, int d, int r, int v, int rk, float scale) {
   return d % 8 == 0 && v % 8 == 0 && rk % 8 == 0 && d <= 256 && r <= 128 && v <= 256 && h <= 65535 && scale > 0.f &&
-         lp_smem((d + 63) / 64 + (r + 63) / 64, (v + 63) / 64, 2, 1) <= 227 * 1024;
+         lp_smem((d + 63) / 64 + (r + 63) / 64, (v + 63) / 64, 2, 1, 1) <= 227 * 1024;
 }
 
 // The new positions' latents must already be in the cache. a.kvx holds b * keys rows of kv_ld elements.
@@ -323,18 +369,20 @@ int fb200_latent_prefill(fb200_device* dev, const fb200_latent_args& a, const fb
   p.window = a.window; p.pos = a.pos; p.kbase = kbase; p.keys = keys; p.cap = a.cap; p.v_col = a.h * a.d;
   p.scale_log2 = a.scale * 1.4426950408889634f; p.status = dev->status;
   const int nv = (a.v + 63) / 64;
-  // three key and two value tiles where two CTAs still fit an SM (or nothing smaller does), else two and one
-  const bool deep = lp_smem(p.nk, nv, 3, 2) <= 113 * 1024 ||
-                    (lp_smem(p.nk, nv, 2, 1) > 113 * 1024 && lp_smem(p.nk, nv, 3, 2) <= 227 * 1024);
-  const size_t smem = deep ? lp_smem(p.nk, nv, 3, 2) : lp_smem(p.nk, nv, 2, 1);
+  // two groups of rows per CTA once one per CTA would not fit the SMs at a time anyway; three key and two value tiles
+  // where they fit
+  const long ctas = (long)((a.s + LP_Q - 1) / LP_Q) * a.h * a.b;
+  if (nv <= 2 && ctas > dev->sm_count && lp_smem(p.nk, nv, 3, 2, 2) <= 227 * 1024)
+    return nv == 1 ? launch_lp<1, 3, 2, 2>(dev, p, a.b, kvmap, cmap) : launch_lp<2, 3, 2, 2>(dev, p, a.b, kvmap, cmap);
+  const bool deep = lp_smem(p.nk, nv, 3, 2, 1) <= 227 * 1024;
   switch (nv * 2 + (deep ? 1 : 0)) {
-    case 2: return launch_lp<1, 2, 1>(dev, p, a.b, kvmap, cmap, smem);
-    case 3: return launch_lp<1, 3, 2>(dev, p, a.b, kvmap, cmap, smem);
-    case 4: return launch_lp<2, 2, 1>(dev, p, a.b, kvmap, cmap, smem);
-    case 5: return launch_lp<2, 3, 2>(dev, p, a.b, kvmap, cmap, smem);
-    case 6: return launch_lp<3, 2, 1>(dev, p, a.b, kvmap, cmap, smem);
-    case 7: return launch_lp<3, 3, 2>(dev, p, a.b, kvmap, cmap, smem);
-    case 8: return launch_lp<4, 2, 1>(dev, p, a.b, kvmap, cmap, smem);
-    default: return launch_lp<4, 3, 2>(dev, p, a.b, kvmap, cmap, smem);
+    case 2: return launch_lp<1, 2, 1, 1>(dev, p, a.b, kvmap, cmap);
+    case 3: return launch_lp<1, 3, 2, 1>(dev, p, a.b, kvmap, cmap);
+    case 4: return launch_lp<2, 2, 1, 1>(dev, p, a.b, kvmap, cmap);
+    case 5: return launch_lp<2, 3, 2, 1>(dev, p, a.b, kvmap, cmap);
+    case 6: return launch_lp<3, 2, 1, 1>(dev, p, a.b, kvmap, cmap);
+    case 7: return launch_lp<3, 3, 2, 1>(dev, p, a.b, kvmap, cmap);
+    case 8: return launch_lp<4, 2, 1, 1>(dev, p, a.b, kvmap, cmap);
+    default: return launch_lp<4, 3, 2, 1>(dev, p, a.b, kvmap, cmap);
   }
 }

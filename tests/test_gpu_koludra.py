@@ -89,6 +89,15 @@ def test_latent_layer(dev, dtype, shape):
     check(dev, cfg, w, t, dtype, [70, 3, 40, 2, 1])
 
 
+@pytest.mark.parametrize("window,sizes", [(1, [700]), (70, [700]), (200, [650, 50]), (64, [300, 400]), (5000, [257, 443])], ids=str)
+@pytest.mark.parametrize("vdim", [64, 128])
+def test_latent_layer_many_rows(dev, window, sizes, vdim):
+    # enough heads and rows for two groups of rows per CTA in the prompt kernel
+    cfg = U.config([U.latent(ff=0, heads=64, dim=16, rot=16, vdim=vdim, rank=24, window=window)], width=64, vocab=64)
+    w = U.weights(cfg, 40, U.identity_head(cfg))
+    check(dev, cfg, w, toks(cfg, 700), "bfloat16", sizes, max_seq_len=704)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_layers_that_share_latents(dev, dtype):
     # the second reader has another window, other heads and value size; the third reads the first one's latents as well
