@@ -182,6 +182,8 @@ def load_library():
         "fb200_exchange_wait_check": (i32, [vp, i32]),
     }
     for name, (res, args) in sig.items():
+        if LIB_PATH.endswith("_dense.so") and not hasattr(L, name):
+            continue  # a library of the dense part alone (build.build(part="dense"))
         fn = getattr(L, name)
         fn.restype = res
         fn.argtypes = args

@@ -247,8 +247,10 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(const fb200_late
     float v = 0.f;
     if (e < a.rk) {
 #pragma unroll 8
-      for (int s = 0; s < a.nsplit; ++s)
-        if (wt[s] != 0.f) v = fmaf(part[(size_t)s * (a.rk + 2) + e], wt[s], v);  // an empty split left nothing there
+      for (int s = 0; s < a.nsplit; ++s) {
+        const float x = part[(size_t)s * (a.rk + 2) + e], w = wt[s];
+        v = fmaf(w != 0.f ? x : 0.f, w, v);  // an empty split left nothing there
+      }
     }
     lsm[e] = v;
   }

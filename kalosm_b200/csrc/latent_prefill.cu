@@ -101,38 +101,76 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
   }
   // ---- Q: rotary positions, bf16, K-major operand layout: [d, zeros to 64 na | r, zeros]
   if (tid < SOFT) {
-    const int half = a.r / 2;
+    const int half = a.r / 2, nchunks = a.na * 8, rchunks = kchunks - nchunks;
     const bool vec = ((a.d + a.r) & 3) == 0;
-    for (int id = tid; id < G * LP_Q * kchunks; id += SOFT) {
-      const int row = (id & 7) + ((id / (8 * kchunks)) << 3), c = (id >> 3) % kchunks;
-      float x[8];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] = 0.f;
-      if (q0 + row < a.s) {
-        const float* q = a.y + ((size_t)b * a.s + q0 + row) * a.ldy + (size_t)head * (a.d + a.r);
-        if (c < a.na * 8) {
-          if (vec && c * 8 < a.d) {  // d is a multiple of 8
-            const float4 x0 = *reinterpret_cast<const float4*>(q + c * 8), x1 = *reinterpret_cast<const float4*>(q + c * 8 + 4);
-            x[0] = x0.x; x[1] = x0.y; x[2] = x0.z; x[3] = x0.w;
-            x[4] = x1.x; x[5] = x1.y; x[6] = x1.z; x[7] = x1.w;
-          } else {
-#pragma unroll
-            for (int e = 0; e < 8; ++e)
-              if (c * 8 + e < a.d) x[e] = q[c * 8 + e];
-          }
-        } else {
-          const int i0 = (c - a.na * 8) * 8;
-          const float *cs = a.rope_cos + (size_t)(a.pos + q0 + row) * half, *sn = a.rope_sin + (size_t)(a.pos + q0 + row) * half;
-#pragma unroll
-          for (int e = 0; e < 8; ++e) {
-            const int i = i0 + e;
-            if (i < half) x[e] = q[a.d + i] * cs[i] - q[a.d + half + i] * sn[i];
-            else if (i < a.r) x[e] = q[a.d + i] * cs[i - half] + q[a.d + i - half] * sn[i - half];
-          }
-        }
-      }
+    auto put = [&](int row, int c, const float (&x)[8]) {
       *reinterpret_cast<uint4*>(Qs + (row >> 7) * qbytes + x_kmajor(row & 127, c, kchunks)) =
           make_uint4(lp_pack(x[0], x[1]), lp_pack(x[2], x[3]), lp_pack(x[4], x[5]), lp_pack(x[6], x[7]));
+    };
+    auto q_row = [&](int row) { return a.y + ((size_t)b * a.s + q0 + row) * a.ldy + (size_t)head * (a.d + a.r); };
+    // eight threads take one 16-byte column piece of eight rows (one core matrix)
+    if (vec) {
+#pragma unroll 6
+      for (int id = tid; id < G * LP_Q * nchunks; id += SOFT) {
+        const int row = (id & 7) + ((id / (8 * nchunks)) << 3), c = (id >> 3) % nchunks;
+        const bool in = q0 + row < a.s && c * 8 < a.d;  // d is a multiple of 8
+        const float4* q = reinterpret_cast<const float4*>(in ? q_row(row) + c * 8 : a.y);
+        const float4 x0 = q[0], x1 = q[1];
+        const float m = in ? 1.f : 0.f;
+        const float x[8] = {in ? x0.x : m, in ? x0.y : m, in ? x0.z : m, in ? x0.w : m, in ? x1.x : m, in ? x1.y : m, in ? x1.z : m, in ? x1.w : m};
+        put(row, c, x);
+      }
+    } else {
+      for (int id = tid; id < G * LP_Q * nchunks; id += SOFT) {
+        const int row = (id & 7) + ((id / (8 * nchunks)) << 3), c = (id >> 3) % nchunks;
+        float x[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = q0 + row < a.s && c * 8 + e < a.d ? q_row(row)[c * 8 + e] : 0.f;
+        put(row, c, x);
+      }
+    }
+    if (vec && (half & 7) == 0) {  // a thread rotates eight pairs: two pieces
+      const int pchunks = half / 8, zchunks = rchunks - 2 * pchunks;
+#pragma unroll 2
+      for (int id = tid; id < G * LP_Q * pchunks; id += SOFT) {
+        const int row = (id & 7) + ((id / (8 * pchunks)) << 3), c = (id >> 3) % pchunks;
+        const bool in = q0 + row < a.s;
+        const float4* u4 = reinterpret_cast<const float4*>(in ? q_row(row) + a.d + c * 8 : a.y);
+        const float4* v4 = reinterpret_cast<const float4*>(in ? q_row(row) + a.d + half + c * 8 : a.y);
+        const size_t tp = (size_t)(a.pos + (in ? q0 + row : 0)) * half + c * 8;
+        const float4 *c4 = reinterpret_cast<const float4*>(a.rope_cos + tp), *s4 = reinterpret_cast<const float4*>(a.rope_sin + tp);
+        float u[8], v[8], cs[8], sn[8], xu[8], xv[8];
+        *reinterpret_cast<float4*>(u) = u4[0]; *reinterpret_cast<float4*>(u + 4) = u4[1];
+        *reinterpret_cast<float4*>(v) = v4[0]; *reinterpret_cast<float4*>(v + 4) = v4[1];
+        *reinterpret_cast<float4*>(cs) = c4[0]; *reinterpret_cast<float4*>(cs + 4) = c4[1];
+        *reinterpret_cast<float4*>(sn) = s4[0]; *reinterpret_cast<float4*>(sn + 4) = s4[1];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          xu[e] = in ? u[e] * cs[e] - v[e] * sn[e] : 0.f;
+          xv[e] = in ? v[e] * cs[e] + u[e] * sn[e] : 0.f;
+        }
+        put(row, nchunks + c, xu);
+        put(row, nchunks + pchunks + c, xv);
+      }
+      const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      for (int id = tid; id < G * LP_Q * zchunks; id += SOFT)
+        put((id & 7) + ((id / (8 * zchunks)) << 3), nchunks + 2 * pchunks + (id >> 3) % zchunks, zero);
+    } else {
+      for (int id = tid; id < G * LP_Q * rchunks; id += SOFT) {
+        const int row = (id & 7) + ((id / (8 * rchunks)) << 3), c = (id >> 3) % rchunks;
+        float x[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const int i = c * 8 + e;
+          x[e] = 0.f;
+          if (q0 + row >= a.s || i >= a.r) continue;
+          const float* q = q_row(row) + a.d;
+          const size_t tp = (size_t)(a.pos + q0 + row) * half;
+          x[e] = i < half ? q[i] * a.rope_cos[tp + i] - q[half + i] * a.rope_sin[tp + i]
+                          : q[i] * a.rope_cos[tp + i - half] + q[i - half] * a.rope_sin[tp + i - half];
+        }
+        put(row, nchunks + c, x);
+      }
     }
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // these stores -> tensor-core reads
   }
@@ -185,18 +223,26 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
   } else if (warp == SOFT / 32) {
     // ---- MMA issuer: per tile and group, S of the next tile (under the softmax of this one), then O += P V
     if (lane == 0) {
-      const int steps_d = (a.d + 15) / 16, steps_r = (a.r + 15) / 16;
-      const uint32_t q_sbo = (uint32_t)kchunks * 128;
+      uint64_t qdesc[G], kdesc[KB], vdesc[VB];  // a descriptor's low bits hold its address / 16
+#pragma unroll
+      for (int g = 0; g < G; ++g) qdesc[g] = x_desc(smem_u32(Qs) + (uint32_t)(g * qbytes), 128, (uint32_t)kchunks * 128);
+#pragma unroll
+      for (int i = 0; i < KB; ++i) kdesc[i] = x_desc(smem_u32(Ks) + (uint32_t)(i * kbytes), 16, 1024, LP_SW128);
+#pragma unroll
+      for (int i = 0; i < VB; ++i) vdesc[i] = x_desc(smem_u32(Vs) + (uint32_t)(i * NV) * LP_BOX, LP_BOX, 1024, LP_SW128);
       auto issue_s = [&](int g, int u) {
         const int tg = t_first + u - tf[g];
         x_wait(bar_kfull + 8 * (u % KB), (uint32_t)((u / KB) & 1), dead, a.status);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const uint32_t ks = smem_u32(Ks) + (uint32_t)((u % KB) * kbytes), qs = smem_u32(Qs) + (uint32_t)(g * qbytes);
-        for (int i = 0; i < steps_d + steps_r; ++i) {
-          const int s = i < steps_d ? i : a.na * 4 + i - steps_d;  // 16-column step of the padded layout
-          x_mma(tmem + (uint32_t)(g * GCOLS + (tg & 1) * LP_K), x_desc(qs + s * 256, 128, q_sbo),
-                x_desc(ks + (s >> 2) * LP_BOX + (s & 3) * 32, 16, 1024, LP_SW128), IDESC_S, i ? 1u : 0u);
-        }
+        uint64_t qd = qdesc[0], kd = kdesc[0];
+#pragma unroll
+        for (int i = 1; i < G; ++i) qd = g == i ? qdesc[i] : qd;
+#pragma unroll
+        for (int i = 1; i < KB; ++i) kd = u % KB == i ? kdesc[i] : kd;
+        const uint32_t dst = tmem + (uint32_t)(g * GCOLS + (tg & 1) * LP_K);
+        for (int i = 0; i < a.nk; ++i, qd += 4 * 256 / 16, kd += LP_BOX / 16)  // a box is four steps of 16 columns (zero columns of Q where it is wider)
+#pragma unroll
+          for (int s = 0; s < 4; ++s) x_mma(dst, qd + s * (256 / 16), kd + s * (32 / 16), IDESC_S, (i | s) ? 1u : 0u);
         x_commit(bar_s + 16 * g + 8 * (tg & 1));
       };
 #pragma unroll
@@ -212,11 +258,11 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
           x_wait(bar_pfull + 8 * g, (uint32_t)(tg & 1), dead, a.status);
           x_wait(bar_vfull + 8 * (u % VB), (uint32_t)((u / VB) & 1), dead, a.status);
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-          const uint32_t vs = smem_u32(Vs) + (uint32_t)((u % VB) * NV) * LP_BOX, tm = tmem + (uint32_t)(g * GCOLS);
+          const uint32_t tm = tmem + (uint32_t)(g * GCOLS), pa = tm + (uint32_t)((tg & 1) * LP_K);
+          const uint64_t vd = VB > 1 && (u & 1) ? vdesc[VB - 1] : vdesc[0];
 #pragma unroll
           for (int s = 0; s < LP_K / 16; ++s)  // 16 keys = 16 rows of 128 bytes further
-            x_mma_ta(tm + 2 * LP_K, tm + (uint32_t)((tg & 1) * LP_K + s * 8), x_desc(vs + s * 2048, LP_BOX, 1024, LP_SW128), IDESC_O,
-                     (tg | s) ? 1u : 0u);
+            x_mma_ta(tm + 2 * LP_K, pa + (uint32_t)(s * 8), vd + s * (2048 / 16), IDESC_O, (tg | s) ? 1u : 0u);
           x_commit(bar_o + 8 * g);
         }
       }

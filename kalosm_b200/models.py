@@ -15,6 +15,10 @@ def _gguf_llama(device, path, max_seq_len=None, max_batch=1, dtype=None):
 REGISTRY = {"llama": _gguf_llama, koludra.ARCHITECTURE: koludra.load}
 
 
+# architectures that the dense part of the library serves (build.build(part="dense"))
+DENSE = (koludra.ARCHITECTURE,)
+
+
 def architecture(path):
     """The architecture name of a checkpoint: a folder with config.json, or a GGUF file."""
     if os.path.isdir(path):

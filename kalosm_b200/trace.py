@@ -61,9 +61,10 @@ def main(argv=None):
     ap.add_argument("--out", required=True, help="folder for the logits")
     ap.add_argument("--max-tokens", type=int, default=4096, help="most tokens a live request holds")
     args = ap.parse_args(argv)
-    from . import Device, build
-    build.build()
-    from . import models
+    import kalosm_b200
+    from . import Device, build, models
+    if "FB200_LIB_PATH" not in os.environ:  # compile what this model needs, if it is not there
+        kalosm_b200.LIB_PATH = build.build(part="dense" if models.architecture(args.model) in models.DENSE else "all")
     model = models.load_model(Device(0), args.model, max_seq_len=max(args.max_tokens, 16), dtype=args.dtype)
 
     def emit(text):
