@@ -613,7 +613,7 @@ int launch_prep(fb200_device* dev, const fb200_delta_args& a) {
 }  // namespace
 
 int fb200_delta_dp(int d) {
-  for (int dp : {32, 64, 128, 256, 512, 1024})
+  for (int dp : {32, 64, 128, 256, 512})
     if (d <= dp) return dp;
   return 0;
 }
@@ -625,7 +625,6 @@ int fb200_delta_step(fb200_device* dev, const fb200_delta_args& a) {
     case 128: return launch_step<32, 4>(dev, a);
     case 256: return launch_step<32, 8>(dev, a);
     case 512: return launch_step<32, 16>(dev, a);
-    case 1024: return launch_step<32, 32>(dev, a);
     default: return fb200_fail(dev, FB200_ERR_INVALID_SHAPE, "delta rule: head size %d", a.d);
   }
 }
@@ -638,7 +637,6 @@ int fb200_delta_prompt(fb200_device* dev, const fb200_delta_args& a) {
     case 128: rc = launch_prep<4>(dev, a); break;
     case 256: rc = launch_prep<8>(dev, a); break;
     case 512: rc = launch_prep<16>(dev, a); break;
-    case 1024: rc = launch_prep<32>(dev, a); break;
     default: return fb200_fail(dev, FB200_ERR_INVALID_SHAPE, "delta rule: head size %d", a.d);
   }
   if (rc) return rc;
@@ -647,8 +645,7 @@ int fb200_delta_prompt(fb200_device* dev, const fb200_delta_args& a) {
     case 64: rc = launch_scan<4, 16, 16>(dev, a); break;
     case 128: rc = launch_scan<4, 32, 16>(dev, a); break;
     case 256: rc = launch_scan<8, 32, 16>(dev, a); break;
-    case 512: rc = launch_scan<16, 32, 8>(dev, a); break;
-    default: rc = launch_scan<32, 32, 4>(dev, a); break;
+    default: rc = launch_scan<16, 32, 8>(dev, a); break;
   }
   if (rc) return rc;
   const size_t warps = (size_t)a.b * a.s * a.h;
