@@ -149,8 +149,8 @@ __global__ void __launch_bounds__(ST_MAX_THREADS) delta_step_kernel(const fb200_
     vpast = conv_past(a, b, a.off_v + h * a.v + c0, pos);
     vw = a.conv_w[(size_t)(a.taps - 1) * a.channels + a.off_v + h * a.v + c0];
   }
-  pdl_launch_dependents();
   pdl_wait();
+  pdl_launch_dependents();
   const float* yr = a.y + (size_t)b * a.ldy;
   float v0 = 0.f;
   if (p == 0 && c0 < a.v) v0 = dr_silu(fmaf(vw, yr[a.off_v + h * a.v + c0], vpast));
@@ -357,7 +357,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prep_kernel(const fb200
   }
 }
 
-constexpr int SC_WARPS = 8, CPT = 4;  // columns per group of lanes
+constexpr int SC_WARPS = 4, CPT = 4;  // columns per group of lanes
 
 // A group of LPC lanes owns CPT columns of S: k and q read from shared memory serve all of them, and the sums are
 // reduced so that lane p ends up with those of column p % 4, so one pass over the four tokens does all columns.
@@ -643,7 +643,11 @@ int fb200_delta_prompt(fb200_device* dev, const fb200_delta_args& a) {
   switch (a.dp) {
     case 32: rc = launch_scan<4, 8, 16>(dev, a); break;
     case 64: rc = launch_scan<4, 16, 16>(dev, a); break;
-    case 128: rc = launch_scan<4, 32, 16>(dev, a); break;
+    case 128:
+      // 16 lanes per column group do less per token (fewer shuffles); 32 lanes make more CTAs where there are few heads
+      if ((a.v + 15) / 16 * a.h * a.b <= dev->sm_count) rc = launch_scan<4, 32, 16>(dev, a);
+      else rc = launch_scan<8, 16, 16>(dev, a);
+      break;
     case 256: rc = launch_scan<8, 32, 16>(dev, a); break;
     default: rc = launch_scan<16, 32, 8>(dev, a); break;
   }

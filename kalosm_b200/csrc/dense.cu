@@ -93,12 +93,11 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
   if (first < a.units) {
     int r0, r1;
     rows_of(first, r0, r1);
-    for (int p = p0 + lane * 8; p < min(p1, p0 + 256 * 4); p += 256) {
+    for (int p = p0 + lane * 8; p < min(p1, p0 + 128); p += 256) {
       asm volatile("prefetch.global.L2 [%0];" ::"l"(w + (size_t)r0 * pieces + p));
       asm volatile("prefetch.global.L2 [%0];" ::"l"(w + (size_t)r1 * pieces + p));
     }
   }
-  pdl_launch_dependents();
   pdl_wait();
   // ---- the activation row: (RMS-normalised) f32, zero padding beyond kx
   float scale = 1.f;
@@ -130,6 +129,8 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
 
   const int rounds = (a.units + stride - 1) / stride;
   for (int it = 0; it < rounds; ++it) {
+    // two CTAs fill an SM's registers: the next kernel is let in only when the last round has begun
+    if (it == rounds - 1) pdl_launch_dependents();
     const int u = first + it * stride;
     float s0 = 0.f, s1 = 0.f;
     if (u < a.units) {

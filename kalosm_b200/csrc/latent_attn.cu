@@ -48,8 +48,8 @@ __global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(const fb200_la
   extern __shared__ __align__(16) float lsm[];  // query head [d + r], or partial sums [LQ_THREADS][E]
   __shared__ float red[LQ_THREADS / 32];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y, b = row / a.s;
-  pdl_launch_dependents();
   pdl_wait();
+  pdl_launch_dependents();
   const int pos = *a.pos_dev + row % a.s;
   const float* yr = a.y + (size_t)row * a.ldy;
   const int half = a.r / 2;
@@ -128,8 +128,8 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attn_kernel(const fb200_
   extern __shared__ __align__(16) float lsm[];  // [LA_WARPS][rk]
   __shared__ float wm[LA_WARPS], wl[LA_WARPS];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, row = blockIdx.z, b = row / a.s;
-  pdl_launch_dependents();
   pdl_wait();
+  pdl_launch_dependents();
   const int pos = *a.pos_dev + row % a.s, n = a.rk + a.r;
   const int lo = a.window ? max(0, pos - a.window + 1) : 0, keys = pos + 1 - lo;
   const int per = (keys + a.nsplit - 1) / a.nsplit, k0 = lo + min(keys, (int)blockIdx.x * per), k1 = min(pos + 1, k0 + per);
@@ -224,8 +224,8 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(const fb200_late
       pre[i][k] = make_uint4(0u, 0u, 0u, 0u);
       if (v0 + i < a.v && lane + 32 * k < np) pre[i][k] = *reinterpret_cast<const uint4*>(w + (size_t)(v0 + i) * a.rkp + (lane + 32 * k) * E);
     }
-  pdl_launch_dependents();
   pdl_wait();
+  pdl_launch_dependents();
   const float* part = a.part + ((size_t)row * a.h + h) * a.nsplit * (a.rk + 2);
   float* wt = lsm + a.rkp;
   if (warp == 0) {  // weights of the splits, normalised
@@ -243,16 +243,33 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(const fb200_late
   }
   const float gate = 1.0f / (1.0f + expf(-a.y[(size_t)row * a.ldy + a.off_g + h]));
   __syncthreads();
-  for (int e = tid; e < a.rkp; e += LO_THREADS) {
-    float v = 0.f;
-    if (e < a.rk) {
-#pragma unroll 8
-      for (int s = 0; s < a.nsplit; ++s) {
-        const float x = part[(size_t)s * (a.rk + 2) + e], w = wt[s];
-        v = fmaf(w != 0.f ? x : 0.f, w, v);  // an empty split left nothing there
+  // merged read-out; an empty split (weight 0) left nothing behind
+  if ((a.rk & 1) == 0) {
+    for (int e = 2 * tid; e < a.rkp; e += 2 * LO_THREADS) {
+      float2 v = make_float2(0.f, 0.f);
+      if (e < a.rk) {
+#pragma unroll 16
+        for (int s = 0; s < a.nsplit; ++s) {
+          const float2 x = *reinterpret_cast<const float2*>(part + (size_t)s * (a.rk + 2) + e);
+          const float w = wt[s];
+          v.x = fmaf(w != 0.f ? x.x : 0.f, w, v.x);
+          v.y = fmaf(w != 0.f ? x.y : 0.f, w, v.y);
+        }
       }
+      *reinterpret_cast<float2*>(lsm + e) = v;
     }
-    lsm[e] = v;
+  } else {
+    for (int e = tid; e < a.rkp; e += LO_THREADS) {
+      float v = 0.f;
+      if (e < a.rk) {
+#pragma unroll 8
+        for (int s = 0; s < a.nsplit; ++s) {
+          const float x = part[(size_t)s * (a.rk + 2) + e], w = wt[s];
+          v = fmaf(w != 0.f ? x : 0.f, w, v);
+        }
+      }
+      lsm[e] = v;
+    }
   }
   __syncthreads();
 #pragma unroll
@@ -316,8 +333,8 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attn_mma_kernel(const fb200
     }
   };
   if (k0 < k1) fetch(k0, true);
-  pdl_launch_dependents();
   pdl_wait();
+  pdl_launch_dependents();
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   float o[NT][4];
 #pragma unroll
