@@ -699,7 +699,7 @@ def hybrid_work(layers, width, vocab, rows, ctx, n_sm):
             add("delta_out_kernel", "hbm", 10.0 * rows * H * V)
         elif rows == 1:
             add("latent_query_kernel", "hbm", 2.0 * H * mx["dim"] * mx["kv_rank"])
-            add("latent_attn_kernel", "hbm", 2.0 * min(mx["mask"]["size"], ctx + 1) * (mx["kv_rank"] + mx["rot_dim"]))
+            add("latent_attn_mma_kernel", "hbm", 2.0 * min(mx["mask"]["size"], ctx + 1) * (mx["kv_rank"] + mx["rot_dim"]))
             add("latent_out_kernel", "hbm", 2.0 * H * V * mx["kv_rank"])
         else:
             win = mx["mask"]["size"]

@@ -244,24 +244,29 @@ constexpr uint32_t PAIR_J = 0u | 0u << 2 | 1u << 4 | 0u << 6 | 1u << 8 | 2u << 1
 constexpr uint32_t PAIR_I = 1u | 2u << 2 | 2u << 4 | 3u << 6 | 3u << 8 | 3u << 10 | 0u << 12 | 1u << 14 | 1u << 16 | 2u << 18 | 2u << 20 |
                             2u << 22 | 3u << 24 | 3u << 26 | 3u << 28 | 3u << 30;
 
-// convolution + SiLU of channel c for the CH tokens from t0 (zeros from token s on)
+// convolution + SiLU of channel c for the CH tokens from t0 (zeros from token s on); inputs before this pass come
+// from the ring. Addresses are selected, not branched on, so that a channel's loads go out together.
 __device__ __forceinline__ void conv_chunk(const fb200_delta_args& a, int b, int c, int t0, int pos, float (&out)[CH]) {
 #pragma unroll
   for (int i = 0; i < CH; ++i) out[i] = 0.f;
-  if (t0 >= a.taps - 1 && t0 + CH <= a.s) {  // every input is a row of this pass
-    const float* y = a.y + ((size_t)b * a.s + t0 - (a.taps - 1)) * a.ldy + c;
-    for (int j = 0; j < a.taps; ++j) {
-      const float w = a.conv_w[(size_t)j * a.channels + c];
+  for (int j0 = 0; j0 < a.taps; j0 += 4) {  // four taps at a time meet seven inputs
+    float w[4], x[CH + 3];
 #pragma unroll
-      for (int i = 0; i < CH; ++i) out[i] = fmaf(w, y[(size_t)(i + j) * a.ldy], out[i]);
+    for (int j = 0; j < 4; ++j) w[j] = j0 + j < a.taps ? a.conv_w[(size_t)(j0 + j) * a.channels + c] : 0.f;
+#pragma unroll
+    for (int r = 0; r < CH + 3; ++r) {
+      const int t = t0 - (a.taps - 1) + j0 + r, p = pos + t;
+      const bool valid = j0 + r < a.taps + CH - 1 && t < a.s && p >= 0;
+      const float* src = t >= 0 ? a.y + ((size_t)b * a.s + t) * a.ldy + c : a.ring + ((size_t)b * a.taps + (valid ? p % a.taps : 0)) * a.channels + c;
+      x[r] = valid ? *src : 0.f;
     }
 #pragma unroll
-    for (int i = 0; i < CH; ++i) out[i] = dr_silu(out[i]);
-  } else {
+    for (int j = 0; j < 4; ++j)
 #pragma unroll
-    for (int i = 0; i < CH; ++i)
-      if (t0 + i < a.s) out[i] = conv_silu(a, b, c, t0 + i, pos);
+      for (int i = 0; i < CH; ++i) out[i] = fmaf(w[j], x[i + j], out[i]);
   }
+#pragma unroll
+  for (int i = 0; i < CH; ++i) out[i] = t0 + i < a.s ? dr_silu(out[i]) : 0.f;
 }
 
 // Sums v[0..31] over the lanes of a warp; lane l returns the total of v[l].
@@ -335,15 +340,18 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) delta_prep_kernel(const fb200
   }
   unit -= a.hk;
   if (unit < vblocks) {
+    float v[PREP_VCH / 32][CH];
 #pragma unroll
     for (int e = 0; e < PREP_VCH / 32; ++e) {
       const int c = unit * PREP_VCH + lane + 32 * e;
-      if (c >= hv) continue;
-      float v[CH];
-      conv_chunk(a, b, a.off_v + c, t0, pos, v);
+      if (c < hv) conv_chunk(a, b, a.off_v + c, t0, pos, v[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < PREP_VCH / 32; ++e) {
+      const int c = unit * PREP_VCH + lane + 32 * e;
 #pragma unroll
       for (int i = 0; i < CH; ++i)
-        if (i < n) a.vn[((size_t)b * a.s + t0 + i) * hv + c] = v[i];
+        if (c < hv && i < n) a.vn[((size_t)b * a.s + t0 + i) * hv + c] = v[e][i];
     }
     return;
   }

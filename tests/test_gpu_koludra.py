@@ -187,6 +187,15 @@ def test_batch_equals_each_sequence_alone(dev, dtype):
         assert U.err(got[i], want[i]) < U.TOL[dtype], i
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_odd_sizes(dev, dtype):
+    cfg = U.config([U.delta(heads=3, kv_heads=1, dim=9, vdim=7, conv=7, ff=37), U.latent(heads=3, dim=7, rot=2, vdim=5, rank=11, window=9, ff=0),
+                    U.latent(heads=1, dim=5, rot=2, vdim=3, rank=11, window=31, kv_from=1, ff=13)], width=75, vocab=53)
+    w = U.weights(cfg, 23)
+    for sizes in ([90], [40, 2, 31, 1]):
+        check(dev, cfg, w, toks(cfg, 90), dtype, sizes)
+
+
 def test_larger_sizes(dev):
     # sizes of the kernels that real layers use: 128-wide heads, 512-wide latents, many weight tiles
     cfg = U.config([U.delta(heads=8, kv_heads=4, dim=128, vdim=128, conv=4, ff=1024),
