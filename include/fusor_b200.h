@@ -305,7 +305,11 @@ typedef enum fb200_llama_tensor {
   FB200_T_MIX_Q = 12, FB200_T_MIX_K = 13, FB200_T_MIX_V = 14, FB200_T_MIX_GATE = 15, FB200_T_MIX_OUT = 16,
   FB200_T_MIX_BETA = 17, FB200_T_MIX_DECAY = 18, FB200_T_MIX_Q_CONV = 19, FB200_T_MIX_K_CONV = 20,
   FB200_T_MIX_V_CONV = 21, FB200_T_MIX_A_LOG = 22, FB200_T_MIX_DT_BIAS = 23, FB200_T_MIX_OUT_NORM = 24,
-  FB200_T_MIX_DKV = 25, FB200_T_MIX_DKV_NORM = 26, FB200_T_MIX_UK = 27, FB200_T_MIX_UV = 28
+  FB200_T_MIX_DKV = 25, FB200_T_MIX_DKV_NORM = 26, FB200_T_MIX_UK = 27, FB200_T_MIX_UV = 28,
+  FB200_T_MIX_Q_NORM = 29, FB200_T_MIX_K_NORM = 30, FB200_T_MIX_SINK = 31, FB200_T_MIX_Q_BIAS = 32,
+  FB200_T_MIX_K_BIAS = 33, FB200_T_MIX_V_BIAS = 34,
+  FB200_T_MIX_HEAD_DECAY = 35, /* f32, one constant per head */
+  FB200_T_LOOP_IN = 36         /* model level: [hidden, 2 hidden] */
 } fb200_llama_tensor;
 
 FB200_API int fb200_llama_create(fb200_device* dev, const fb200_llama_config* cfg, fb200_llama** out);
@@ -323,26 +327,55 @@ FB200_API int fb200_llama_free(fb200_llama* m);
  *                     x dim^-1/2); per head S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q with
  *                     g = exp(-exp(A_log) softplus(decay + dt_bias)), beta = sigmoid(beta projection);
  *                     o is RMS-normalised over vdim, x FB200_T_MIX_OUT_NORM, x silu(gate).
+ *   FB200_MIX_ATTENTION  softmax attention with grouped key/value heads (query head n reads key/value head
+ *                     n / (heads / kv_heads)). `parts` (FB200_ATTN_*) names what a layer has: biases of q, k and v; an
+ *                     RMSNorm per q and k head; a sink per head (one more term exp(sink) of the softmax's
+ *                     denominator); head n's output x sigmoid(gate_n). rot_dim > 0: rotate-half positions on the first
+ *                     rot_dim of every q and k head, with YaRN scaling where yarn_factor > 0. Scores x scale, then
+ *                     softcap tanh(score / softcap) where softcap > 0, over the last `window` positions (0: all).
+ *   FB200_MIX_LINEAR  linear attention with a fixed decay per head: q, k (heads x dim), v (heads x vdim) through SiLU;
+ *                     S <- decay S + k v^T, o = S^T q; the heads' outputs RMS-normalised together x
+ *                     FB200_T_MIX_OUT_NORM [heads vdim], x sigmoid(gate), a gate per element.
  *   FB200_MIX_LATENT  latent attention: FB200_T_MIX_DKV gives kv_rank latent rows (RMS-normalised) and rot_dim
  *                     rows of a key part shared by the heads (rotated); key n = [uk_n c, key part], value n =
  *                     uv_n c; rotate-half positions on the last rot_dim of every query head; scores
  *                     x scale over the last `window` positions (0: all); head n x sigmoid(gate_n).
  *                     kv_from >= 0: the layer reads the cache of that earlier latent layer (same kv_rank,
  *                     rot_dim and rotation) and has no FB200_T_MIX_DKV of its own.
+ * Variants of a layer: `two_norms` gives the feed-forward a norm of its own (FB200_T_FFN_NORM) of the same x;
+ * ffn_act FB200_FFN_GELU is down(gelu(up h)), gelu in its tanh form, without a gate; an entry with `beside` = 1 is
+ * not a layer but one more mixer of the layer in front of it, reading the same norm. A mixer's output counts
+ * out_scale times. Tensors are set by entry; norms and the feed-forward belong to a layer's first entry.
  * Recurrent states cannot be rewound: fb200_llama_truncate accepts 0 and the current length. */
-typedef enum fb200_mixer_kind { FB200_MIX_DELTA = 1, FB200_MIX_LATENT = 2 } fb200_mixer_kind;
+typedef enum fb200_mixer_kind { FB200_MIX_DELTA = 1, FB200_MIX_LATENT = 2, FB200_MIX_ATTENTION = 3, FB200_MIX_LINEAR = 4 } fb200_mixer_kind;
 typedef enum fb200_compute { FB200_COMPUTE_BF16 = 0, FB200_COMPUTE_F32 = 1 } fb200_compute;
+typedef enum fb200_ffn_act { FB200_FFN_SWIGLU = 0, FB200_FFN_GELU = 1 } fb200_ffn_act;
+typedef enum fb200_attn_parts { FB200_ATTN_QK_NORM = 1, FB200_ATTN_BIAS = 2, FB200_ATTN_SINK = 4, FB200_ATTN_GATE = 8 } fb200_attn_parts;
 typedef struct fb200_layer_config {
   int mixer;                                   /* fb200_mixer_kind */
   int ffn;                                     /* width of the feed-forward, 0: none */
-  int heads, kv_heads, dim, vdim;              /* kv_heads: delta rule only */
+  int heads, kv_heads, dim, vdim;              /* kv_heads: delta rule and softmax attention */
   int conv;                                    /* delta rule: taps of the short convolution */
   int kv_rank, rot_dim, window, kv_from;       /* latent attention; kv_from -1: a cache of its own */
   float rope_base, scale;
+  int beside, two_norms, ffn_act;
+  float out_scale;
+  int parts;                                   /* softmax attention: fb200_attn_parts */
+  float softcap, yarn_factor, yarn_fast, yarn_slow;
+  int yarn_original;
 } fb200_layer_config;
-/* cfg: n_layer, hidden, vocab, max_seq_len, max_batch and rms_eps are read; layers[n_layer]. */
-FB200_API int fb200_llama_create_layers(fb200_device* dev, const fb200_llama_config* cfg,
-                                        const fb200_layer_config* layers, int compute, fb200_llama** out);
+/* Around the layers: x = embed_scale * embedding; x <- x + residual_mult * (..) in every layer; logits
+ * through logit_softcap tanh(. / logit_softcap) where that is > 0. loop_times > 0: the layers loop_start ..
+ * loop_stop - 1 (counted without `beside` entries) run loop_times times in a row, each pass with caches and states of
+ * its own, and before the first layer of each pass x <- FB200_T_LOOP_IN [x; embedded x]. */
+typedef struct fb200_stack_config {
+  float embed_scale, residual_mult, logit_softcap;
+  int loop_start, loop_stop, loop_times;
+} fb200_stack_config;
+/* cfg: n_layer (entries), hidden, vocab, max_seq_len, max_batch and rms_eps are read; layers[n_layer]; stack may be
+ * NULL (factors of 1, no softcap, no loop). */
+FB200_API int fb200_llama_create_layers(fb200_device* dev, const fb200_llama_config* cfg, const fb200_layer_config* layers,
+                                        const fb200_stack_config* stack, int compute, fb200_llama** out);
 /* Tensor names of raw/mod.rs:473-646: blk.{i}.attn_q.weight ... ; norms are f32 vectors
  * (ggml_type FB200_F32), everything else raw GGUF blocks of shape [N, K]. `layer` is ignored
  * for the three model-level tensors. Missing FB200_T_OUTPUT ties it to the embedding

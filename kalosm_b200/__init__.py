@@ -73,13 +73,27 @@ class LlamaConfig(C.Structure):
 
 
 class LayerConfig(C.Structure):
-    """fb200_layer_config: one token-mixer layer (fb200_llama_create_layers)."""
+    """fb200_layer_config: one token-mixer layer, or a mixer beside the one before it (fb200_llama_create_layers)."""
     _fields_ = [("mixer", C.c_int), ("ffn", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int),
                 ("vdim", C.c_int), ("conv", C.c_int), ("kv_rank", C.c_int), ("rot_dim", C.c_int), ("window", C.c_int),
-                ("kv_from", C.c_int), ("rope_base", C.c_float), ("scale", C.c_float)]
+                ("kv_from", C.c_int), ("rope_base", C.c_float), ("scale", C.c_float), ("beside", C.c_int),
+                ("two_norms", C.c_int), ("ffn_act", C.c_int), ("out_scale", C.c_float), ("parts", C.c_int),
+                ("softcap", C.c_float), ("yarn_factor", C.c_float), ("yarn_fast", C.c_float), ("yarn_slow", C.c_float),
+                ("yarn_original", C.c_int)]
 
 
-MIX_DELTA, MIX_LATENT = 1, 2
+class StackConfig(C.Structure):
+    """fb200_stack_config: what stands around the layers (factors, logit softcap, a loop over some of them)."""
+    _fields_ = [("embed_scale", C.c_float), ("residual_mult", C.c_float), ("logit_softcap", C.c_float),
+                ("loop_start", C.c_int), ("loop_stop", C.c_int), ("loop_times", C.c_int)]
+
+    def __init__(self, embed_scale=1.0, residual_mult=1.0, logit_softcap=0.0, loop_start=0, loop_stop=0, loop_times=0):
+        super().__init__(embed_scale, residual_mult, logit_softcap, loop_start, loop_stop, loop_times)
+
+
+MIX_DELTA, MIX_LATENT, MIX_ATTENTION, MIX_LINEAR = 1, 2, 3, 4
+FFN_SWIGLU, FFN_GELU = 0, 1
+ATTN_QK_NORM, ATTN_BIAS, ATTN_SINK, ATTN_GATE = 1, 2, 4, 8
 COMPUTE = {"bfloat16": 0, "float32": 1}
 
 
@@ -171,7 +185,7 @@ def load_library():
         "fb200_llama_generate_greedy": (i32, [vp, vp, i32, i32, vp]),
         "fb200_llama_logits_dev": (i32, [vp, pp]),
         "fb200_llama_set_tensor_parallel": (i32, [vp, vp]),
-        "fb200_llama_create_layers": (i32, [vp, C.POINTER(LlamaConfig), C.POINTER(LayerConfig), i32, pp]),
+        "fb200_llama_create_layers": (i32, [vp, C.POINTER(LlamaConfig), C.POINTER(LayerConfig), C.POINTER(StackConfig), i32, pp]),
         "fb200_llama_logits_at": (i32, [vp, vp, i32, vp]),
         "fb200_comm_unique_id": (i32, [vp, sz]),
         "fb200_comm_create": (i32, [vp, i32, i32, vp, sz, pp]),
@@ -607,7 +621,9 @@ class Decoder:
                "ffn_norm": 10, "output_norm": 11,
                "mix_q": 12, "mix_k": 13, "mix_v": 14, "mix_gate": 15, "mix_out": 16, "mix_beta": 17, "mix_decay": 18,
                "mix_q_conv": 19, "mix_k_conv": 20, "mix_v_conv": 21, "mix_a_log": 22, "mix_dt_bias": 23,
-               "mix_out_norm": 24, "mix_dkv": 25, "mix_dkv_norm": 26, "mix_uk": 27, "mix_uv": 28}
+               "mix_out_norm": 24, "mix_dkv": 25, "mix_dkv_norm": 26, "mix_uk": 27, "mix_uv": 28, "mix_q_norm": 29,
+               "mix_k_norm": 30, "mix_sink": 31, "mix_q_bias": 32, "mix_k_bias": 33, "mix_v_bias": 34, "mix_head_decay": 35,
+               "loop_in": 36}
     h = None
 
     def set_tensor(self, name: str, layer: int, ggml_type: int, shape, raw) -> None:
@@ -712,12 +728,14 @@ class Llama(Decoder):
 
 class HybridDecoder(Decoder):
     """A decoder of token-mixer layers over dense weights (fb200_llama_create_layers). `layers` is a list of
-    keyword dictionaries with the fields of LayerConfig; `compute` is "bfloat16" or "float32"."""
+    keyword dictionaries with the fields of LayerConfig, `stack` one with those of StackConfig; `compute` is "bfloat16" or
+    "float32"."""
 
-    def __init__(self, device: Device, *, hidden, vocab, layers, max_seq_len, max_batch=1, rms_eps=1e-5, compute="bfloat16"):
+    def __init__(self, device: Device, *, hidden, vocab, layers, max_seq_len, max_batch=1, rms_eps=1e-5, compute="bfloat16", stack=None):
         self.device, self.comm, self.vocab = device, None, vocab
         self.cfg = LlamaConfig(n_layer=len(layers), hidden=hidden, vocab=vocab, max_seq_len=max_seq_len, max_batch=max_batch, rms_eps=rms_eps)
-        self.layers = (LayerConfig * len(layers))(*[LayerConfig(**dict({"kv_from": -1}, **kw)) for kw in layers])
+        self.layers = (LayerConfig * len(layers))(*[LayerConfig(**dict({"kv_from": -1, "out_scale": 1.0}, **kw)) for kw in layers])
         out = C.c_void_p()
-        device._check(device.lib.fb200_llama_create_layers(device.h, C.byref(self.cfg), self.layers, COMPUTE[compute], C.byref(out)))
+        device._check(device.lib.fb200_llama_create_layers(device.h, C.byref(self.cfg), self.layers, C.byref(StackConfig(**(stack or {}))),
+                                                       COMPUTE[compute], C.byref(out)))
         self.h = out.value

@@ -81,7 +81,7 @@ struct fb200_llama {
 // Session buffers common to all architectures (llama.cu); the model's dev and cfg are set.
 int fb200_decoder_session(fb200_llama* m);
 
-// Token-mixer layers (hybrid.cu). A forward pass takes the embedded rows in m->x and leaves logits and greedy ids.
+// Token-mixer layers (hybrid.cu). A forward pass takes the ids in m->ids and leaves logits and greedy ids.
 int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows);
 int fb200_hybrid_finalize(fb200_llama* m);
 int fb200_hybrid_forward(fb200_llama* m, int batch, int seq, bool commit);

@@ -39,11 +39,13 @@ struct GemvArgs {
   const void* w;
   const float* x;
   const float* norm_w;
+  const float* ff_norm_w;
   const float* add;
+  const float* bias;
   float* y;
   float* z;
-  int k, kx, row0, n_plain, gate0, up0, ff, ks, units;
-  float eps;
+  int k, kx, row0, n_plain, gate0, up0, ff, act, ks, units;
+  float eps, alpha, softcap;
 };
 
 __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
@@ -66,12 +68,20 @@ __device__ __forceinline__ void gv_fma(const uint4& u, const float4& x0, const f
   acc = fmaf(__uint_as_float(u.w), x0.w, acc);
 }
 
+// value of a plain output row
+__device__ __forceinline__ float plain_value(float acc, float alpha, const float* bias, const float* add, float softcap, int n) {
+  float v = alpha * acc;
+  if (bias) v += bias[n];
+  if (add) v += add[n];
+  return softcap > 0.f ? softcap * tanhf(v / softcap) : v;
+}
+
 // The activation row is kept as float4 planes: plane p holds elements 4 p .. 4 p + 3 of every 16-byte piece of a
 // weight row (two planes for bf16 weights, one for f32), so that consecutive lanes read consecutive float4.
 template <typename WT>
 __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArgs a) {
   constexpr int E = 16 / (int)sizeof(WT), P = E / 4;  // elements and float4 planes per piece
-  extern __shared__ __align__(16) float4 xs[];        // [P][k / E]
+  extern __shared__ __align__(16) float4 xs[];        // [P][k / E], twice where the feed-forward rows have their own norm
   __shared__ float red[2 * GV_WARPS];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int pieces = a.k / E;
@@ -82,6 +92,9 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
     if (u < plain_units) {
       r0 = a.row0 + 2 * u;
       r1 = 2 * u + 1 < a.n_plain ? r0 + 1 : r0;
+    } else if (a.act == FB200_FFN_GELU) {
+      r0 = a.up0 + 2 * (u - plain_units);
+      r1 = 2 * (u - plain_units) + 1 < a.ff ? r0 + 1 : r0;
     } else {
       r0 = a.gate0 + u - plain_units;
       r1 = a.up0 + u - plain_units;
@@ -117,13 +130,15 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
     __syncthreads();
   }
   for (int i = tid; i < a.k; i += GV_THREADS) {
-    float v = 0.f;
+    float v = 0.f, v2 = 0.f;
     if (i < a.kx) {
       v = __ldcg(a.x + i);
+      if (a.ff_norm_w) v2 = (v / scale) * a.ff_norm_w[i];
       if (a.norm_w) v = (v / scale) * a.norm_w[i];
     }
-    const int piece = i / E, e = i % E;
-    reinterpret_cast<float*>(xs)[((e >> 2) * pieces + piece) * 4 + (e & 3)] = v;
+    const int piece = i / E, e = i % E, at = ((e >> 2) * pieces + piece) * 4 + (e & 3);
+    reinterpret_cast<float*>(xs)[at] = v;
+    if (a.ff_norm_w) reinterpret_cast<float*>(xs + P * pieces)[at] = v2;
   }
   __syncthreads();
 
@@ -138,6 +153,7 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
       rows_of(u, r0, r1);
       const uint4* w0 = w + (size_t)r0 * pieces;
       const uint4* w1 = w + (size_t)r1 * pieces;
+      const float4* xu = a.ff_norm_w && u >= plain_units ? xs + P * pieces : xs;
       int p = p0 + lane;
       for (; p + 96 < p1; p += 128) {
         uint4 b0[4], b1[4];
@@ -145,14 +161,14 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
         for (int i = 0; i < 4; ++i) { b0[i] = __ldcs(w0 + p + 32 * i); b1[i] = __ldcs(w1 + p + 32 * i); }
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          const float4 x0 = xs[p + 32 * i], x1 = P > 1 ? xs[(P - 1) * pieces + p + 32 * i] : x0;
+          const float4 x0 = xu[p + 32 * i], x1 = P > 1 ? xu[(P - 1) * pieces + p + 32 * i] : x0;
           gv_fma(b0[i], x0, x1, s0, WT());
           gv_fma(b1[i], x0, x1, s1, WT());
         }
       }
       for (; p < p1; p += 32) {
         const uint4 b0 = __ldcs(w0 + p), b1 = __ldcs(w1 + p);
-        const float4 x0 = xs[p], x1 = P > 1 ? xs[(P - 1) * pieces + p] : x0;
+        const float4 x0 = xu[p], x1 = P > 1 ? xu[(P - 1) * pieces + p] : x0;
         gv_fma(b0, x0, x1, s0, WT());
         gv_fma(b1, x0, x1, s1, WT());
       }
@@ -174,8 +190,12 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
     if (u < a.units && part == 0 && lane == 0) {
       if (u < plain_units) {
         const int n = 2 * u;
-        a.y[n] = a.add ? s0 + a.add[n] : s0;
-        if (n + 1 < a.n_plain) a.y[n + 1] = a.add ? s1 + a.add[n + 1] : s1;
+        a.y[n] = plain_value(s0, a.alpha, a.bias, a.add, a.softcap, n);
+        if (n + 1 < a.n_plain) a.y[n + 1] = plain_value(s1, a.alpha, a.bias, a.add, a.softcap, n + 1);
+      } else if (a.act == FB200_FFN_GELU) {
+        const int n = 2 * (u - plain_units);
+        a.z[n] = fb_gelu_tanh(s0);
+        if (n + 1 < a.ff) a.z[n + 1] = fb_gelu_tanh(s1);
       } else {
         a.z[u - plain_units] = silu_f(s0) * s1;
       }
@@ -190,19 +210,22 @@ struct GemmF32Args {
   const float* w;
   const float* x;
   const float* add;
+  const float* bias;
   float* y;
   float* z;
-  size_t ldx, ldy, ldadd, ldz;
-  int m, k, kx, wrows, row0, n_plain, gate0, up0, ff, plain_tiles;
+  size_t ldx, ldy, ldadd, ldz, ff_off;
+  int m, k, kx, row0, n_plain, gate0, up0, ff, act, plain_tiles;
+  float alpha, softcap;
 };
 
 __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const GemmF32Args a) {
   __shared__ float ws[2][GF_K][GF_T + 4], xs[GF_K][GF_T + 4];
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;  // 4 output rows at tx * 4, 4 activation rows at ty * 4
-  const bool pair = (int)blockIdx.x >= a.plain_tiles;
-  const int nt = pair ? (int)blockIdx.x - a.plain_tiles : (int)blockIdx.x;
-  const int r0 = (pair ? a.gate0 : a.row0) + nt * GF_T, r1 = a.up0 + nt * GF_T;
-  const int lim = pair ? a.ff - nt * GF_T : a.n_plain - nt * GF_T;  // rows of this tile that exist
+  const bool ffn = (int)blockIdx.x >= a.plain_tiles, gelu = a.act == FB200_FFN_GELU, pair = ffn && !gelu;
+  const int nt = ffn ? (int)blockIdx.x - a.plain_tiles : (int)blockIdx.x;
+  const int r0 = (ffn ? gelu ? a.up0 : a.gate0 : a.row0) + nt * GF_T, r1 = a.up0 + nt * GF_T;
+  const int lim = ffn ? a.ff - nt * GF_T : a.n_plain - nt * GF_T;  // rows of this tile that exist
+  const float* x = ffn ? a.x + a.ff_off : a.x;
   const int m0 = (int)blockIdx.y * GF_T;
   float acc[2][4][4];
 #pragma unroll
@@ -217,7 +240,7 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const GemmF32Args a
       const bool kin = k0 + c < a.kx;
       ws[0][c][r] = kin && r < lim ? a.w[(size_t)(r0 + r) * a.k + k0 + c] : 0.f;
       if (pair) ws[1][c][r] = kin && r < lim ? a.w[(size_t)(r1 + r) * a.k + k0 + c] : 0.f;
-      xs[c][r] = kin && m0 + r < a.m ? a.x[(size_t)(m0 + r) * a.ldx + k0 + c] : 0.f;
+      xs[c][r] = kin && m0 + r < a.m ? x[(size_t)(m0 + r) * a.ldx + k0 + c] : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -250,19 +273,20 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const GemmF32Args a
     for (int i = 0; i < 4; ++i) {
       const int r = tx * 4 + i, n = nt * GF_T + r;
       if (r >= lim) continue;
-      if (pair) a.z[(size_t)m * a.ldz + n] = silu_f(acc[0][i][q]) * acc[1][i][q];
-      else a.y[(size_t)m * a.ldy + n] = a.add ? acc[0][i][q] + a.add[(size_t)m * a.ldadd + n] : acc[0][i][q];
+      if (ffn) a.z[(size_t)m * a.ldz + n] = gelu ? fb_gelu_tanh(acc[0][i][q]) : silu_f(acc[0][i][q]) * acc[1][i][q];
+      else a.y[(size_t)m * a.ldy + n] = plain_value(acc[0][i][q], a.alpha, a.bias, a.add ? a.add + (size_t)m * a.ldadd : nullptr, a.softcap, n);
     }
   }
 }
 
 // f32 rows -> (normalised) bf16 rows with zero padding, one CTA per row
 __global__ void __launch_bounds__(256)
-rows_to_bf16_kernel(const float* __restrict__ x, size_t ldx, const int* __restrict__ index, const float* __restrict__ w, float eps,
+rows_to_bf16_kernel(const float* __restrict__ x, size_t ldx, const float* __restrict__ w, const float* __restrict__ w2, float eps,
                     int n, int np, __nv_bfloat16* __restrict__ y) {
   __shared__ float sh[8];
   const size_t row = blockIdx.x;
-  const float* xr = x + (index ? (size_t)index[row] : row) * ldx;
+  const float* xr = x + row * ldx;
+  y += row * (w2 ? 2 : 1) * (size_t)np;
   float rms = 1.f;
   if (w) {
     float ss = 0.f;
@@ -276,17 +300,18 @@ rows_to_bf16_kernel(const float* __restrict__ x, size_t ldx, const int* __restri
     rms = sqrtf(ss / (float)n + eps);
   }
   for (int i = threadIdx.x; i < np; i += 256) {
-    const float v = i < n ? (w ? (xr[i] / rms) * w[i] : xr[i]) : 0.f;
-    y[row * np + i] = __float2bfloat16(v);
+    const float u = i < n ? xr[i] / rms : 0.f;
+    y[i] = __float2bfloat16(w && i < n ? u * w[i] : u);
+    if (w2) y[np + i] = __float2bfloat16(i < n ? u * w2[i] : 0.f);
   }
 }
 
 }  // namespace
 
-int fb200_rows_to_bf16(fb200_device* dev, const float* x, size_t ldx, const int* index, const float* w, float eps, size_t rows,
+int fb200_rows_to_bf16(fb200_device* dev, const float* x, size_t ldx, const float* w, const float* w2, float eps, size_t rows,
                        int n, int np, __nv_bfloat16* y) {
   if (rows == 0) return FB200_OK;
-  rows_to_bf16_kernel<<<(unsigned)rows, 256, 0, dev->stream>>>(x, ldx, index, w, eps, n, np, y);
+  rows_to_bf16_kernel<<<(unsigned)rows, 256, 0, dev->stream>>>(x, ldx, w, w2, eps, n, np, y);
   FB_LAUNCH_CHECK(dev);
   return FB200_OK;
 }
@@ -296,12 +321,24 @@ int fb200_dense_gemv(fb200_device* dev, const fb200_dense_job& j) {
   const int e = bf ? 8 : 4;
   if (j.m != 1 || j.y_bf16 || j.w->k % e || j.w->k * 4 > 200 * 1024)
     return fb200_fail(dev, FB200_ERR_INVALID_SHAPE, "dense product: one row of %llu columns is not covered", (unsigned long long)j.w->k);
+  if (j.ff && j.n_plain && (j.ff_off || (j.ff_norm_w && j.w->k * 8 > 200 * 1024))) {  // the two groups one after the other
+    fb200_dense_job p = j, f = j;
+    p.ff = 0;
+    f.n_plain = 0;
+    f.x = (const float*)j.x + j.ff_off;
+    f.norm_w = j.ff_norm_w ? j.ff_norm_w : j.norm_w;
+    p.ff_norm_w = f.ff_norm_w = nullptr;
+    p.ff_off = f.ff_off = 0;
+    const int rc = fb200_dense_gemv(dev, p);
+    return rc ? rc : fb200_dense_gemv(dev, f);
+  }
   GemvArgs a = {};
-  a.w = j.w->data; a.x = (const float*)j.x; a.norm_w = j.norm_w; a.add = j.add; a.y = (float*)j.y; a.z = (float*)j.z;
+  a.w = j.w->data; a.x = (const float*)j.x; a.norm_w = j.norm_w; a.ff_norm_w = j.ff ? j.ff_norm_w : nullptr; a.add = j.add; a.bias = j.bias;
+  a.y = (float*)j.y; a.z = (float*)j.z; a.alpha = j.alpha; a.softcap = j.softcap; a.act = j.act;
   a.k = (int)j.w->k; a.kx = j.kx; a.row0 = j.row0; a.n_plain = j.n_plain; a.gate0 = j.gate0; a.up0 = j.up0; a.ff = j.ff; a.eps = j.eps;
-  a.units = (j.n_plain + 1) / 2 + j.ff;
+  a.units = (j.n_plain + 1) / 2 + (j.act == FB200_FFN_GELU ? (j.ff + 1) / 2 : j.ff);
   if (a.units == 0) return FB200_OK;
-  const size_t smem = (size_t)j.w->k * 4;
+  const size_t smem = (size_t)j.w->k * (a.ff_norm_w ? 8 : 4);
   const int per_sm = smem <= 100 * 1024 ? 2 : 1;
   const int ctas = dev->sm_count * per_sm;
   // warps per unit: the split of K that leaves the fewest warps idle in the last round (ties: the smaller split)
@@ -328,7 +365,8 @@ int fb200_dense_gemm_f32(fb200_device* dev, const fb200_dense_job& j) {
   if (j.w->type != FB200_F32 || j.norm_w || j.y_bf16)
     return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "dense product: f32 rows need F32 weights");
   GemmF32Args a = {};
-  a.w = (const float*)j.w->data; a.x = (const float*)j.x; a.add = j.add; a.y = (float*)j.y; a.z = (float*)j.z;
+  a.w = (const float*)j.w->data; a.x = (const float*)j.x; a.add = j.add; a.bias = j.bias; a.y = (float*)j.y; a.z = (float*)j.z;
+  a.alpha = j.alpha; a.softcap = j.softcap; a.act = j.act; a.ff_off = j.ff_off;
   a.ldx = j.ldx; a.ldy = j.ldy; a.ldadd = j.ldadd; a.ldz = j.ldz;
   a.m = j.m; a.k = (int)j.w->k; a.kx = j.kx; a.row0 = j.row0; a.n_plain = j.n_plain; a.gate0 = j.gate0; a.up0 = j.up0; a.ff = j.ff;
   a.plain_tiles = (j.n_plain + GF_T - 1) / GF_T;

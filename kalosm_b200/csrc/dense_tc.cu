@@ -8,8 +8,8 @@
 //    outside the matrices arrive as zeros;
 //  * MMA issuer (one thread): 4 NH tcgen05.mma (M = 128, N = BM, K = 16, kind::f16 with bf16 operands and fp32
 //    accumulation) per stage, tcgen05.commit hands the stage back;
-//  * epilogue (8 warps): tcgen05.ld, then f32 or bf16 rows (+ a residual), or SwiGLU: gate and up rows of an
-//    output are the two halves of the same CTA, so they sit in the same TMEM lane BM columns apart.
+//  * epilogue (8 warps): tcgen05.ld, then f32 or bf16 rows (factor, bias, residual, softcap), gelu rows, or SwiGLU:
+//    gate and up rows of an output are the two halves of the same CTA, so they sit in the same TMEM lane BM columns apart.
 // Every wait is bounded (2^22 polls): a wait that gives up sets the device status word and a flag that makes the
 // other roles leave; TMEM is released on every path.
 #include <algorithm>
@@ -39,9 +39,11 @@ struct DenseTcArgs {
   float* y;
   __nv_bfloat16* yb;
   const float* add;
+  const float* bias;
   __nv_bfloat16* z;
   size_t ldy, ldadd, ldz;
-  int m, kblocks, row0, n_plain, gate0, up0, ff, plain_tiles, m_tiles;
+  int m, kblocks, row0, n_plain, gate0, up0, ff, gelu, ff_col, plain_tiles, m_tiles;
+  float alpha, softcap;
   int* status;
 };
 
@@ -62,8 +64,8 @@ dense_tc_kernel(const DenseTcArgs a, const __grid_constant__ CUtensorMap wmap, c
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   // activation tiles fastest: the CTAs that run together share their weight rows in L2
   const int mt = (int)blockIdx.x % a.m_tiles, nt = (int)blockIdx.x / a.m_tiles;
-  const bool pair = nt >= a.plain_tiles;
-  const int n0 = pair ? (nt - a.plain_tiles) * TC_BN : nt * TC_BN * NH;  // first output row of the tile
+  const bool ffn = nt >= a.plain_tiles, pair = ffn && !a.gelu;
+  const int n0 = ffn ? (nt - a.plain_tiles) * TC_BN * (pair ? 1 : NH) : nt * TC_BN * NH;  // first output row of the tile
   const int m0 = mt * BM;
   if (tid == 0) {
     *dead = 0;
@@ -82,7 +84,7 @@ dense_tc_kernel(const DenseTcArgs a, const __grid_constant__ CUtensorMap wmap, c
 
   if (warp == TC_EPI_WARPS) {
     if (lane == 0) {
-      const int r0 = pair ? a.gate0 + n0 : a.row0 + n0, r1 = pair ? a.up0 + n0 : r0 + TC_BN;
+      const int r0 = (pair ? a.gate0 : ffn ? a.up0 : a.row0) + n0, r1 = pair ? a.up0 + n0 : r0 + TC_BN, xc = ffn ? a.ff_col : 0;
       int issued = 0;
       for (int kb = 0; kb < a.kblocks; ++kb, ++issued) {
         const int s = kb % S::STAGES;
@@ -91,7 +93,7 @@ dense_tc_kernel(const DenseTcArgs a, const __grid_constant__ CUtensorMap wmap, c
         mbar_expect_tx(bar, S::STAGE);
         x_tma_box2(dst, &wmap, kb * TC_BK, r0, bar);
         if (NH == 2) x_tma_box2(dst + TC_BN * TC_BK * 2, &wmap, kb * TC_BK, r1, bar);
-        x_tma_box2(dst + S::A_BYTES, &xmap, kb * TC_BK, m0, bar);
+        x_tma_box2(dst + S::A_BYTES, &xmap, xc + kb * TC_BK, m0, bar);
       }
       if (*dead)
         for (int kb = max(0, issued - S::STAGES); kb < issued; ++kb) x_drain(full + 8 * (kb % S::STAGES), (uint32_t)((kb / S::STAGES) & 1));
@@ -146,8 +148,25 @@ dense_tc_kernel(const DenseTcArgs a, const __grid_constant__ CUtensorMap wmap, c
 #pragma unroll
           for (int h = 0; h < NH; ++h) {
             const int n = n0 + h * TC_BN + r;
-            if (n >= a.n_plain) continue;
-            const uint32_t (&v)[16] = h ? v1 : v0;
+            if (n >= (ffn ? a.ff : a.n_plain)) continue;
+            uint32_t (&v)[16] = h ? v1 : v0;
+            if (ffn) {
+              __nv_bfloat16* zp = a.z + (size_t)(m0 + c) * a.ldz + n;
+#pragma unroll
+              for (int i = 0; i < 16; ++i)
+                if (i < lim) {
+                  const float t = __uint_as_float(v[i]), u = 0.7978845608028654f * fmaf(0.044715f * t * t, t, t);
+                  zp[(size_t)i * a.ldz] = __float2bfloat16(__fdividef(t, 1.0f + __expf(-2.0f * u)));
+                }
+              continue;
+            }
+            const float bias = a.bias ? a.bias[n] : 0.f;
+#pragma unroll
+            for (int i = 0; i < 16; ++i) v[i] = __float_as_uint(fmaf(a.alpha, __uint_as_float(v[i]), bias));
+            if (a.softcap > 0.f) {  // of a product without a residual
+#pragma unroll
+              for (int i = 0; i < 16; ++i) v[i] = __float_as_uint(a.softcap * tanhf(__uint_as_float(v[i]) / a.softcap));
+            }
             if (a.yb) {
               __nv_bfloat16* yp = a.yb + (size_t)(m0 + c) * a.ldy + n;
 #pragma unroll
@@ -183,18 +202,24 @@ typedef CUresult (*encode_fn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, voi
                               const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                               CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
+// feed-forward tiles: a gated pair takes both halves of a tile
+int tc_ff_tiles(const fb200_dense_job& j, int nh) {
+  const int rows = j.act == FB200_FFN_GELU ? TC_BN * nh : TC_BN;
+  return (j.ff + rows - 1) / rows;
+}
+
 template <int BM, int NH>
 int launch_tc(fb200_device* dev, const fb200_dense_job& j, DenseTcArgs a) {
   using S = TcShape<BM, NH>;
   static_assert(S::STAGES >= 2, "at least two stages");
   CUtensorMap wmap, xmap;
   if (!fb200_make_map_2d(&wmap, j.w->data, 1, j.w->k, j.w->n, j.w->k * 2, TC_BN) ||
-      !fb200_make_map_2d(&xmap, j.x, 1, (uint64_t)j.kx, (uint64_t)j.m, j.ldx * 2, BM))
+      !fb200_make_map_2d(&xmap, j.x, 1, (uint64_t)(j.ff_off + j.kx), (uint64_t)j.m, j.ldx * 2, BM))
     return fb200_fail(dev, FB200_ERR_CUDA, "dense product: tensor map refused (w %llu x %llu, x %d x %d stride %zu)",
                       (unsigned long long)j.w->n, (unsigned long long)j.w->k, j.m, j.kx, j.ldx);
   a.plain_tiles = (j.n_plain + TC_BN * NH - 1) / (TC_BN * NH);
   a.m_tiles = (j.m + BM - 1) / BM;
-  const int tiles = a.plain_tiles + (NH == 2 ? (j.ff + TC_BN - 1) / TC_BN : 0);
+  const int tiles = a.plain_tiles + tc_ff_tiles(j, NH);
   if (tiles == 0) return FB200_OK;
   static bool configured[64] = {false};
   if (!configured[dev->ordinal & 63]) {
@@ -225,18 +250,20 @@ bool fb200_make_map_2d(CUtensorMap_st* map, const void* base, int bf16, uint64_t
 }
 
 int fb200_dense_gemm_tc(fb200_device* dev, const fb200_dense_job& j) {
-  if (j.w->type != FB200_BF16 || j.norm_w || j.w->k % 8 || j.ldx % 8 || ((uintptr_t)j.x & 15u))
+  if (j.w->type != FB200_BF16 || j.norm_w || j.w->k % 8 || j.ldx % 8 || ((uintptr_t)j.x & 15u) || j.ff_off % 8 ||
+      (j.ff_off && j.ff_off + (size_t)j.kx > j.ldx))
     return fb200_fail(dev, FB200_ERR_INVALID_ARGUMENT, "dense product: bf16 rows and BF16 weights of an aligned width needed");
   DenseTcArgs a = {};
   if (j.y_bf16) a.yb = (__nv_bfloat16*)j.y;
   else a.y = (float*)j.y;
   a.add = j.add; a.z = (__nv_bfloat16*)j.z; a.ldy = j.ldy; a.ldadd = j.ldadd; a.ldz = j.ldz;
+  a.bias = j.bias; a.alpha = j.alpha; a.softcap = j.softcap; a.gelu = j.act == FB200_FFN_GELU; a.ff_col = (int)j.ff_off;
   a.m = j.m; a.kblocks = (j.kx + TC_BK - 1) / TC_BK; a.row0 = j.row0; a.n_plain = j.n_plain; a.gate0 = j.gate0; a.up0 = j.up0; a.ff = j.ff;
   a.status = dev->status;
   // tile shape by a small cost model: rounds of CTAs over the SMs x time of one tile (relative to 256 x 256)
   auto cost = [&](int bm, int nh, double tile) {
-    if (nh == 1 && j.ff) return 1e30;
-    const long tiles = (long)((j.n_plain + TC_BN * nh - 1) / (TC_BN * nh) + (nh == 2 ? (j.ff + TC_BN - 1) / TC_BN : 0)) * ((j.m + bm - 1) / bm);
+    if (nh == 1 && j.ff && j.act != FB200_FFN_GELU) return 1e30;
+    const long tiles = (long)((j.n_plain + TC_BN * nh - 1) / (TC_BN * nh) + tc_ff_tiles(j, nh)) * ((j.m + bm - 1) / bm);
     const int slots = dev->sm_count * (bm <= 64 ? 2 : 1);
     const long full = tiles / slots, rest = tiles % slots;
     // two small tiles on one SM share it: a last round that half fills the slots takes half a round's time

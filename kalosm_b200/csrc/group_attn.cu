@@ -1,0 +1,335 @@
+// Grouped softmax attention, row by row: per-head norms, rotary positions, softcap, sliding window, sinks, head gates.
+//
+//  * attn_prep_kernel (prompts): a warp per head of a row normalises and rotates it; queries go to a scratch buffer, keys
+//    and values into the cache.
+//  * attn_rows_kernel: one CTA per (split of the visible keys, up to NQ query heads of one key/value head, row). A
+//    group of LPK lanes reads a cached key and value in 16-byte pieces and serves all NQ heads with them; every group keeps a running
+//    softmax of its own, merged at the end over lanes, warps and (by the CTA that arrives last) splits. f32 arithmetic,
+//    bf16 or f32 cache. A step of one position per sequence prepares its heads here too: one kernel. Bound: HBM on the
+//    cache. Prompts run it for F32 models, short passes and head sizes above those of the tensor-core kernel (latent_prefill.cu).
+#include <algorithm>
+
+#include "mixers.cuh"
+#include "qgemv_common.cuh"
+
+namespace {
+
+constexpr int GA_WARPS = 4, GA_THREADS = GA_WARPS * 32, GA_MIN_KEYS = 64, GA_MAX_SPLITS = 32;
+
+__device__ __forceinline__ float ga_warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+  return v;
+}
+__device__ __forceinline__ void ga_unpack(const uint4& u, float (&f)[8], __nv_bfloat16) {
+  f[0] = __uint_as_float(u.x << 16); f[1] = __uint_as_float(u.x & 0xFFFF0000u);
+  f[2] = __uint_as_float(u.y << 16); f[3] = __uint_as_float(u.y & 0xFFFF0000u);
+  f[4] = __uint_as_float(u.z << 16); f[5] = __uint_as_float(u.z & 0xFFFF0000u);
+  f[6] = __uint_as_float(u.w << 16); f[7] = __uint_as_float(u.w & 0xFFFF0000u);
+}
+__device__ __forceinline__ void ga_unpack(const uint4& u, float (&f)[4], float) {
+  f[0] = __uint_as_float(u.x); f[1] = __uint_as_float(u.y); f[2] = __uint_as_float(u.z); f[3] = __uint_as_float(u.w);
+}
+__device__ __forceinline__ void ga_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void ga_store(float* p, float v) { *p = v; }
+
+// A warp writes one head of n elements: normalised under w (null: not), its first r dimensions rotated (cs, sn: this
+// position's row of the tables), x mul; zeros up to np.
+template <typename T>
+__device__ __forceinline__ void ga_head(const float* x, int n, int np, const float* w, float eps, const float* cs, const float* sn, int r,
+                                        float mul, T* dst) {
+  const int lane = threadIdx.x & 31, half = r >> 1;
+  float rms = 1.f;
+  if (w) {
+    float ss = 0.f;
+    for (int i = lane; i < n; i += 32) ss = fmaf(x[i], x[i], ss);
+    rms = sqrtf(ga_warp_sum(ss) / (float)n + eps);
+  }
+  auto value = [&](int i) { return w ? (x[i] / rms) * w[i] : x[i]; };
+  for (int i = lane; i < half; i += 32) {
+    const float u = value(i), v = value(i + half);
+    ga_store(dst + i, (u * cs[i] - v * sn[i]) * mul);
+    ga_store(dst + half + i, (v * cs[i] + u * sn[i]) * mul);
+  }
+  for (int i = r + lane; i < np; i += 32) ga_store(dst + i, i < n ? value(i) * mul : 0.f);
+}
+
+template <typename T, typename QT>
+__global__ void __launch_bounds__(256) attn_prep_kernel(const fb200_attn_args a) {
+  const int slots = a.h + 2 * a.g;
+  const size_t id = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5), total = (size_t)a.b * a.s * slots;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (id >= total) return;
+  const size_t row = id / slots;
+  const int slot = (int)(id % slots), b = (int)(row / a.s), pos = *a.pos_dev + (int)(row % a.s), half = a.r >> 1;
+  const float* y = a.y + row * a.ldy;
+  const float *cs = a.rope_cos + (size_t)pos * half, *sn = a.rope_sin + (size_t)pos * half;
+  T* cache = reinterpret_cast<T*>(a.cache) + ((size_t)b * a.cap + pos) * a.ldc;
+  if (slot < a.h) {
+    ga_head(y + (size_t)slot * a.d, a.d, a.dp, a.q_norm, a.eps, cs, sn, a.r, 1.f, reinterpret_cast<QT*>(a.qn) + (row * a.h + slot) * a.dp);
+  } else if (slot < a.h + a.g) {
+    const int k = slot - a.h;
+    ga_head(y + a.off_k + (size_t)k * a.d, a.d, a.dp, a.k_norm, a.eps, cs, sn, a.r, 1.f, cache + k * a.dp);
+  } else {
+    const int k = slot - a.h - a.g;
+    ga_head(y + a.off_v + (size_t)k * a.v, a.v, a.vp, nullptr, 0.f, cs, sn, 0, 1.f, cache + a.g * a.dp + k * a.vp);
+  }
+}
+
+// T: element type of the cache; a piece is 16 bytes, E elements; LPK lanes take NP pieces each of a key and of a value.
+template <typename T, int NP, int NQ>
+__global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_args a, int nsplit) {
+  constexpr int E = 16 / (int)sizeof(T), LPK = 64 / E, KS = 32 / LPK, U = 2;  // U: keys per lane group in flight
+  constexpr int STEP = GA_WARPS * KS * U;
+  extern __shared__ __align__(16) float gsm[];  // queries [NQ][dp], later outputs [GA_WARPS][NQ][vp]
+  __shared__ float wm[GA_WARPS][NQ], wl[GA_WARPS][NQ], wt[NQ][GA_MAX_SPLITS], tot[NQ];
+  __shared__ int last;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, slot = lane / LPK, p = lane % LPK;
+  const int split = (int)(blockIdx.x % nsplit), gq = a.h / a.g, hgroups = (gq + NQ - 1) / NQ, kvh = blockIdx.y / hgroups;
+  const size_t row = blockIdx.x / nsplit;
+  const int b = (int)(row / a.s), h0 = kvh * gq + ((int)blockIdx.y % hgroups) * NQ, nq = min(NQ, (kvh + 1) * gq - h0);
+  const int pos = *a.pos_dev + (int)(row % a.s);
+  const int lo = a.window ? max(0, pos - a.window + 1) : 0, keys = pos + 1 - lo;
+  const int per = max(GA_MIN_KEYS, (keys + nsplit - 1) / nsplit), active = (keys + per - 1) / per;
+  if (split >= active) return;
+  const int k0 = lo + split * per, k1 = min(pos + 1, k0 + per);
+  T* cache = reinterpret_cast<T*>(a.cache) + (size_t)b * a.cap * a.ldc;
+  const T *kc = cache + kvh * a.dp, *vc = cache + a.g * a.dp + kvh * a.vp;
+  if (a.s == 1) {  // cached rows do not depend on the kernel in front: request the first ones
+    const int k = k0 + warp * KS * U + slot;
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (k + u * KS < min(k1, pos)) {
+        if (p * 128 < a.dp * (int)sizeof(T)) asm volatile("prefetch.global.L2 [%0];" ::"l"(kc + (size_t)(k + u * KS) * a.ldc + p * (128 / (int)sizeof(T))));
+        if (p * 128 < a.vp * (int)sizeof(T)) asm volatile("prefetch.global.L2 [%0];" ::"l"(vc + (size_t)(k + u * KS) * a.ldc + p * (128 / (int)sizeof(T))));
+      }
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  if (a.s == 1) {  // this position's queries, and its key and value where this split holds it
+    const float* y = a.y + row * a.ldy;
+    const int half = a.r >> 1;
+    const float *cs = a.rope_cos + (size_t)pos * half, *sn = a.rope_sin + (size_t)pos * half;
+    for (int job = warp; job < nq + (k1 == pos + 1 ? 2 : 0); job += GA_WARPS) {
+      T* dst = cache + (size_t)pos * a.ldc;
+      if (job < nq) ga_head(y + (size_t)(h0 + job) * a.d, a.d, a.dp, a.q_norm, a.eps, cs, sn, a.r, a.scale, gsm + job * a.dp);
+      else if (job == nq) ga_head(y + a.off_k + (size_t)kvh * a.d, a.d, a.dp, a.k_norm, a.eps, cs, sn, a.r, 1.f, dst + kvh * a.dp);
+      else ga_head(y + a.off_v + (size_t)kvh * a.v, a.v, a.vp, nullptr, 0.f, cs, sn, 0, 1.f, dst + a.g * a.dp + kvh * a.vp);
+    }
+  } else {
+    const float* q = reinterpret_cast<const float*>(a.qn) + (row * a.h + h0) * a.dp;
+    for (int i = tid; i < nq * a.dp; i += GA_THREADS) gsm[i] = q[i] * a.scale;
+  }
+  __syncthreads();
+  float q[NQ][NP * E], acc[NQ][NP * E], m[NQ], l[NQ];
+#pragma unroll
+  for (int n = 0; n < NQ; ++n) {
+    m[n] = -INFINITY;
+    l[n] = 0.f;
+#pragma unroll
+    for (int i = 0; i < NP; ++i)
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int at = (i * LPK + p) * E + e;
+        q[n][i * E + e] = n < nq && at < a.dp ? gsm[n * a.dp + at] : 0.f;
+        acc[n][i * E + e] = 0.f;
+      }
+  }
+  __syncthreads();  // the outputs take the queries' place
+  for (int kt = k0 + warp * KS * U; kt < k1; kt += STEP) {
+    uint4 kr[U][NP], vr[U][NP];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const size_t key = min(kt + u * KS + slot, k1 - 1);
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        const int at = (i * LPK + p) * E;
+        kr[u][i] = at < a.dp ? *reinterpret_cast<const uint4*>(kc + key * a.ldc + at) : make_uint4(0u, 0u, 0u, 0u);
+        vr[u][i] = at < a.vp ? *reinterpret_cast<const uint4*>(vc + key * a.ldc + at) : make_uint4(0u, 0u, 0u, 0u);
+      }
+    }
+    float s[U][NQ];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+#pragma unroll
+      for (int n = 0; n < NQ; ++n) s[u][n] = 0.f;
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        float f[E];
+        ga_unpack(kr[u][i], f, T());
+#pragma unroll
+        for (int n = 0; n < NQ; ++n)
+#pragma unroll
+          for (int e = 0; e < E; ++e) s[u][n] = fmaf(f[e], q[n][i * E + e], s[u][n]);
+      }
+#pragma unroll
+      for (int n = 0; n < NQ; ++n) {
+#pragma unroll
+        for (int o = LPK / 2; o > 0; o >>= 1) s[u][n] += __shfl_xor_sync(0xFFFFFFFFu, s[u][n], o);
+        if (a.softcap > 0.f) s[u][n] = a.softcap * tanhf(s[u][n] / a.softcap);
+        if (kt + u * KS + slot >= k1) s[u][n] = -INFINITY;
+      }
+    }
+    float pr[U][NQ];
+#pragma unroll
+    for (int n = 0; n < NQ; ++n) {
+      float mx = m[n];
+#pragma unroll
+      for (int u = 0; u < U; ++u) mx = fmaxf(mx, s[u][n]);
+      const float base = mx == -INFINITY ? 0.f : mx, alpha = expf(m[n] - base);
+      m[n] = mx;
+      l[n] *= alpha;
+#pragma unroll
+      for (int i = 0; i < NP * E; ++i) acc[n][i] *= alpha;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        pr[u][n] = expf(s[u][n] - base);
+        l[n] += pr[u][n];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        float f[E];
+        ga_unpack(vr[u][i], f, T());
+#pragma unroll
+        for (int n = 0; n < NQ; ++n)
+#pragma unroll
+          for (int e = 0; e < E; ++e) acc[n][i * E + e] = fmaf(pr[u][n], f[e], acc[n][i * E + e]);
+      }
+  }
+  // ---- over the lane groups of a warp, then over the warps
+#pragma unroll
+  for (int n = 0; n < NQ; ++n) {
+    float mx = m[n];
+#pragma unroll
+    for (int o = LPK; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, o));
+    const float w = m[n] == -INFINITY ? 0.f : expf(m[n] - mx);
+    float lt = l[n] * w;
+#pragma unroll
+    for (int o = LPK; o < 32; o <<= 1) lt += __shfl_xor_sync(0xFFFFFFFFu, lt, o);
+    if (lane == 0) { wm[warp][n] = mx; wl[warp][n] = lt; }
+#pragma unroll
+    for (int i = 0; i < NP; ++i)
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        float v = acc[n][i * E + e] * w;
+#pragma unroll
+        for (int o = LPK; o < 32; o <<= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+        const int at = (i * LPK + p) * E + e;
+        if (slot == 0 && at < a.vp) gsm[(warp * NQ + n) * a.vp + at] = v;
+      }
+  }
+  __syncthreads();
+  const float* y = a.y + row * a.ldy;
+  auto put = [&](int n, int c, float v) {  // v: the output with weights of sum 1
+    if (a.off_g >= 0) v *= 1.0f / (1.0f + expf(-y[a.off_g + h0 + n]));
+    v *= a.out_scale;
+    const size_t zi = row * a.ldz + (size_t)(h0 + n) * a.v + c;
+    if (a.z_bf16) reinterpret_cast<__nv_bfloat16*>(a.z)[zi] = __float2bfloat16(v);
+    else reinterpret_cast<float*>(a.z)[zi] = v;
+  };
+  float* part = a.part + ((row * a.h + h0) * (size_t)nsplit) * (a.v + 2);  // [head][split][v + 2]
+  for (int i = tid; i < nq * a.v; i += GA_THREADS) {
+    const int n = i / a.v, c = i % a.v;
+    float mx = -INFINITY, v = 0.f, lt = 0.f;
+#pragma unroll
+    for (int w = 0; w < GA_WARPS; ++w) mx = fmaxf(mx, wm[w][n]);
+#pragma unroll
+    for (int w = 0; w < GA_WARPS; ++w) {
+      const float f = wm[w][n] == -INFINITY ? 0.f : expf(wm[w][n] - mx);
+      v = fmaf(gsm[(w * NQ + n) * a.vp + c], f, v);
+      lt = fmaf(wl[w][n], f, lt);
+    }
+    if (active == 1) {
+      if (a.sink) lt += expf(a.sink[h0 + n] - mx);
+      put(n, c, v / lt);
+    } else {
+      float* out = part + ((size_t)n * nsplit + split) * (a.v + 2);
+      out[c] = v;
+      if (c == 0) { out[a.v] = mx; out[a.v + 1] = lt; }
+    }
+  }
+  if (active == 1) return;
+  // ---- the last split of these heads merges all of them
+  __threadfence();
+  __syncthreads();
+  int* done = a.done + row * gridDim.y + blockIdx.y;
+  if (tid == 0) last = atomicAdd(done, 1) == active - 1;
+  __syncthreads();
+  if (!last) return;
+  __threadfence();
+  if (tid == 0) *done = 0;
+  for (int n = warp; n < nq; n += GA_WARPS) {
+    const float* src = part + ((size_t)n * nsplit + lane) * (a.v + 2) + a.v;
+    const float ms = lane < active ? __ldcg(src) : -INFINITY, ls = lane < active ? __ldcg(src + 1) : 0.f;
+    float mx = ms;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, o));
+    const float w = lane < active ? expf(ms - mx) : 0.f;
+    float lt = ga_warp_sum(ls * w);
+    wt[n][lane] = w;
+    if (lane == 0) tot[n] = a.sink ? lt + expf(a.sink[h0 + n] - mx) : lt;
+  }
+  __syncthreads();
+  for (int i = tid; i < nq * a.v; i += GA_THREADS) {
+    const int n = i / a.v, c = i % a.v;
+    float v = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < active; ++s) v = fmaf(__ldcg(part + ((size_t)n * nsplit + s) * (a.v + 2) + c), wt[n][s], v);
+    put(n, c, v / tot[n]);
+  }
+}
+
+// query heads per CTA: as many as the registers hold, no more than a group has
+int ga_heads(int np, int gq) { return std::min(np <= 2 ? 4 : np <= 4 ? 2 : 1, gq >= 3 ? 4 : gq); }
+
+template <typename T, int NP, int NQ>
+int launch_rows(fb200_device* dev, const fb200_attn_args& a) {
+  const int gq = a.h / a.g, gy = a.g * ((gq + NQ - 1) / NQ);
+  const size_t rows = (size_t)a.b * a.s;
+  const int keys = a.window && a.window < a.cap ? a.window : a.cap;
+  // enough CTAs for two per SM; fb200_attn_part_floats counts on rows gy nsplit <= 2 SMs where nsplit > 1
+  int ns = (int)std::min<size_t>(GA_MAX_SPLITS, 2 * (size_t)dev->sm_count / (rows * gy));
+  ns = std::max(1, std::min(ns, (keys + GA_MIN_KEYS - 1) / GA_MIN_KEYS));
+  const size_t smem = (size_t)std::max(NQ * a.dp, GA_WARPS * NQ * a.vp) * 4;
+  return fb200_launch(dev, attn_rows_kernel<T, NP, NQ>, dim3((unsigned)(rows * ns), (unsigned)gy), dim3(GA_THREADS), smem, true, a, ns);
+}
+
+template <typename T>
+int attn_rows(fb200_device* dev, const fb200_attn_args& a) {
+  int rc;
+  if (a.s > 1 && (rc = fb200_attn_prepare(dev, a, false))) return rc;
+  const int n = (std::max(a.dp, a.vp) + 63) / 64, np = n <= 1 ? 1 : n <= 2 ? 2 : n <= 4 ? 4 : 8, nq = ga_heads(np, a.h / a.g);
+  switch (np * 8 + nq) {
+    case 9: return launch_rows<T, 1, 1>(dev, a);
+    case 10: return launch_rows<T, 1, 2>(dev, a);
+    case 12: return launch_rows<T, 1, 4>(dev, a);
+    case 17: return launch_rows<T, 2, 1>(dev, a);
+    case 18: return launch_rows<T, 2, 2>(dev, a);
+    case 20: return launch_rows<T, 2, 4>(dev, a);
+    case 33: return launch_rows<T, 4, 1>(dev, a);
+    case 34: return launch_rows<T, 4, 2>(dev, a);
+    default: return launch_rows<T, 8, 1>(dev, a);
+  }
+}
+
+}  // namespace
+
+bool fb200_attn_covers(int d, int v) { return d > 0 && v > 0 && d <= 512 && v <= 512; }
+
+size_t fb200_attn_part_floats(const fb200_device* dev, int v) { return (size_t)2 * dev->sm_count * 4 * (v + 2); }
+
+int fb200_attn_prepare(fb200_device* dev, const fb200_attn_args& a, bool q_bf16) {
+  const size_t warps = (size_t)a.b * a.s * (a.h + 2 * a.g);
+  const dim3 grid((unsigned)((warps + 7) / 8)), block(256);
+  if (a.cache_f32) return fb200_launch(dev, attn_prep_kernel<float, float>, grid, block, 0, true, a);
+  if (q_bf16) return fb200_launch(dev, attn_prep_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, 0, true, a);
+  return fb200_launch(dev, attn_prep_kernel<__nv_bfloat16, float>, grid, block, 0, true, a);
+}
+
+int fb200_attn_rows(fb200_device* dev, const fb200_attn_args& a) {
+  return a.cache_f32 ? attn_rows<float>(dev, a) : attn_rows<__nv_bfloat16>(dev, a);
+}

@@ -1,10 +1,12 @@
-// Latent attention of a prompt pass on the 5th-generation tensor cores.
+// Attention of a prompt pass of the token-mixer layers on the 5th-generation tensor cores: latent attention and grouped
+// attention.
 //
-// For many query rows the keys and values are expanded once, K | V = W_ukv c for the visible positions (a bf16
-// product, dense_tc.cu), and the attention runs over them; the rotated key part, shared by the heads, is read
+// Latent attention: for many query rows the keys and values are expanded once, K | V = W_ukv c for the visible positions (a
+// bf16 product, dense_tc.cu), and the attention runs over them; the rotated key part, shared by the heads, is read
 // from the cache as it is. Bound: tensor cores, 2 (d + r + v) flops per head and visible (query, key) pair.
+// Grouped attention: keys and values are the cache rows themselves, queries come prepared (normalised, rotated, bf16).
 //
-// latent_prefill_kernel: the scheme of attn_prefill_tc.cu (128 query rows of one head: a softmax thread per row; a
+// mixer_prefill_kernel: the scheme of attn_prefill_tc.cu (128 query rows of one head: a softmax thread per row; a
 // warp that issues the MMAs, a warp that requests the tiles; S = Q K^T double-buffered in TMEM, P written back
 // over S, O accumulated in TMEM and rescaled lazily), with
 //  * one or two groups of 128 rows per CTA (G): two groups share every key and value tile and take turns, one group's
@@ -13,7 +15,10 @@
 //    box may run into the next head's columns, which meet zero columns of Q), the rest from the cache's key part,
 //  * a sliding window: tiles in front of the first visible key are never visited, and only tiles that touch the
 //    diagonal or the window's edge run the mask arithmetic,
-//  * rotary positions applied while Q is staged, the head's sigmoid gate applied to O, bf16 rows out.
+//  * latent queries: rotary positions applied while Q is staged,
+//  * an optional softcap c tanh(. / c) of the scores, with tanh(z) = 1 - 2 / (1 + exp(2 z)); bound then: exponentials and
+//    reciprocals, three per score,
+//  * an optional sink in the denominator, the head's sigmoid gate applied to O, bf16 rows out.
 // Waits are bounded as in attn_prefill_tc.cu.
 #include <algorithm>
 
@@ -29,14 +34,19 @@ constexpr int LP_TAIL = 256;
 constexpr float LP_RESCALE = 8.0f;  // log2 of the growth of a row maximum that triggers a rescale of O
 constexpr uint32_t LP_SW128 = 2;    // layout code of the 128-byte swizzle
 
+enum { LP_LATENT = 0, LP_GROUPED = 1, LP_GROUPED_CAP = 2 };
+
 struct LpArgs {
-  const float* y;  // projections: q at column 0, gate at off_g
+  const float* y;  // projections: q at column 0 (latent), gate at off_g (-1: none)
   size_t ldy;
-  const float *rope_cos, *rope_sin;
+  const __nv_bfloat16* q16;  // grouped: prepared queries [rows][h][dq]
+  const float *rope_cos, *rope_sin, *sink;
   __nv_bfloat16* z;
   size_t ldz;
-  int off_g, s, h, d, r, v, na, nk, rk, window, pos, kbase, keys, cap, v_col;  // v_col: first value column
-  float scale_log2;
+  // d: columns of a head's keys in kvmap, heads dk apart, `group` query heads per key head; v_col: first value column,
+  // heads dv apart; kv_rows: rows of kvmap per sequence
+  int off_g, s, h, d, r, v, na, nk, rk, window, pos, kbase, cap, v_col, group, dq, dk, dv, kv_rows, z_vec;
+  float scale_log2, cap_in, cap_out, out_scale;  // softcap in exponents of two: s -> cap_out tanh(log(2) / 2 cap_in s)
   int* status;
 };
 
@@ -45,10 +55,16 @@ __device__ __forceinline__ uint32_t lp_pack(float lo, float hi) {
   return *reinterpret_cast<const uint32_t*>(&t);
 }
 
-// NV: 64-column boxes of a value tile; KB, VB: key and value tiles in shared memory; G: groups of 128 query rows
-template <int NV, int KB, int VB, int G>
+__device__ __forceinline__ float lp_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// KIND: LP_*; NV: 64-column boxes of a value tile; KB, VB: key and value tiles in shared memory; G: groups of 128 query rows
+template <int KIND, int NV, int KB, int VB, int G>
 __global__ void __launch_bounds__(G * LP_THREADS + 64)
-latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, const __grid_constant__ CUtensorMap cmap) {
+mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, const __grid_constant__ CUtensorMap cmap) {
   // TMEM of a group: S buffers in columns 0..63 and 64..127, O from 128
   constexpr int GCOLS = NV <= 2 ? 256 : 512, COLS = G * GCOLS;
   static_assert(COLS <= 512, "two groups need values of at most 128 columns");
@@ -99,8 +115,20 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "n"(COLS) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
-  // ---- Q: rotary positions, bf16, K-major operand layout: [d, zeros to 64 na | r, zeros]
-  if (tid < SOFT) {
+  // ---- Q, bf16, K-major operand layout
+  if (KIND != LP_LATENT) {
+    if (tid < SOFT) {  // [d, zeros to 64 nk]: eight threads take one 16-byte column piece of eight rows (one core matrix)
+      const __nv_bfloat16* q = a.q16 + ((size_t)b * a.s + q0) * a.h * a.dq + (size_t)head * a.dq;
+#pragma unroll 4
+      for (int id = tid; id < G * LP_Q * kchunks; id += SOFT) {
+        const int row = (id & 7) + ((id / (8 * kchunks)) << 3), c = (id >> 3) % kchunks;
+        uint4 x = make_uint4(0u, 0u, 0u, 0u);
+        if (q0 + row < a.s && c * 8 < a.dq) x = *reinterpret_cast<const uint4*>(q + (size_t)row * a.h * a.dq + c * 8);
+        *reinterpret_cast<uint4*>(Qs + (row >> 7) * qbytes + x_kmajor(row & 127, c, kchunks)) = x;
+      }
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");  // these stores -> tensor-core reads
+    }
+  } else if (tid < SOFT) {  // rotary positions; [d, zeros to 64 na | r, zeros]
     const int half = a.r / 2, nchunks = a.na * 8, rchunks = kchunks - nchunks;
     const bool vec = ((a.d + a.r) & 3) == 0;
     auto put = [&](int row, int c, const float (&x)[8]) {
@@ -186,19 +214,19 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
   if (warp == SOFT / 32 + 1) {
     // ---- copy requester; tile u of the CTA is tile t_first + u
     if (lane == 0) {
-      const int ky = b * a.keys, cy = b * a.cap;
+      const int ky = b * a.kv_rows, cy = b * a.cap, kvh = head / a.group;
       auto fetch_k = [&](int u) {
         const uint32_t dst = smem_u32(Ks) + (uint32_t)((u % KB) * kbytes), bar = bar_kfull + 8 * (u % KB);
         const int j0 = (t_first + u) * LP_K;
         mbar_expect_tx(bar, (uint32_t)kbytes);
-        for (int i = 0; i < a.na; ++i) x_tma_box2(dst + i * LP_BOX, &kvmap, head * a.d + 64 * i, ky + j0, bar);
+        for (int i = 0; i < a.na; ++i) x_tma_box2(dst + i * LP_BOX, &kvmap, kvh * a.dk + 64 * i, ky + j0, bar);
         for (int i = a.na; i < a.nk; ++i) x_tma_box2(dst + i * LP_BOX, &cmap, a.rk + 64 * (i - a.na), cy + j0, bar);
       };
       auto fetch_v = [&](int u) {
         const uint32_t dst = smem_u32(Vs) + (uint32_t)((u % VB) * NV) * LP_BOX, bar = bar_vfull + 8 * (u % VB);
         const int j0 = (t_first + u) * LP_K;
         mbar_expect_tx(bar, NV * LP_BOX);
-        for (int i = 0; i < NV; ++i) x_tma_box2(dst + i * LP_BOX, &kvmap, a.v_col + head * a.v + 64 * i, ky + j0, bar);
+        for (int i = 0; i < NV; ++i) x_tma_box2(dst + i * LP_BOX, &kvmap, a.v_col + kvh * a.dv + 64 * i, ky + j0, bar);
       };
       int nkt = 0, nvt = 0;  // tiles requested
       while (nkt < KB && nkt < ntiles) fetch_k(nkt++);
@@ -287,6 +315,13 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
       x_ld32(tl_base + (uint32_t)(sb * LP_K), sv[0]);
       x_ld32(tl_base + (uint32_t)(sb * LP_K + 32), sv[1]);
       asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+      if (KIND == LP_GROUPED_CAP) {
+#pragma unroll
+        for (int j = 0; j < LP_K; ++j) {
+          const float e = x_ex2(__uint_as_float(sv[j >> 5][j & 31]) * a.cap_in);
+          sv[j >> 5][j & 31] = __float_as_uint(fmaf(-2.0f * a.cap_out, lp_rcp(1.0f + e), a.cap_out));
+        }
+      }
       if (kt + LP_K - 1 > hi_min || kt < lo_max) {  // the tile touches the diagonal or the window's edge of some row
 #pragma unroll
         for (int j = 0; j < LP_K; ++j)
@@ -295,7 +330,8 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
       float mx = -INFINITY;
 #pragma unroll
       for (int j = 0; j < LP_K; ++j) mx = fmaxf(mx, __uint_as_float(sv[j >> 5][j & 31]));
-      const float m_new = fmaxf(m_ref, mx * a.scale_log2);
+      const float sl2 = KIND == LP_GROUPED_CAP ? 1.0f : a.scale_log2;
+      const float m_new = fmaxf(m_ref, mx * sl2);
       const bool grow = m_new > m_ref + LP_RESCALE;  // also true for the first finite maximum
       const float alpha = grow ? x_ex2(m_ref - m_new) : 1.0f;
       if (grow) m_ref = m_new;
@@ -304,8 +340,8 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
       uint32_t pk[LP_K / 2];  // P as bf16 pairs
 #pragma unroll
       for (int j = 0; j < LP_K / 2; ++j) {
-        const float e0 = x_ex2(fmaf(__uint_as_float(sv[(2 * j) >> 5][(2 * j) & 31]), a.scale_log2, -msafe));
-        const float e1 = x_ex2(fmaf(__uint_as_float(sv[(2 * j + 1) >> 5][(2 * j + 1) & 31]), a.scale_log2, -msafe));
+        const float e0 = x_ex2(fmaf(__uint_as_float(sv[(2 * j) >> 5][(2 * j) & 31]), sl2, -msafe));
+        const float e1 = x_ex2(fmaf(__uint_as_float(sv[(2 * j + 1) >> 5][(2 * j + 1) & 31]), sl2, -msafe));
         psum += e0 + e1;
         pk[j] = lp_pack(e0, e1);
       }
@@ -337,8 +373,9 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
       const bool store = row < a.s && !*dead;
       float scale = 0.f;
       if (store) {
-        const float gate = a.y[((size_t)b * a.s + row) * a.ldy + a.off_g + head];
-        scale = (1.0f / l_run) / (1.0f + expf(-gate));
+        if (KIND != LP_LATENT && a.sink) l_run += exp2f(a.sink[head] * 1.4426950408889634f - m_ref);
+        scale = a.out_scale / l_run;
+        if (a.off_g >= 0) scale /= 1.0f + expf(-a.y[((size_t)b * a.s + row) * a.ldy + a.off_g + head]);
       }
       __nv_bfloat16* dst = a.z + ((size_t)b * a.s + row) * a.ldz + (size_t)head * a.v;
 #pragma unroll
@@ -346,7 +383,11 @@ latent_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap,
         uint32_t ov[32];
         x_ld32(tl_base + 2 * LP_K + 32 * c, ov);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-        if (store) {
+        if (store && KIND != LP_LATENT && !a.z_vec) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (32 * c + i < a.v) dst[32 * c + i] = __float2bfloat16(__uint_as_float(ov[i]) * scale);
+        } else if (store) {
 #pragma unroll
           for (int i = 0; i < 4; ++i)  // v is a multiple of 8: whole 16-byte pieces
             if (32 * c + 8 * i < a.v) {
@@ -372,16 +413,39 @@ size_t lp_smem(int nk, int nv, int kb, int vb, int g) {
   return n;
 }
 
-template <int NV, int KB, int VB, int G>
+template <int KIND, int NV, int KB, int VB, int G>
 int launch_lp(fb200_device* dev, const LpArgs& a, int b, const CUtensorMap& kvmap, const CUtensorMap& cmap) {
   const size_t smem = lp_smem(a.nk, NV, KB, VB, G);
   static size_t configured[64] = {0};
   if (configured[dev->ordinal & 63] < smem) {
-    FB_CUDA(dev, cudaFuncSetAttribute(latent_prefill_kernel<NV, KB, VB, G>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    FB_CUDA(dev, cudaFuncSetAttribute(mixer_prefill_kernel<KIND, NV, KB, VB, G>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured[dev->ordinal & 63] = smem;
   }
-  return fb200_launch(dev, latent_prefill_kernel<NV, KB, VB, G>, dim3((unsigned)((a.s + LP_Q * G - 1) / (LP_Q * G)), (unsigned)a.h, (unsigned)b),
+  return fb200_launch(dev, mixer_prefill_kernel<KIND, NV, KB, VB, G>, dim3((unsigned)((a.s + LP_Q * G - 1) / (LP_Q * G)), (unsigned)a.h, (unsigned)b),
                       dim3(G * LP_THREADS + 64), smem, false, a, kvmap, cmap);
+}
+
+constexpr float LP_LOG2E = 1.4426950408889634f;
+
+template <int KIND>
+int launch_kind(fb200_device* dev, const LpArgs& p, int b, const CUtensorMap& kvmap, const CUtensorMap& cmap) {
+  const int nv = (p.v + 63) / 64;
+  // two groups of rows per CTA once one per CTA would not fit the SMs at a time anyway; three key and two value tiles
+  // where they fit
+  const long ctas = (long)((p.s + LP_Q - 1) / LP_Q) * p.h * b;
+  if (nv <= 2 && ctas > dev->sm_count && lp_smem(p.nk, nv, 3, 2, 2) <= 227 * 1024)
+    return nv == 1 ? launch_lp<KIND, 1, 3, 2, 2>(dev, p, b, kvmap, cmap) : launch_lp<KIND, 2, 3, 2, 2>(dev, p, b, kvmap, cmap);
+  const bool deep = lp_smem(p.nk, nv, 3, 2, 1) <= 227 * 1024;
+  switch (nv * 2 + (deep ? 1 : 0)) {
+    case 2: return launch_lp<KIND, 1, 2, 1, 1>(dev, p, b, kvmap, cmap);
+    case 3: return launch_lp<KIND, 1, 3, 2, 1>(dev, p, b, kvmap, cmap);
+    case 4: return launch_lp<KIND, 2, 2, 1, 1>(dev, p, b, kvmap, cmap);
+    case 5: return launch_lp<KIND, 2, 3, 2, 1>(dev, p, b, kvmap, cmap);
+    case 6: return launch_lp<KIND, 3, 2, 1, 1>(dev, p, b, kvmap, cmap);
+    case 7: return launch_lp<KIND, 3, 3, 2, 1>(dev, p, b, kvmap, cmap);
+    case 8: return launch_lp<KIND, 4, 2, 1, 1>(dev, p, b, kvmap, cmap);
+    default: return launch_lp<KIND, 4, 3, 2, 1>(dev, p, b, kvmap, cmap);
+  }
 }
 
 }  // namespace
@@ -412,23 +476,35 @@ int fb200_latent_prefill(fb200_device* dev, const fb200_latent_args& a, const fb
   LpArgs p = {};
   p.y = a.y; p.ldy = a.ldy; p.rope_cos = a.rope_cos; p.rope_sin = a.rope_sin; p.z = (__nv_bfloat16*)a.z; p.ldz = a.ldz; p.off_g = a.off_g;
   p.s = a.s; p.h = a.h; p.d = a.d; p.r = a.r; p.v = a.v; p.na = (a.d + 63) / 64; p.nk = p.na + (a.r + 63) / 64; p.rk = a.rk;
-  p.window = a.window; p.pos = a.pos; p.kbase = kbase; p.keys = keys; p.cap = a.cap; p.v_col = a.h * a.d;
-  p.scale_log2 = a.scale * 1.4426950408889634f; p.status = dev->status;
-  const int nv = (a.v + 63) / 64;
-  // two groups of rows per CTA once one per CTA would not fit the SMs at a time anyway; three key and two value tiles
-  // where they fit
-  const long ctas = (long)((a.s + LP_Q - 1) / LP_Q) * a.h * a.b;
-  if (nv <= 2 && ctas > dev->sm_count && lp_smem(p.nk, nv, 3, 2, 2) <= 227 * 1024)
-    return nv == 1 ? launch_lp<1, 3, 2, 2>(dev, p, a.b, kvmap, cmap) : launch_lp<2, 3, 2, 2>(dev, p, a.b, kvmap, cmap);
-  const bool deep = lp_smem(p.nk, nv, 3, 2, 1) <= 227 * 1024;
-  switch (nv * 2 + (deep ? 1 : 0)) {
-    case 2: return launch_lp<1, 2, 1, 1>(dev, p, a.b, kvmap, cmap);
-    case 3: return launch_lp<1, 3, 2, 1>(dev, p, a.b, kvmap, cmap);
-    case 4: return launch_lp<2, 2, 1, 1>(dev, p, a.b, kvmap, cmap);
-    case 5: return launch_lp<2, 3, 2, 1>(dev, p, a.b, kvmap, cmap);
-    case 6: return launch_lp<3, 2, 1, 1>(dev, p, a.b, kvmap, cmap);
-    case 7: return launch_lp<3, 3, 2, 1>(dev, p, a.b, kvmap, cmap);
-    case 8: return launch_lp<4, 2, 1, 1>(dev, p, a.b, kvmap, cmap);
-    default: return launch_lp<4, 3, 2, 1>(dev, p, a.b, kvmap, cmap);
+  p.window = a.window; p.pos = a.pos; p.kbase = kbase; p.kv_rows = keys; p.cap = a.cap; p.v_col = a.h * a.d;
+  p.group = 1; p.dk = a.d; p.dv = a.v; p.z_vec = 1; p.out_scale = 1.f;
+  p.scale_log2 = a.scale * LP_LOG2E; p.status = dev->status;
+  return launch_kind<LP_LATENT>(dev, p, a.b, kvmap, cmap);
+}
+
+bool fb200_attn_prefill_covers(int h, int d, int v, float scale) {
+  return d <= 256 && v <= 256 && h <= 65535 && scale > 0.f && lp_smem((d + 63) / 64, (v + 63) / 64, 2, 1, 1) <= 227 * 1024;
+}
+
+// a.qn holds b * s rows of prepared bf16 queries; keys and values are the cache rows.
+int fb200_attn_prefill(fb200_device* dev, const fb200_attn_args& a) {
+  int rc;
+  if ((rc = fb200_attn_prepare(dev, a, true))) return rc;
+  const int kbase = a.window ? std::max(0, a.pos - a.window + 1) : 0, keys = a.pos + a.s - kbase;
+  CUtensorMap map;
+  if (!fb200_make_map_2d(&map, (const __nv_bfloat16*)a.cache + (size_t)kbase * a.ldc, 1, (uint64_t)a.ldc, (uint64_t)(a.b - 1) * a.cap + keys,
+                         (uint64_t)a.ldc * 2, LP_K))
+    return fb200_fail(dev, FB200_ERR_CUDA, "grouped attention: tensor map refused");
+  LpArgs p = {};
+  p.y = a.y; p.ldy = a.ldy; p.q16 = (const __nv_bfloat16*)a.qn; p.sink = a.sink; p.z = (__nv_bfloat16*)a.z; p.ldz = a.ldz; p.off_g = a.off_g;
+  p.s = a.s; p.h = a.h; p.d = a.d; p.v = a.v; p.na = p.nk = (a.d + 63) / 64; p.window = a.window; p.pos = a.pos; p.kbase = kbase;
+  p.cap = p.kv_rows = a.cap; p.v_col = a.g * a.dp; p.group = a.h / a.g; p.dq = p.dk = a.dp; p.dv = a.vp;
+  p.z_vec = a.v % 8 == 0 && a.ldz % 8 == 0 && ((uintptr_t)a.z & 15u) == 0; p.out_scale = a.out_scale;
+  p.scale_log2 = a.scale * LP_LOG2E; p.status = dev->status;
+  if (a.softcap > 0.f) {
+    p.cap_in = 2.f * LP_LOG2E * a.scale / a.softcap;
+    p.cap_out = a.softcap * LP_LOG2E;
+    return launch_kind<LP_GROUPED_CAP>(dev, p, a.b, map, map);
   }
+  return launch_kind<LP_GROUPED>(dev, p, a.b, map, map);
 }

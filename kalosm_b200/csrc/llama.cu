@@ -467,8 +467,8 @@ int run_forward(fb200_llama* m, int batch, int seq, bool commit = true) {
   const size_t rows = (size_t)batch * seq;
   const int E = c.hidden, H = c.n_head, HK = c.n_kv_head, D = c.head_dim;
   int rc;
-  if ((rc = fb200_embedding_lookup(dev, m->token_embd, m->ids, rows, m->x))) return rc;
   if (m->hybrid) return fb200_hybrid_forward(m, batch, seq, commit);
+  if ((rc = fb200_embedding_lookup(dev, m->token_embd, m->ids, rows, m->x))) return rc;
   const float scale = (float)(1.0 / sqrt((double)D));  // attention_layer.rs:674
   const int nsplit = fb200_attention_nsplit(dev, batch, HK, H / HK, seq, seq > 1 ? seq : c.max_seq_len);
   size_t part_bytes;

@@ -1,5 +1,5 @@
 // Token mixers of the hybrid decoder layers: what a layer's host code hands to the kernels of
-// delta_rule.cu and latent_attn.cu. Every size and constant is an argument.
+// delta_rule.cu, latent_attn.cu, group_attn.cu and linear_attn.cu. Every size and constant is an argument.
 #pragma once
 
 #include "common.cuh"
@@ -66,3 +66,62 @@ int fb200_latent_append(fb200_device* dev, const fb200_latent_args& a);  // the 
 int fb200_latent_rows(fb200_device* dev, const fb200_latent_args& a);    // any s: append, latent-space attention row by row
 bool fb200_latent_prefill_covers(int h, int d, int r, int v, int rk, float scale);
 int fb200_latent_prefill(fb200_device* dev, const fb200_latent_args& a, const fb200_qmatrix* w_ukv);  // after the append
+
+// ---- grouped softmax attention ---------------------------------------------------------------------------
+// Projections [b * s, ldy]: q [h][d] at column 0, k [g][d] at off_k, v [g][v] at off_v, output gate [h] at off_g (-1:
+// none). q and k heads are RMS-normalised under q_norm / k_norm (null: not), then rotated on their first r dimensions (i pairs
+// with i + r / 2). The cache holds per position k [g][dp] | v [g][vp] (dp, vp: sizes padded to 8, the padding zero), ldc
+// elements apart, bf16 or f32. Scores (q . k) scale, through softcap tanh(. / softcap) if softcap > 0; query i sees the keys j
+// with 0 <= i - j < window (window 0: all of 0 .. i); sink (null: none) adds exp(sink[head]) to the denominator. The
+// output is x sigmoid(gate) x out_scale.
+struct fb200_attn_args {
+  const float* y;
+  size_t ldy;
+  int off_k, off_v, off_g;
+  const float *q_norm, *k_norm, *sink;
+  float eps, scale, softcap, out_scale;
+  const float *rope_cos, *rope_sin;  // [cap, r / 2]
+  void* cache;
+  int cache_f32, ldc, cap;
+  int b, s, h, g, d, v, dp, vp, r, window;
+  const int* pos_dev;
+  int pos;  // the same on the host (prompt passes)
+  void* z;
+  size_t ldz;
+  int z_bf16;
+  void* qn;     // prompt passes: prepared queries [rows][h][dp], f32 (rows) or bf16 (tensor cores)
+  float* part;  // fb200_attn_part_floats
+  int* done;    // [rows * h] arrival counters, zero between launches
+};
+bool fb200_attn_covers(int d, int v);
+size_t fb200_attn_part_floats(const fb200_device* dev, int v);
+int fb200_attn_prepare(fb200_device* dev, const fb200_attn_args& a, bool q_bf16);  // queries into qn, keys and values into the cache
+int fb200_attn_rows(fb200_device* dev, const fb200_attn_args& a);                  // any s, row by row; s == 1 is one kernel
+bool fb200_attn_prefill_covers(int h, int d, int v, float scale);
+int fb200_attn_prefill(fb200_device* dev, const fb200_attn_args& a);               // bf16, tensor cores
+
+// ---- linear attention with a fixed decay per head ----------------------------------------------------------
+// Projections [b * s, ldy]: q [h][d] at column 0, k [h][d] at off_k, v [h][v] at off_v (all through SiLU), gate [h v] at
+// off_g. The state of a sequence is S, f32 [h][v][dp]; position 0 starts from zero whatever the buffer holds. decay
+// [h][FB200_LINEAR_CHUNK + 1] holds the powers 0 .. of every head's decay.
+constexpr int FB200_LINEAR_CHUNK = 64;
+struct fb200_linear_args {
+  const float* y;
+  size_t ldy;
+  int off_k, off_v, off_g;
+  const float *decay, *out_norm;
+  float eps, out_scale;
+  float* state;
+  int b, s, h, d, v, dp;
+  const int* pos_dev;
+  void* z;
+  size_t ldz;
+  int z_bf16;
+  int commit;  // 0: a dry run of a decode step, the state stays as it is
+  int bf16;    // prompt operands may be bf16
+  float* o;    // read-out [rows][h v]
+  int* done;   // [b] arrival counters, zero between launches
+};
+int fb200_linear_dp(int d);                                              // padded head size, 0 when d is not covered
+int fb200_linear_step(fb200_device* dev, const fb200_linear_args& a);    // s == 1: one kernel
+int fb200_linear_prompt(fb200_device* dev, const fb200_linear_args& a);  // s > 1

@@ -161,6 +161,33 @@ void fb200_rope_tables_host(int head_dim, int ctx, float theta, float factor, fl
     }
 }
 
+// Rotary tables [ctx, dims / 2] with YaRN scaling (factor > 0): frequencies that turn often inside the original context stay,
+// slow ones are divided by the factor, a ramp lies in between, and cos and sin grow with the factor's logarithm.
+void fb200_rope_tables_yarn_host(int dims, int ctx, double base, double factor, double fast, double slow, double original,
+                                 std::vector<float>& cs, std::vector<float>& sn) {
+  const int half = dims / 2;
+  const double PI = 3.14159265358979323846;
+  std::vector<double> f(half);
+  for (int i = 0; i < half; ++i) f[i] = std::pow(base, -2.0 * i / dims);
+  double mul = 1.0;
+  if (factor > 0) {
+    auto dim_of = [&](double turns) { return dims * std::log(original / (2.0 * PI * turns)) / (2.0 * std::log(base)); };
+    const double lo = std::max(std::floor(dim_of(fast)), 0.0), hi = std::min(std::ceil(dim_of(slow)), dims - 1.0);
+    for (int i = 0; i < half; ++i) {
+      const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+      f[i] = f[i] / factor * ramp + f[i] * (1.0 - ramp);
+    }
+    mul = 0.1 * std::log(factor) + 1.0;
+  }
+  cs.resize((size_t)ctx * half);
+  sn.resize((size_t)ctx * half);
+  for (int p = 0; p < ctx; ++p)
+    for (int i = 0; i < half; ++i) {
+      cs[(size_t)p * half + i] = (float)(std::cos(p * f[i]) * mul);
+      sn[(size_t)p * half + i] = (float)(std::sin(p * f[i]) * mul);
+    }
+}
+
 int fb200_launch_rms_norm(fb200_device* dev, const float* x, const float* res, const float* w,
                           const float* b, float eps, size_t rows, size_t n, float* y) {
   if (rows == 0 || n == 0) return FB200_OK;

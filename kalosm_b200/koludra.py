@@ -5,14 +5,8 @@ config.json: "vocab", "width", "norm": {"eps"} and "layers", each with its mixer
 ("mixer") and its feed-forward ("mlp", or null). Tensors: "embed", "head", "final.norm" and per layer
 "l<i>.norm1", "l<i>.mix.*", "l<i>.mlp.*".
 """
-import json
-import os
-import re
-
-import numpy as np
-
 from . import MIX_DELTA, MIX_LATENT, HybridDecoder
-from .safetensors import SafetensorsFile
+from .checkpoint import ConfigError, fill, mixer_kind, open_checkpoint
 
 ARCHITECTURE = "Koludra"
 # suffix of a layer tensor -> the library's tensor name
@@ -23,15 +17,6 @@ DELTA = {"mix.k": "mix_k", "mix.v": "mix_v", "mix.b": "mix_beta", "mix.a": "mix_
          "mix.norm": "mix_out_norm"}
 LATENT = {"mix.uk": "mix_uk", "mix.uv": "mix_uv"}
 LATENT_OWN = {"mix.dkv": "mix_dkv", "mix.dkv.norm": "mix_dkv_norm"}
-
-
-class ConfigError(ValueError):
-    pass
-
-
-def mixer_kind(name):
-    """'delta' or 'latent_attention': a trailing _<n> only tells apart variants of other sizes."""
-    return re.sub(r"_\d+$", "", name)
 
 
 def layer_config(index, layer):
@@ -70,24 +55,11 @@ def build(device, config, tensor, max_seq_len, max_batch=1, dtype="bfloat16"):
     m = HybridDecoder(device, hidden=int(config["width"]), vocab=int(config["vocab"]), rms_eps=float(config["norm"]["eps"]),
                       layers=[layer_config(i, layer) for i, layer in enumerate(config["layers"])], max_seq_len=max_seq_len,
                       max_batch=max_batch, compute=dtype)
-
-    def put(short, layer, name):
-        ty, shape, raw = tensor(name)
-        m.set_tensor(short, layer, ty, shape, np.asarray(raw))
-    put("token_embd", -1, "embed")
-    put("output", -1, "head")
-    put("output_norm", -1, "final.norm")
-    for i, layer in enumerate(config["layers"]):
-        for suffix, short in layer_tensors(layer).items():
-            put(short, i, f"l{i}.{suffix}")
-    return m
+    return fill(m, tensor, [(short, i, f"l{i}.{suffix}") for i, layer in enumerate(config["layers"])
+                            for suffix, short in layer_tensors(layer).items()])
 
 
 def load(device, path, max_seq_len=None, max_batch=1, dtype="bfloat16"):
     """Loads a checkpoint folder (config.json and model.safetensors)."""
-    with open(os.path.join(path, "config.json")) as f:
-        config = json.load(f)
-    if config.get("architecture") != ARCHITECTURE:
-        raise ConfigError(f"architecture {config.get('architecture')!r} is not {ARCHITECTURE!r}")
-    weights = SafetensorsFile(os.path.join(path, "model.safetensors"))
-    return build(device, config, weights.raw, max_seq_len or 4096, max_batch, dtype)
+    config, tensor = open_checkpoint(path, ARCHITECTURE)
+    return build(device, config, tensor, max_seq_len or 4096, max_batch, dtype)

@@ -2,7 +2,7 @@
 import json
 import os
 
-from . import gguf, koludra
+from . import gguf, koludra, sofudra
 
 
 def _gguf_llama(device, path, max_seq_len=None, max_batch=1, dtype=None):
@@ -12,11 +12,11 @@ def _gguf_llama(device, path, max_seq_len=None, max_batch=1, dtype=None):
 
 
 # architecture name -> loader(device, path, max_seq_len, max_batch, dtype)
-REGISTRY = {"llama": _gguf_llama, koludra.ARCHITECTURE: koludra.load}
+REGISTRY = {"llama": _gguf_llama, koludra.ARCHITECTURE: koludra.load, sofudra.ARCHITECTURE: sofudra.load}
 
 
 # architectures that the dense part of the library serves (build.build(part="dense"))
-DENSE = (koludra.ARCHITECTURE,)
+DENSE = (koludra.ARCHITECTURE, sofudra.ARCHITECTURE)
 
 
 def architecture(path):
