@@ -600,7 +600,7 @@ def run_tensor_parallel(args):
         sys.exit(3)
 
 
-# ---- --hybrid: a Koludra decoder (delta rule + latent attention, dense bf16) beside a Llama decoder of equal size --------
+# ---- --hybrid: decoders of token-mixer layers (dense bf16) beside a Llama decoder of equal size --------------------------
 
 def hybrid_layers(width, ffn, window, n_layer):
     """Layer list with the sizes of real layers: 128-wide heads, 512-wide latents, 3 delta rules to 2 attentions."""
@@ -657,6 +657,116 @@ def build_hybrid_model(dev, torch, width, ffn, window, n_layer, vocab, ctx, seed
     return koludra.build(dev, cfg, tensor, ctx, 1), layers, params[0]
 
 
+def sofudra_config(width, ffn, window, n_layer, vocab):
+    """Layers of real sizes: 128-wide heads, four query heads per key head; n_layer layer runs, two of the layers run twice."""
+    h, mlp = width // 128, {"kind": "dense", "ff": ffn}
+    att = dict(heads=h, kv_heads=h // 4, dim=128, vdim=128, scale=128 ** -0.5)
+    a = {"type": "attention", "mlp": mlp, "mixer": dict(att, mask={"size": window}, rot={
+        "base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}})}
+    p = {"type": "parallel", "mlp": mlp, "mixer": dict(left_scale=0.7, right_scale=0.8, left=dict(att, softcap=50.0), right=dict(
+        heads=h, dim=128, vdim=128, decay=[1.0 - 2.0 ** -(1 + 7.0 * i / h) for i in range(h)]))}
+    return {"architecture": "Sofudra", "embedding": {"scale": width ** 0.5}, "layers": [(p, a)[i % 2] for i in range(n_layer - 2)], "logit_softcap": 30.0,
+            "loop": {"start": 2, "stop": 4, "times": 2}, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "vocab": vocab, "width": width}
+
+
+def sofudra_shape(cfg, name):
+    width, vocab = cfg["width"], cfg["vocab"]
+    if name in ("embed", "head"):
+        return (vocab, width)
+    if name == "loop.in":
+        return (width, 2 * width)
+    if name == "final.norm" or name.split(".")[1].startswith("norm"):
+        return (width,)
+    layer, part, rest = name.split(".", 2)
+    L = cfg["layers"][int(layer[1:])]
+    if part == "mlp":
+        return (width, L["mlp"]["ff"]) if rest == "down" else (L["mlp"]["ff"], width)
+    mx, linear = L["mixer"], rest.startswith("right.")
+    if L["type"] == "parallel":
+        side, rest = rest.split(".", 1)
+        mx = mx[side]
+    H, D, V = mx["heads"], mx["dim"], mx["vdim"]
+    G = mx.get("kv_heads", H)
+    rows = {"q": H * D, "k": G * D, "v": G * V, "g": H * V if linear else H}
+    if rest.endswith(".b"):
+        return (rows[rest[0]],)
+    if rest.endswith(".norm"):
+        return (D,)
+    return {"o": (width, H * V), "norm": (H * V,), "sink": (H,)}.get(rest) or (rows[rest], width)
+
+
+def build_sofudra_model(dev, torch, cfg, ctx, seed=0):
+    """Random weights made on the GPU. Returns (model, parameters of the matrices a step streams)."""
+    import kalosm_b200 as kb
+    from kalosm_b200 import sofudra
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    loop = cfg["loop"]
+    params = [0]
+
+    def tensor(name):
+        shape = sofudra_shape(cfg, name)
+        w = torch.randn(shape, generator=g, device="cuda", dtype=torch.float32)
+        if len(shape) == 1:
+            w = 1.0 + 0.1 * w if "norm" in name else 0.2 * w
+        elif name != "embed":
+            w *= shape[1] ** -0.5
+            inside = name.startswith("l") and name != "loop.in" and loop["start"] <= int(name.split(".")[0][1:]) < loop["stop"]
+            params[0] += shape[0] * shape[1] * (loop["times"] if inside or name == "loop.in" else 1)
+        return kb.BF16, shape, w.to(torch.bfloat16).view(torch.int16).cpu().numpy()
+    return sofudra.build(dev, cfg, tensor, ctx, 1), params[0]
+
+
+def mixer_peaks(n_sm):
+    """hbm in bytes/s, tensor and f32 (nominal FMA rate) in flop/s, sfu in special functions/s (16 per SM and clock)."""
+    return {"hbm": peaks()[0] * 1e9, "tensor": tensor_peak()[0] * 1e12, "f32": n_sm * 128 * 2 * 1.965e9, "sfu": n_sm * 16 * 1.965e9}
+
+
+def sofudra_work(cfg, rows, ctx, n_sm):
+    """As hybrid_work, for the layer runs of a Sofudra decoder. Where a kernel has two bounds the later one counts."""
+    peak, w, width, loop = mixer_peaks(n_sm), {}, cfg["width"], cfg["loop"]
+
+    def add(name, *bounds):
+        kind, amount = max(bounds, key=lambda b: b[1] / peak[b[0]])
+        w[name] = w.get(name, 0.0) + amount / peak[kind]
+        kinds.setdefault(name, set()).add(kind)
+    kinds = {}
+    gemm = "dense_gemv_kernel" if rows == 1 else "dense_tc_kernel"
+
+    def matrix(params):
+        add(gemm, ("hbm", 2.0 * params) if rows == 1 else ("tensor", 2.0 * params * rows))
+
+    def attention(mx):
+        H, G, D, V, win = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"], (mx.get("mask") or {}).get("size") or (1 << 30)
+        if rows == 1:
+            add("attn_rows_kernel", ("hbm", 2.0 * min(win, ctx + 1) * G * (D + V)))
+        else:
+            pairs = float(sum(min(win, ctx + i + 1) for i in range(rows))) * H
+            add("mixer_prefill_kernel", ("tensor", 2.0 * pairs * (D + V)), ("sfu", pairs * (3 if mx.get("softcap") else 1)))
+            add("attn_prep_kernel", ("hbm", rows * (6.0 * H * D + 6.0 * G * (D + V))))
+        return (H * D + G * (D + V)) * width + H * V * width
+
+    def linear(mx):
+        H, D, V = mx["heads"], mx["dim"], mx["vdim"]
+        if rows == 1:
+            add("linear_scan_kernel", ("hbm", 8.0 * H * V * D))
+        else:
+            add("linear_scan_kernel", ("hbm", rows * H * (8.0 * D + 8.0 * V)), ("f32", 4.0 * rows * H * V * D))
+            add("linear_prep_kernel", ("hbm", 6.0 * rows * H * (2 * D + V)))
+            # inside a chunk of 128 tokens, the state's read-out and its update
+            add("linear_prefill_kernel", ("hbm", rows * H * (4.0 * D + 6.0 * V)), ("tensor", rows * H * (2.0 * 128 * (D + V) / 2 + 4.0 * D * V)))
+            add("linear_out_kernel", ("hbm", 10.0 * rows * H * V))
+        return (2 * H * D + 3 * H * V) * width
+    runs = [L for i, L in enumerate(cfg["layers"]) for _ in range(loop["times"] if loop["start"] <= i < loop["stop"] else 1)]
+    for L in runs:
+        mx = L["mixer"]
+        mats = 2 * L["mlp"]["ff"] * width + (attention(mx) if L["type"] == "attention" else attention(mx["left"]) + mx["left"]["heads"] * width + linear(mx["right"]))
+        matrix(mats)
+    matrix(2 * width * width * loop["times"])
+    if rows == 1:
+        matrix(cfg["vocab"] * width)
+    return {n: ("+".join(sorted(kinds[n])), t, 1.0) for n, t in w.items()}
+
+
 def device_table(torch, fn, reps):
     """Device time per kernel of `reps` calls of fn (CUPTI): {short kernel name: (us per call, launches per call)}."""
     from torch.profiler import ProfilerActivity, profile
@@ -678,7 +788,7 @@ def device_table(torch, fn, reps):
 def hybrid_work(layers, width, vocab, rows, ctx, n_sm):
     """Roofline work of one pass of `rows` new positions behind `ctx` cached ones: {kernel: (kind, amount, peak)}; kind "hbm"
     in bytes, "tensor" and "f32" in flops."""
-    peak = {"hbm": peaks()[0] * 1e9, "tensor": tensor_peak()[0] * 1e12, "f32": n_sm * 128 * 2 * 1.965e9}  # f32: nominal FMA rate
+    peak = mixer_peaks(n_sm)
     w = {}
 
     def add(name, kind, amount):
@@ -705,7 +815,7 @@ def hybrid_work(layers, width, vocab, rows, ctx, n_sm):
             win = mx["mask"]["size"]
             add("dense_tc_kernel", "tensor", 2.0 * (rows + min(win - 1, ctx)) * H * (mx["dim"] + V) * mx["kv_rank"])
             pairs = float(sum(min(win, ctx + i + 1) for i in range(rows)))
-            add("latent_prefill_kernel", "tensor", 2.0 * pairs * H * (mx["dim"] + mx["rot_dim"] + V))
+            add("mixer_prefill_kernel", "tensor", 2.0 * pairs * H * (mx["dim"] + mx["rot_dim"] + V))
     if rows == 1:
         add("dense_gemv_kernel", "hbm", 2.0 * vocab * width)
     return {n: (k, a, peak[k]) for n, (k, a) in w.items()}
@@ -731,8 +841,8 @@ def kernel_rows(table, work):
 
 
 def run_hybrid(args):
-    """Prefill and decode of a Koludra decoder with layers of real-model sizes (random bf16 weights) beside a Llama decoder
-    (Q4_K / Q6_K weights, the closest existing model) of the same width, feed-forward, layers and vocabulary; one JSON line per size
+    """Prefill and decode of Koludra and Sofudra decoders with layers of real-model sizes (random bf16 weights) beside a Llama
+    decoder (Q4_K / Q6_K weights) of the same width, feed-forward, layers and vocabulary; one JSON line per size
     with the device time and roofline fraction of every kernel. Kernels of a decode step overlap their predecessors' tails (programmatic
     dependent launch), so their times in the table contain waiting; FB200_PDL=0 gives stand-alone times. Not the bench line."""
     import torch
@@ -761,12 +871,16 @@ def run_hybrid(args):
         line = {"bench": "hybrid", "width": width, "ffn": ffn, "window": window, "layers": n_layer, "vocab": vocab,
                 "data": "synthetic (random weights, random token ids)", "peaks": {"hbm_gbs": peaks()[0], "bf16_tflops": tensor_peak()[0]},
                 "pdl": os.environ.get("FB200_PDL", "1"), "l2": "every pass streams more weights than the L2 holds"}
-        for kind in ("koludra",) if args.no_llama else ("koludra", "llama"):
+        for kind in args.hybrid_models.split(","):
             dev = kb.Device(0, stream.cuda_stream)
-            layers = None
+            dense = kind in ("koludra", "sofudra")
             if kind == "koludra":
                 m, layers, params = build_hybrid_model(dev, torch, width, ffn, window, n_layer, vocab, ctx)
-                wbytes = 2.0 * params
+                wbytes, work_of = 2.0 * params, lambda rows, at: hybrid_work(layers, width, vocab, rows, at, n_sm)
+            elif kind == "sofudra":
+                scfg = sofudra_config(width, ffn, window, n_layer, vocab)
+                m, params = build_sofudra_model(dev, torch, scfg, ctx)
+                wbytes, work_of = 2.0 * params, lambda rows, at: sofudra_work(scfg, rows, at, n_sm)
             else:
                 cfg = dict(n_layer=n_layer, hidden=width, ffn=ffn, n_head=width // 128, n_kv_head=width // 512, head_dim=128, vocab=vocab)
                 m = build_gpu_model(dev, torch, cfg, 1, ctx, seed=1)
@@ -785,13 +899,13 @@ def run_hybrid(args):
                     m.forward(prompt, want_logits=False)
                 ms = timed(prefill, 3 if n > 4096 else 5)
                 table = device_table(torch, prefill, 2)
-                work = hybrid_work(layers, width, vocab, n, 0, n_sm) if layers else llama_work(cfg, n, 0)
+                work = work_of(n, 0) if dense else llama_work(cfg, n, 0)
                 out["prefill"].append({"tokens": n, "ms": ms, "tok_s": n / ms * 1e3, "kernels": kernel_rows(table, work)})
                 m.generate_greedy(last, 8)
                 ms = timed(lambda: m.generate_greedy(last, steps), 1) / steps
-                kv = 0 if layers else 4.0 * n_layer * (width // 512) * 128 * (n + 8 + steps * 1.5)
+                kv = 0 if dense else 4.0 * n_layer * (width // 512) * 128 * (n + 8 + steps * 1.5)
                 table = {k: (us / 16, c / 16) for k, (us, c) in device_table(torch, lambda: m.generate_greedy(last, 16), 1).items()}
-                work = hybrid_work(layers, width, vocab, 1, n, n_sm) if layers else {"fused_step_kernel": ("hbm", wbytes + kv, peaks()[0] * 1e9)}
+                work = work_of(1, n) if dense else {"fused_step_kernel": ("hbm", wbytes + kv, peaks()[0] * 1e9)}
                 out["decode"].append({"context": n, "ms": ms, "tok_s": 1e3 / ms, "hbm_frac": (wbytes + kv) / (ms * 1e-3) / (peaks()[0] * 1e9),
                                       "kernels": kernel_rows(table, work)})
             out["clocks"] = sampler.stop(t0, time.time())
@@ -1134,9 +1248,9 @@ def main():
     ap.add_argument("--tp-nccl", action="store_true", help="with --tp: keep the decode step on NCCL all-reduces")
     ap.add_argument("--no-tp", action="store_true", help="with --gpus N > 1: skip the tensor-parallel leg after the replicas")
     ap.add_argument("--hybrid", action="store_true",
-                    help="prefill and decode of a Koludra decoder at two layer sizes beside a Llama decoder of equal size")
+                    help="prefill and decode of decoders of token-mixer layers at two layer sizes beside a Llama decoder of equal size")
     ap.add_argument("--hybrid-only", type=int, default=0, help="with --hybrid: only this width (2048 or 4096)")
-    ap.add_argument("--no-llama", action="store_true", help="with --hybrid: skip the Llama side")
+    ap.add_argument("--hybrid-models", default="koludra,llama", help="with --hybrid: which of koludra, sofudra, llama")
     ap.add_argument("--gemv-reps", type=int, default=8)
     ap.add_argument("--kernel-table", action="store_true",
                     help="add the device time per kernel of 8 extra decode steps (torch.profiler) as `kernel_table`")

@@ -11,7 +11,7 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libfusor_b200.so")
 SOURCES = ["api.cu", "repack.cu", "qgemv.cu", "qgemv1.cu", "q5gemv.cu", "dense.cu", "dense_tc.cu", "qgemm.cu", "ops.cu", "attention.cu", "attn_prefill.cu", "attn_prefill_tc.cu", "attn_decode_tc.cu",
-           "fused_step.cu", "llama.cu", "hybrid.cu", "delta_rule.cu", "latent_attn.cu", "latent_prefill.cu", "group_attn.cu", "linear_attn.cu", "comm.cu", "sampling.cu"]
+           "fused_step.cu", "llama.cu", "hybrid.cu", "delta_rule.cu", "latent_attn.cu", "latent_prefill.cu", "group_attn.cu", "linear_attn.cu", "linear_prefill.cu", "comm.cu", "sampling.cu"]
 HEADERS = ["common.cuh", "formats.cuh", "qgemv_common.cuh", "qgemv1_groups.cuh", "packed_act.cuh",
            "attn_decode.cuh", "attn_mma.cuh", "qgemv1_groups2.cuh", "fused_step.cuh", "decoder.cuh", "dense.cuh", "mixers.cuh", "state_columns.cuh", "tcgen05.cuh", os.path.join("..", "..", "include", "fusor_b200.h")]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -28,7 +28,7 @@ def _nvcc() -> str:
 # What a decoder of token-mixer layers over dense weights needs. A library of this part alone has the other sources'
 # functions as stubs that answer FB200_ERR_UNSUPPORTED_DTYPE, and lacks their C entry points.
 DENSE_PART = ["api.cu", "repack.cu", "dense.cu", "dense_tc.cu", "ops.cu", "sampling.cu", "llama.cu", "hybrid.cu", "delta_rule.cu",
-              "latent_attn.cu", "latent_prefill.cu", "group_attn.cu", "linear_attn.cu"]
+              "latent_attn.cu", "latent_prefill.cu", "group_attn.cu", "linear_attn.cu", "linear_prefill.cu"]
 DENSE_LIB = os.path.join(HERE, "libfusor_b200_dense.so")
 
 

@@ -379,6 +379,7 @@ int run_mixer(fb200_llama* m, const Mixer& M, int pass, int batch, int seq, bool
     a.eps = m->cfg.rms_eps; a.out_scale = c.out_scale; a.state = M.state + pass * M.pass_state; a.b = batch; a.s = seq; a.h = c.heads;
     a.d = c.dim; a.v = c.vdim; a.dp = M.dp; a.pos_dev = m->pos_dev; a.z = z; a.ldz = hy->ldz; a.z_bf16 = !wide; a.commit = commit;
     a.o = hy->o; a.done = hy->done + hy->done_linear; a.bf16 = !hy->f32;
+    a.q16 = (__nv_bfloat16*)hy->qn; a.k16 = (__nv_bfloat16*)hy->kn; a.v16 = (__nv_bfloat16*)hy->vn;
     return seq == 1 ? fb200_linear_step(dev, a) : fb200_linear_prompt(dev, a);
   }
   if (c.mixer == FB200_MIX_ATTENTION) {
@@ -500,6 +501,10 @@ int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows) {
       kvh = std::max(kvh, (size_t)c.kv_heads);
     } else if (c.mixer == FB200_MIX_LINEAR) {
       o = std::max(o, (size_t)M.ko);
+      if (!hy->f32) {
+        qk = std::max(qk, (size_t)c.heads * M.dp / 2);
+        hv = std::max(hv, c.heads * up_to(c.vdim, 8) / 2);
+      }
     } else if (c.mixer == FB200_MIX_ATTENTION) {
       q = std::max(q, (size_t)c.heads * M.dp);
       part = std::max(part, fb200_attn_part_floats(dev, c.vdim));
@@ -513,7 +518,8 @@ int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows) {
     }
   }
   q = std::max(q, qk);
-  o = std::max(o, hv);
+  for (const auto& M : hy->mixers)
+    if (M.c.mixer == FB200_MIX_DELTA) o = std::max(o, hv);
   hy->done_linear = done;
   bool norm2 = false;
   for (const auto& L : hy->layers) norm2 = norm2 || L.norm2;

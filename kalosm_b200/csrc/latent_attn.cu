@@ -300,12 +300,6 @@ __global__ void __launch_bounds__(LO_THREADS) latent_out_kernel(const fb200_late
 // tiles of the latent per warp at most. Positions before this pass are requested before the kernel in front has finished.
 constexpr int LM_KEYS = 64, LM_THREADS = 128, LM_PS = LM_KEYS + 8;
 
-__device__ __forceinline__ void lm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
 template <int NT>
 __global__ void __launch_bounds__(LM_THREADS) latent_attn_mma_kernel(const fb200_latent_args a) {
   extern __shared__ __align__(16) float lsm[];
@@ -367,10 +361,10 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attn_mma_kernel(const fb200
       pf_ldsm4(qa_h + ks * 32, ah);
       pf_ldsm4(qa_l + ks * 32, al);
       pf_ldsm4(kb + ks * 32, bb);
-      lm_mma(s[0], ah, bb[0], bb[1]);
-      lm_mma(s[1], ah, bb[2], bb[3]);
-      lm_mma(s[0], al, bb[0], bb[1]);
-      lm_mma(s[1], al, bb[2], bb[3]);
+      pf_mma_bf16(s[0], ah, bb[0], bb[1]);
+      pf_mma_bf16(s[1], ah, bb[2], bb[3]);
+      pf_mma_bf16(s[0], al, bb[0], bb[1]);
+      pf_mma_bf16(s[1], al, bb[2], bb[3]);
     }
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -422,8 +416,8 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attn_mma_kernel(const fb200
         if (i >= ntiles) break;
         uint32_t bb[4];
         pf_ldsm4_t(vb + (uint32_t)(ks * 16 * stride + i * 8) * 2, bb);
-        lm_mma(o[i], pa, bb[0], bb[1]);
-        if (i + 1 < NT) lm_mma(o[i + 1 < NT ? i + 1 : i], pa, bb[2], bb[3]);
+        pf_mma_bf16(o[i], pa, bb[0], bb[1]);
+        if (i + 1 < NT) pf_mma_bf16(o[i + 1 < NT ? i + 1 : i], pa, bb[2], bb[3]);
       }
     }
     if (kt + LM_KEYS < k1) {

@@ -104,7 +104,7 @@ int fb200_attn_prefill(fb200_device* dev, const fb200_attn_args& a);            
 // Projections [b * s, ldy]: q [h][d] at column 0, k [h][d] at off_k, v [h][v] at off_v (all through SiLU), gate [h v] at
 // off_g. The state of a sequence is S, f32 [h][v][dp]; position 0 starts from zero whatever the buffer holds. decay
 // [h][FB200_LINEAR_CHUNK + 1] holds the powers 0 .. of every head's decay.
-constexpr int FB200_LINEAR_CHUNK = 64;
+constexpr int FB200_LINEAR_CHUNK = 128;
 struct fb200_linear_args {
   const float* y;
   size_t ldy;
@@ -121,7 +121,10 @@ struct fb200_linear_args {
   int bf16;    // prompt operands may be bf16
   float* o;    // read-out [rows][h v]
   int* done;   // [b] arrival counters, zero between launches
+  __nv_bfloat16 *q16, *k16, *v16;  // prompt scratch: SiLU'd q, k [rows][h][dp], v [rows][h][vp], vp = v padded to 8
 };
 int fb200_linear_dp(int d);                                              // padded head size, 0 when d is not covered
 int fb200_linear_step(fb200_device* dev, const fb200_linear_args& a);    // s == 1: one kernel
 int fb200_linear_prompt(fb200_device* dev, const fb200_linear_args& a);  // s > 1
+bool fb200_linear_prefill_covers(const fb200_linear_args& a);
+int fb200_linear_prefill(fb200_device* dev, const fb200_linear_args& a);  // read-out of a prompt from q16, k16, v16: tensor cores

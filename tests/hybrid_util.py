@@ -99,11 +99,11 @@ def gpu_model(dev, cfg, w, dtype, max_seq_len=512, max_batch=1):
     return koludra.build(dev, cfg, lambda n: (kb.BF16, sh[n], w[n].view(np.uint8).reshape(-1)), max_seq_len, max_batch, dtype)
 
 
-def write_checkpoint(folder, cfg, w):
+def write_checkpoint(folder, cfg, w, sh=None):
     os.makedirs(folder, exist_ok=True)
     with open(os.path.join(folder, "config.json"), "w") as f:
         json.dump(cfg, f)
-    sh = shapes(cfg)
+    sh = sh or shapes(cfg)
     write_safetensors(os.path.join(folder, "model.safetensors"), [(n, "BF16", sh[n], b) for n, b in w.items()])
 
 
