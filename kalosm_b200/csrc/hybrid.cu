@@ -80,7 +80,7 @@ struct fb200_hybrid {
   float* xend = nullptr;    // where a pass leaves the residual stream
   float *proj = nullptr, *zf = nullptr;
   __nv_bfloat16 *hb = nullptr, *zb = nullptr;
-  float *qn = nullptr, *kn = nullptr, *vn = nullptr, *gb = nullptr, *kq = nullptr, *o = nullptr;
+  float *qn = nullptr, *kn = nullptr, *vn = nullptr, *gb = nullptr, *kq = nullptr, *o = nullptr, *seg = nullptr;
   float *qa = nullptr, *part = nullptr;
   int* done = nullptr;      // arrival counters, zero between launches
   size_t done_linear = 0;   // first counter of the linear attention
@@ -380,6 +380,7 @@ int run_mixer(fb200_llama* m, const Mixer& M, int pass, int batch, int seq, bool
     a.d = c.dim; a.v = c.vdim; a.dp = M.dp; a.pos_dev = m->pos_dev; a.z = z; a.ldz = hy->ldz; a.z_bf16 = !wide; a.commit = commit;
     a.o = hy->o; a.done = hy->done + hy->done_linear; a.bf16 = !hy->f32;
     a.q16 = (__nv_bfloat16*)hy->qn; a.k16 = (__nv_bfloat16*)hy->kn; a.v16 = (__nv_bfloat16*)hy->vn;
+    a.seg = hy->seg;
     return seq == 1 ? fb200_linear_step(dev, a) : fb200_linear_prompt(dev, a);
   }
   if (c.mixer == FB200_MIX_ATTENTION) {
@@ -491,7 +492,7 @@ int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows) {
   fb200_device* dev = m->dev;
   fb200_hybrid* hy = m->hybrid;
   const size_t E = m->cfg.hidden, nb = m->cfg.max_batch;
-  size_t q = 0, qk = 0, hv = 0, o = 0, heads = 0, kvh = 0, qa = 0, part = 0, done = 0;
+  size_t q = 0, qk = 0, hv = 0, o = 0, heads = 0, kvh = 0, qa = 0, part = 0, done = 0, seg = 0;
   for (const auto& M : hy->mixers) {
     const auto& c = M.c;
     if (c.mixer == FB200_MIX_DELTA) {
@@ -504,6 +505,7 @@ int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows) {
       if (!hy->f32) {
         qk = std::max(qk, (size_t)c.heads * M.dp / 2);
         hv = std::max(hv, c.heads * up_to(c.vdim, 8) / 2);
+        seg = std::max(seg, FB200_LINEAR_SEGMENTS * M.pass_state);
       }
     } else if (c.mixer == FB200_MIX_ATTENTION) {
       q = std::max(q, (size_t)c.heads * M.dp);
@@ -528,7 +530,7 @@ int fb200_hybrid_ensure_rows(fb200_llama* m, size_t rows) {
       {(void**)&m->x, rows * hy->ldx * 4}, {(void**)&hy->x2, hy->w_loop ? rows * hy->ldx * 4 : 0}, {(void**)&m->xn, (norm2 ? 2 : 1) * rows * E * 4},
       {(void**)&hy->proj, rows * hy->ldy * 4}, {(void**)&hy->zf, rows * hy->ldz * 4}, {(void**)&hy->hb, rows * hb * 2},
       {(void**)&hy->zb, rows * hy->ldz * 2}, {(void**)&hy->qn, rows * q * 4}, {(void**)&hy->kn, rows * qk * 4}, {(void**)&hy->vn, rows * hv * 4},
-      {(void**)&hy->gb, rows * heads * 8}, {(void**)&hy->kq, (rows + 3 * nb) / 4 * kvh * 64 + 64}, {(void**)&hy->o, rows * o * 4},
+      {(void**)&hy->gb, rows * heads * 8}, {(void**)&hy->kq, (rows + 3 * nb) / 4 * kvh * 64 + 64}, {(void**)&hy->o, rows * o * 4}, {(void**)&hy->seg, seg * 4},
       {(void**)&hy->qa, qa * 4}, {(void**)&hy->part, part * 4}, {(void**)&hy->done, (done + nb) * 4}};
   for (auto& b : bufs) {
     if (*b.p) { cudaFree(*b.p); *b.p = nullptr; }
@@ -638,7 +640,7 @@ void fb200_hybrid_free(fb200_llama* m) {
     for (void* b : bufs) if (b) cudaFree(b);
   }
   if (hy->w_loop) fb200_qmatrix_free(hy->w_loop);
-  void* bufs[] = {hy->proj, hy->zf, hy->hb, hy->zb, hy->qn, hy->kn, hy->vn, hy->gb, hy->kq, hy->o, hy->qa, hy->part, hy->done, hy->x2, hy->kvx};
+  void* bufs[] = {hy->proj, hy->zf, hy->hb, hy->zb, hy->qn, hy->kn, hy->vn, hy->gb, hy->kq, hy->o, hy->seg, hy->qa, hy->part, hy->done, hy->x2, hy->kvx};
   for (void* b : bufs) if (b) cudaFree(b);
   delete hy;
   m->hybrid = nullptr;

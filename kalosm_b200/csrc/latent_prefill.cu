@@ -76,12 +76,14 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
   uint8_t* Vs = Ks + KB * kbytes;               // [VB][NV boxes]
   uint8_t* Qs = Vs + VB * NV * (int)LP_BOX;     // [G][128][64 nk], core-matrix layout
   uint64_t* bars = reinterpret_cast<uint64_t*>(Qs + G * qbytes);
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 25);
   volatile int* dead = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  // per group: S done (one per S buffer), O += P V done, P written; per tile buffer: keys landed, values landed
-  const uint32_t bar_s = smem_u32(bars), bar_o = smem_u32(bars + 4), bar_pfull = smem_u32(bars + 6), bar_kfull = smem_u32(bars + 8),
-                 bar_vfull = smem_u32(bars + 11);
+  const int tid = threadIdx.x, warp = __shfl_sync(0xFFFFFFFFu, tid >> 5, 0), lane = tid & 31;
+  // per group: S done [2] (one per S buffer), O += P V done, P written [2]; per tile buffer: keys landed [3], values landed [2]; per
+  // group and tile buffer: keys read [3], values read [2]. No barrier may run a phase ahead of its waiter: each of these
+  // completes again only after what its waiter does next
+  const uint32_t bar_s = smem_u32(bars), bar_o = smem_u32(bars + 4), bar_pfull = smem_u32(bars + 6), bar_kfull = smem_u32(bars + 10),
+                 bar_vfull = smem_u32(bars + 13), bar_kfree = smem_u32(bars + 15), bar_vfree = smem_u32(bars + 21);
   const int qt = gridDim.x - 1 - blockIdx.x;  // longest key ranges first
   const int head = blockIdx.y, b = blockIdx.z;
   const int q0 = qt * LP_Q * G;
@@ -105,7 +107,10 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
       mbar_init(bar_s + 16 * g, 1);
       mbar_init(bar_s + 16 * g + 8, 1);
       mbar_init(bar_o + 8 * g, 1);
-      mbar_init(bar_pfull + 8 * g, LP_THREADS);
+      mbar_init(bar_pfull + 16 * g, LP_THREADS);
+      mbar_init(bar_pfull + 16 * g + 8, LP_THREADS);
+      for (int i = 0; i < KB; ++i) mbar_init(bar_kfree + 24 * g + 8 * i, 1);
+      for (int i = 0; i < VB; ++i) mbar_init(bar_vfree + 16 * g + 8 * i, 1);
     }
     for (int i = 0; i < KB; ++i) mbar_init(bar_kfull + 8 * i, 1);
     for (int i = 0; i < VB; ++i) mbar_init(bar_vfull + 8 * i, 1);
@@ -205,7 +210,7 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
   __syncthreads();  // barriers initialised, TMEM columns allocated, Q staged
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-  const uint32_t tmem = *tmem_slot;
+  const uint32_t tmem = __shfl_sync(0xFFFFFFFFu, *tmem_slot, 0);
   // instruction descriptors: fp32 accumulator, bf16 operands, M = 128; S: N = 64, both K-major; O: N = 64 NV, B MN-major
   constexpr uint32_t IDESC_S = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(LP_K >> 3) << 17) | ((uint32_t)(LP_Q >> 4) << 24);
   constexpr uint32_t IDESC_O = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(NV * 8) << 17) | ((uint32_t)(LP_Q >> 4) << 24);
@@ -232,15 +237,24 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
       while (nkt < KB && nkt < ntiles) fetch_k(nkt++);
       while (nvt < VB && nvt < ntiles) fetch_v(nvt++);
       bool ok = true;
+      int kread[G] = {}, vread[G] = {};  // per group: bit i = parity of the next phase of buffer i
       for (int u = 0; u + VB < ntiles && ok; ++u) {
         const int t = t_first + u;
+        if (u + KB < ntiles) {
 #pragma unroll
-        for (int g = 0; g < G; ++g)  // S of every group that uses the tile is done: its key buffer is free
-          if (in_range(g, t)) ok = ok && x_wait(bar_s + 16 * g + 8 * ((t - tf[g]) & 1), (uint32_t)(((t - tf[g]) >> 1) & 1), dead, a.status);
-        if (ok && u + KB < ntiles) fetch_k(nkt++);
+          for (int g = 0; g < G; ++g)  // S of every group that uses the tile is done: its key buffer is free
+            if (in_range(g, t)) {
+              ok = ok && x_wait(bar_kfree + 24 * g + 8 * (u % KB), (uint32_t)(kread[g] >> (u % KB)) & 1, dead, a.status);
+              kread[g] ^= 1 << (u % KB);
+            }
+          if (ok) fetch_k(nkt++);
+        }
 #pragma unroll
         for (int g = 0; g < G; ++g)  // and O: its value buffer is free
-          if (in_range(g, t)) ok = ok && x_wait(bar_o + 8 * g, (uint32_t)((t - tf[g]) & 1), dead, a.status);
+          if (in_range(g, t)) {
+            ok = ok && x_wait(bar_vfree + 16 * g + 8 * (u % VB), (uint32_t)(vread[g] >> (u % VB)) & 1, dead, a.status);
+            vread[g] ^= 1 << (u % VB);
+          }
         if (ok) fetch_v(nvt++);
       }
       if (*dead) {
@@ -250,7 +264,7 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
     }
   } else if (warp == SOFT / 32) {
     // ---- MMA issuer: per tile and group, S of the next tile (under the softmax of this one), then O += P V
-    if (lane == 0) {
+    {  // the whole warp runs these loops, one lane issues
       uint64_t qdesc[G], kdesc[KB], vdesc[VB];  // a descriptor's low bits hold its address / 16
 #pragma unroll
       for (int g = 0; g < G; ++g) qdesc[g] = x_desc(smem_u32(Qs) + (uint32_t)(g * qbytes), 128, (uint32_t)kchunks * 128);
@@ -260,7 +274,7 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
       for (int i = 0; i < VB; ++i) vdesc[i] = x_desc(smem_u32(Vs) + (uint32_t)(i * NV) * LP_BOX, LP_BOX, 1024, LP_SW128);
       auto issue_s = [&](int g, int u) {
         const int tg = t_first + u - tf[g];
-        x_wait(bar_kfull + 8 * (u % KB), (uint32_t)((u / KB) & 1), dead, a.status);
+        w_wait(bar_kfull + 8 * (u % KB), (uint32_t)((u / KB) & 1), dead, a.status);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         uint64_t qd = qdesc[0], kd = kdesc[0];
 #pragma unroll
@@ -270,8 +284,9 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
         const uint32_t dst = tmem + (uint32_t)(g * GCOLS + (tg & 1) * LP_K);
         for (int i = 0; i < a.nk; ++i, qd += 4 * 256 / 16, kd += LP_BOX / 16)  // a box is four steps of 16 columns (zero columns of Q where it is wider)
 #pragma unroll
-          for (int s = 0; s < 4; ++s) x_mma(dst, qd + s * (256 / 16), kd + s * (32 / 16), IDESC_S, (i | s) ? 1u : 0u);
-        x_commit(bar_s + 16 * g + 8 * (tg & 1));
+          for (int s = 0; s < 4; ++s) w_mma(dst, qd + s * (256 / 16), kd + s * (32 / 16), IDESC_S, (i | s) ? 1u : 0u);
+        w_commit(bar_s + 16 * g + 8 * (tg & 1));
+        w_commit(bar_kfree + 24 * g + 8 * (u % KB));
       };
 #pragma unroll
       for (int g = 0; g < G; ++g)
@@ -283,15 +298,16 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
           if (u + 1 < ntiles && in_range(g, t + 1)) issue_s(g, u + 1);
           if (!in_range(g, t)) continue;
           const int tg = t - tf[g];
-          x_wait(bar_pfull + 8 * g, (uint32_t)(tg & 1), dead, a.status);
-          x_wait(bar_vfull + 8 * (u % VB), (uint32_t)((u / VB) & 1), dead, a.status);
+          w_wait(bar_pfull + 16 * g + 8 * (tg & 1), (uint32_t)((tg >> 1) & 1), dead, a.status);
+          w_wait(bar_vfull + 8 * (u % VB), (uint32_t)((u / VB) & 1), dead, a.status);
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
           const uint32_t tm = tmem + (uint32_t)(g * GCOLS), pa = tm + (uint32_t)((tg & 1) * LP_K);
           const uint64_t vd = VB > 1 && (u & 1) ? vdesc[VB - 1] : vdesc[0];
 #pragma unroll
           for (int s = 0; s < LP_K / 16; ++s)  // 16 keys = 16 rows of 128 bytes further
-            x_mma_ta(tm + 2 * LP_K, pa + (uint32_t)(s * 8), vd + s * (2048 / 16), IDESC_O, (tg | s) ? 1u : 0u);
-          x_commit(bar_o + 8 * g);
+            w_mma_ta(tm + 2 * LP_K, pa + (uint32_t)(s * 8), vd + s * (2048 / 16), IDESC_O, (tg | s) ? 1u : 0u);
+          w_commit(bar_o + 8 * g);
+          w_commit(bar_vfree + 16 * g + 8 * (u % VB));
         }
       }
     }
@@ -300,7 +316,7 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
     const int g = G > 1 ? warp >> 2 : 0, r = tid & 127;
     const int t0 = G > 1 && g ? tf[G - 1] : tf[0], n = (G > 1 && g ? tl[G - 1] : tl[0]) - t0 + 1;
     const uint32_t tl_base = tmem + (uint32_t)(g * GCOLS) + ((uint32_t)(32 * (warp & 3)) << 16);
-    const uint32_t my_s = bar_s + 16 * g, my_o = bar_o + 8 * g, my_p = bar_pfull + 8 * g;
+    const uint32_t my_s = bar_s + 16 * g, my_o = bar_o + 8 * g, my_p = bar_pfull + 16 * g;
     float m_ref = -INFINITY, l_run = 0.f;
     const int qg = q0 + g * LP_Q, row = qg + r;
     const int hi = a.pos + row - a.kbase;                      // last visible key of this row
@@ -365,7 +381,7 @@ mixer_prefill_kernel(const LpArgs a, const __grid_constant__ CUtensorMap kvmap, 
       // before the last product can start, the one before it is seen complete: the final wait below then is for the
       // phase in progress (a parity wait must be neither two phases early nor two late)
       if (t > 0 && t == n - 1) x_wait(my_o, (uint32_t)((t - 1) & 1), dead, a.status);
-      mbar_arrive(my_p);
+      mbar_arrive(my_p + 8 * sb);
     }
     if (n > 0) {
       x_wait(my_o, (uint32_t)((n - 1) & 1), dead, a.status);

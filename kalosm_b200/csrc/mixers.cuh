@@ -104,7 +104,7 @@ int fb200_attn_prefill(fb200_device* dev, const fb200_attn_args& a);            
 // Projections [b * s, ldy]: q [h][d] at column 0, k [h][d] at off_k, v [h][v] at off_v (all through SiLU), gate [h v] at
 // off_g. The state of a sequence is S, f32 [h][v][dp]; position 0 starts from zero whatever the buffer holds. decay
 // [h][FB200_LINEAR_CHUNK + 1] holds the powers 0 .. of every head's decay.
-constexpr int FB200_LINEAR_CHUNK = 128;
+constexpr int FB200_LINEAR_CHUNK = 128, FB200_LINEAR_SEGMENTS = 4;
 struct fb200_linear_args {
   const float* y;
   size_t ldy;
@@ -122,6 +122,7 @@ struct fb200_linear_args {
   float* o;    // read-out [rows][h v]
   int* done;   // [b] arrival counters, zero between launches
   __nv_bfloat16 *q16, *k16, *v16;  // prompt scratch: SiLU'd q, k [rows][h][dp], v [rows][h][vp], vp = v padded to 8
+  float* seg;  // prompt scratch: [FB200_LINEAR_SEGMENTS][b][h][v][dp]
 };
 int fb200_linear_dp(int d);                                              // padded head size, 0 when d is not covered
 int fb200_linear_step(fb200_device* dev, const fb200_linear_args& a);    // s == 1: one kernel

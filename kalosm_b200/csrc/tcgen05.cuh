@@ -8,6 +8,7 @@
 
 namespace {
 
+// Waits for a phase of an mbarrier, with a limit; false: it or another role of the CTA gave up.
 __device__ __forceinline__ bool x_wait(uint32_t bar, uint32_t parity, volatile int* dead, int* status) {
   for (int it = 0; it < (1 << 22); ++it) {
     uint32_t ok;
@@ -21,6 +22,14 @@ __device__ __forceinline__ bool x_wait(uint32_t bar, uint32_t parity, volatile i
   *dead = 1;
   if (status) atomicExch(status, FB200_ERR_TIMEOUT);
   return false;
+}
+// The same for a converged warp: one lane polls. (Lanes that poll for themselves drift apart, and one that is held up in a later
+// wait can find the phase of the earlier one overtaken.)
+__device__ __forceinline__ bool w_wait(uint32_t bar, uint32_t parity, volatile int* dead, int* status) {
+  int ok = 0;
+  if ((threadIdx.x & 31) == 0) ok = x_wait(bar, parity, dead, status);
+  __syncwarp();
+  return __shfl_sync(0xFFFFFFFFu, ok, 0);
 }
 __device__ __forceinline__ void mbar_arrive(uint32_t bar) {
   asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
@@ -54,6 +63,26 @@ __device__ __forceinline__ void x_mma_ta(uint32_t tmem_d, uint32_t tmem_a, uint6
 __device__ __forceinline__ void x_commit(uint32_t bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
 }
+// The same, called by a whole converged warp: one elected lane issues. Loops around them stay uniform, so that the
+// descriptors are formed by the scalar unit and need no transfer to it.
+__device__ __forceinline__ void w_mma(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n.reg .pred p, q;\nelect.sync _|q, 0xFFFFFFFF;\nsetp.ne.b32 p, %4, 0;\n"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}"
+      ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
+}
+__device__ __forceinline__ void w_mma_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n.reg .pred p, q;\nelect.sync _|q, 0xFFFFFFFF;\nsetp.ne.b32 p, %4, 0;\n"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}"
+      ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
+}
+__device__ __forceinline__ void w_commit(uint32_t bar) {
+  asm volatile(
+      "{\n.reg .pred q;\nelect.sync _|q, 0xFFFFFFFF;\n"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n}"
+      ::"r"(bar) : "memory");
+}
 __device__ __forceinline__ void x_ld32(uint32_t taddr, uint32_t (&v)[32]) {
   asm volatile(
       "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
@@ -72,6 +101,24 @@ __device__ __forceinline__ void x_st32(uint32_t taddr, const uint32_t (&v)[32]) 
         "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]), "r"(v[16]), "r"(v[17]),
         "r"(v[18]), "r"(v[19]), "r"(v[20]), "r"(v[21]), "r"(v[22]), "r"(v[23]), "r"(v[24]), "r"(v[25]), "r"(v[26]),
         "r"(v[27]), "r"(v[28]), "r"(v[29]), "r"(v[30]), "r"(v[31])
+      : "memory");
+}
+// 16 lanes x 64 columns: v[4 i + e] of lane l is row l / 4 + 8 (e / 2), column 8 i + 2 (l % 4) + e % 2
+__device__ __forceinline__ void x_ld16x256(uint32_t taddr, uint32_t (&v)[32]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.16x256b.x8.b32 "
+      "{%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
+        "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]),
+        "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]),
+        "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
+      : "r"(taddr) : "memory");
+}
+__device__ __forceinline__ void x_st16(uint32_t taddr, const uint32_t (&v)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
+      ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]),
+        "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15])
       : "memory");
 }
 // 2^x, flushing denormals (2^-inf = 0)
