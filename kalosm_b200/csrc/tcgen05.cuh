@@ -23,13 +23,10 @@ __device__ __forceinline__ bool x_wait(uint32_t bar, uint32_t parity, volatile i
   if (status) atomicExch(status, FB200_ERR_TIMEOUT);
   return false;
 }
-// The same for a converged warp: one lane polls. (Lanes that poll for themselves drift apart, and one that is held up in a later
-// wait can find the phase of the earlier one overtaken.)
+// The same for a whole warp, which leaves it together: the vote keeps what follows uniform. (Lanes left to themselves drift apart,
+// and one that is held up in a later wait can find the phase of the earlier one overtaken.)
 __device__ __forceinline__ bool w_wait(uint32_t bar, uint32_t parity, volatile int* dead, int* status) {
-  int ok = 0;
-  if ((threadIdx.x & 31) == 0) ok = x_wait(bar, parity, dead, status);
-  __syncwarp();
-  return __shfl_sync(0xFFFFFFFFu, ok, 0);
+  return __all_sync(0xFFFFFFFFu, x_wait(bar, parity, dead, status));
 }
 __device__ __forceinline__ void mbar_arrive(uint32_t bar) {
   asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
