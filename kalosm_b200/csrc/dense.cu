@@ -6,8 +6,8 @@
 // their own:
 //  * dense_gemv_kernel (one activation row; HBM-bound: the matrix is streamed once): the row sits in shared
 //    memory as f32 (RMSNorm runs in the prologue), a warp forms two output rows at a time -- or the gate row and
-//    the up row of one SwiGLU output -- with 16-byte loads, KS warps of a CTA sharing a pair along K when there
-//    are few rows. f32 activations, f32 accumulation, sums in a fixed order.
+//    the up row of one SwiGLU output -- with 16-byte loads, KS warps of a CTA sharing a pair along K when
+//    few rows are left. f32 activations, f32 accumulation, sums in a fixed order.
 //  * dense_gemm_f32_kernel (F32 weights, any number of rows): a 64 x 64 register-blocked product in true f32.
 //  * BF16 weights with more rows: dense_tc.cu.
 #include <algorithm>
@@ -44,7 +44,7 @@ struct GemvArgs {
   const float* bias;
   float* y;
   float* z;
-  int k, kx, row0, n_plain, gate0, up0, ff, act, ks, units;
+  int k, kx, row0, n_plain, gate0, up0, ff, act, ks, whole, units;
   float eps, alpha, softcap;
 };
 
@@ -84,10 +84,7 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
   extern __shared__ __align__(16) float4 xs[];        // [P][k / E], twice where the feed-forward rows have their own norm
   __shared__ float red[2 * GV_WARPS];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int pieces = a.k / E;
-  const int ks = a.ks, teams = GV_WARPS / ks, team = warp / ks, part = warp % ks;
-  const int per = (pieces + ks - 1) / ks, p0 = part * per, p1 = min(pieces, p0 + per);
-  const int plain_units = (a.n_plain + 1) >> 1;
+  const int pieces = a.k / E, plain_units = (a.n_plain + 1) >> 1;
   auto rows_of = [&](int u, int& r0, int& r1) {
     if (u < plain_units) {
       r0 = a.row0 + 2 * u;
@@ -101,106 +98,157 @@ __global__ void __launch_bounds__(GV_THREADS, 2) dense_gemv_kernel(const GemvArg
     }
   };
   const uint4* w = reinterpret_cast<const uint4*>(a.w);
-  const int first = (int)blockIdx.x * teams + team, stride = (int)gridDim.x * teams;
+  // `whole` rounds in which every warp has a unit of its own, then one round of the rest, `ks` warps to a unit
+  const int gw = (int)blockIdx.x * GV_WARPS + warp, warps = (int)gridDim.x * GV_WARPS;
+  const int team = gw / a.ks, part = gw % a.ks, per = (pieces + a.ks - 1) / a.ks, rest = a.whole * warps + team;
   // weights do not depend on the kernel before this one: request the first pieces while it drains
-  if (first < a.units) {
-    int r0, r1;
-    rows_of(first, r0, r1);
-    for (int p = p0 + lane * 8; p < min(p1, p0 + 128); p += 256) {
-      asm volatile("prefetch.global.L2 [%0];" ::"l"(w + (size_t)r0 * pieces + p));
-      asm volatile("prefetch.global.L2 [%0];" ::"l"(w + (size_t)r1 * pieces + p));
+  {
+    const int u = a.whole ? gw : rest, p0 = a.whole ? 0 : part * per, p1 = min(pieces, a.whole ? 128 : p0 + min(per, 128));
+    if (u < a.units) {
+      int r0, r1;
+      rows_of(u, r0, r1);
+      for (int p = p0 + lane * 8; p < p1; p += 256) {
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(w + (size_t)r0 * pieces + p));
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(w + (size_t)r1 * pieces + p));
+      }
     }
   }
   pdl_wait();
   // ---- the activation row: (RMS-normalised) f32, zero padding beyond kx
-  float scale = 1.f;
-  if (a.norm_w) {
-    float ss = 0.f;
-    for (int i = tid; i < a.kx; i += GV_THREADS) {
-      const float v = __ldcg(a.x + i);
-      ss = fmaf(v, v, ss);
-    }
+  auto root = [&](float ss) {  // of the mean square, over the CTA
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, o);
     if (lane == 0) red[warp] = ss;
     __syncthreads();
     ss = 0.f;
     for (int i = 0; i < GV_WARPS; ++i) ss += red[i];
-    scale = sqrtf(ss / (float)a.kx + a.eps);
-    __syncthreads();
-  }
-  for (int i = tid; i < a.k; i += GV_THREADS) {
-    float v = 0.f, v2 = 0.f;
-    if (i < a.kx) {
-      v = __ldcg(a.x + i);
-      if (a.ff_norm_w) v2 = (v / scale) * a.ff_norm_w[i];
-      if (a.norm_w) v = (v / scale) * a.norm_w[i];
+    return sqrtf(ss / (float)a.kx + a.eps);
+  };
+  // four elements 4 i .. of the row into their plane
+  auto put = [&](float4* to, int i, const float4& v) { to[((4 * i % E) >> 2) * pieces + 4 * i / E] = v; };
+  auto times = [](const float4& v, float scale, const float4& n) {
+    return make_float4((v.x / scale) * n.x, (v.y / scale) * n.y, (v.z / scale) * n.z, (v.w / scale) * n.w);
+  };
+  const bool vec = (a.kx & 3) == 0 && (reinterpret_cast<uintptr_t>(a.x) & 15u) == 0;
+  const float4* x4 = reinterpret_cast<const float4*>(a.x);
+  const int n4 = a.k >> 2, nx4 = a.kx >> 2;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (vec && a.norm_w && n4 <= 2 * GV_THREADS) {  // the row stays in registers between the sum of squares and the norm
+    const float4 *n1 = reinterpret_cast<const float4*>(a.norm_w), *n2 = reinterpret_cast<const float4*>(a.ff_norm_w);
+    float4 v[2], m1[2], m2[2];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = tid + j * GV_THREADS;
+      v[j] = i < nx4 ? __ldcg(x4 + i) : zero;
+      m1[j] = i < nx4 ? n1[i] : zero;
+      m2[j] = n2 && i < nx4 ? n2[i] : zero;
     }
-    const int piece = i / E, e = i % E, at = ((e >> 2) * pieces + piece) * 4 + (e & 3);
-    reinterpret_cast<float*>(xs)[at] = v;
-    if (a.ff_norm_w) reinterpret_cast<float*>(xs + P * pieces)[at] = v2;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) ss = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, ss))));
+    const float scale = root(ss);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int i = tid + j * GV_THREADS;
+      if (i >= n4) continue;
+      put(xs, i, times(v[j], scale, m1[j]));
+      if (n2) put(xs + P * pieces, i, times(v[j], scale, m2[j]));
+    }
+  } else if (vec && !a.norm_w) {
+#pragma unroll 4
+    for (int i = tid; i < n4; i += GV_THREADS) put(xs, i, i < nx4 ? __ldcg(x4 + i) : zero);
+  } else {
+    float scale = 1.f;
+    if (a.norm_w) {
+      float ss = 0.f;
+      for (int i = tid; i < a.kx; i += GV_THREADS) {
+        const float v = __ldcg(a.x + i);
+        ss = fmaf(v, v, ss);
+      }
+      scale = root(ss);
+    }
+    for (int i = tid; i < a.k; i += GV_THREADS) {
+      float v = 0.f, v2 = 0.f;
+      if (i < a.kx) {
+        v = __ldcg(a.x + i);
+        if (a.ff_norm_w) v2 = (v / scale) * a.ff_norm_w[i];
+        if (a.norm_w) v = (v / scale) * a.norm_w[i];
+      }
+      const int piece = i / E, e = i % E, at = ((e >> 2) * pieces + piece) * 4 + (e & 3);
+      reinterpret_cast<float*>(xs)[at] = v;
+      if (a.ff_norm_w) reinterpret_cast<float*>(xs + P * pieces)[at] = v2;
+    }
   }
   __syncthreads();
 
-  const int rounds = (a.units + stride - 1) / stride;
-  for (int it = 0; it < rounds; ++it) {
-    // two CTAs fill an SM's registers: the next kernel is let in only when the last round has begun
-    if (it == rounds - 1) pdl_launch_dependents();
-    const int u = first + it * stride;
-    float s0 = 0.f, s1 = 0.f;
-    if (u < a.units) {
-      int r0, r1;
-      rows_of(u, r0, r1);
-      const uint4* w0 = w + (size_t)r0 * pieces;
-      const uint4* w1 = w + (size_t)r1 * pieces;
-      const float4* xu = a.ff_norm_w && u >= plain_units ? xs + P * pieces : xs;
-      int p = p0 + lane;
-      for (; p + 96 < p1; p += 128) {
-        uint4 b0[4], b1[4];
+  // this lane's share of the two sums of unit u over pieces p0 .. p1
+  auto dots = [&](int u, int p0, int p1, float& s0, float& s1) {
+    int r0, r1;
+    rows_of(u, r0, r1);
+    const uint4* w0 = w + (size_t)r0 * pieces;
+    const uint4* w1 = w + (size_t)r1 * pieces;
+    const float4* xu = a.ff_norm_w && u >= plain_units ? xs + P * pieces : xs;
+    int p = p0 + lane;
+    for (; p + 96 < p1; p += 128) {
+      uint4 b0[4], b1[4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) { b0[i] = __ldcs(w0 + p + 32 * i); b1[i] = __ldcs(w1 + p + 32 * i); }
+      for (int i = 0; i < 4; ++i) { b0[i] = __ldcs(w0 + p + 32 * i); b1[i] = __ldcs(w1 + p + 32 * i); }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float4 x0 = xu[p + 32 * i], x1 = P > 1 ? xu[(P - 1) * pieces + p + 32 * i] : x0;
-          gv_fma(b0[i], x0, x1, s0, WT());
-          gv_fma(b1[i], x0, x1, s1, WT());
-        }
-      }
-      for (; p < p1; p += 32) {
-        const uint4 b0 = __ldcs(w0 + p), b1 = __ldcs(w1 + p);
-        const float4 x0 = xu[p], x1 = P > 1 ? xu[(P - 1) * pieces + p] : x0;
-        gv_fma(b0, x0, x1, s0, WT());
-        gv_fma(b1, x0, x1, s1, WT());
+      for (int i = 0; i < 4; ++i) {
+        const float4 x0 = xu[p + 32 * i], x1 = P > 1 ? xu[(P - 1) * pieces + p + 32 * i] : x0;
+        gv_fma(b0[i], x0, x1, s0, WT());
+        gv_fma(b1[i], x0, x1, s1, WT());
       }
     }
+    for (; p < p1; p += 32) {
+      const uint4 b0 = __ldcs(w0 + p), b1 = __ldcs(w1 + p);
+      const float4 x0 = xu[p], x1 = P > 1 ? xu[(P - 1) * pieces + p] : x0;
+      gv_fma(b0, x0, x1, s0, WT());
+      gv_fma(b1, x0, x1, s1, WT());
+    }
+  };
+  auto total = [](float& s0, float& s1) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       s0 += __shfl_xor_sync(0xFFFFFFFFu, s0, o);
       s1 += __shfl_xor_sync(0xFFFFFFFFu, s1, o);
     }
-    if (ks > 1) {  // the parts of a unit meet in shared memory, added in part order
-      if (lane == 0) { red[2 * warp] = s0; red[2 * warp + 1] = s1; }
-      __syncthreads();
-      if (part == 0 && lane == 0) {
-        s0 = s1 = 0.f;
-        for (int i = 0; i < ks; ++i) { s0 += red[2 * (warp + i)]; s1 += red[2 * (warp + i) + 1]; }
-      }
-      __syncthreads();
+  };
+  auto store = [&](int u, float s0, float s1) {
+    if (u < plain_units) {
+      const int n = 2 * u;
+      a.y[n] = plain_value(s0, a.alpha, a.bias, a.add, a.softcap, n);
+      if (n + 1 < a.n_plain) a.y[n + 1] = plain_value(s1, a.alpha, a.bias, a.add, a.softcap, n + 1);
+    } else if (a.act == FB200_FFN_GELU) {
+      const int n = 2 * (u - plain_units);
+      a.z[n] = fb_gelu_tanh(s0);
+      if (n + 1 < a.ff) a.z[n + 1] = fb_gelu_tanh(s1);
+    } else {
+      a.z[u - plain_units] = silu_f(s0) * s1;
     }
-    if (u < a.units && part == 0 && lane == 0) {
-      if (u < plain_units) {
-        const int n = 2 * u;
-        a.y[n] = plain_value(s0, a.alpha, a.bias, a.add, a.softcap, n);
-        if (n + 1 < a.n_plain) a.y[n + 1] = plain_value(s1, a.alpha, a.bias, a.add, a.softcap, n + 1);
-      } else if (a.act == FB200_FFN_GELU) {
-        const int n = 2 * (u - plain_units);
-        a.z[n] = fb_gelu_tanh(s0);
-        if (n + 1 < a.ff) a.z[n + 1] = fb_gelu_tanh(s1);
-      } else {
-        a.z[u - plain_units] = silu_f(s0) * s1;
-      }
+  };
+  for (int it = 0; it < a.whole; ++it) {
+    const int u = it * warps + gw;
+    float s0 = 0.f, s1 = 0.f;
+    dots(u, 0, pieces, s0, s1);
+    total(s0, s1);
+    if (lane == 0) store(u, s0, s1);
+  }
+  // two CTAs fill an SM's registers: the next kernel is let in only when the last round begins
+  pdl_launch_dependents();
+  float s0 = 0.f, s1 = 0.f;
+  if (rest < a.units) dots(rest, part * per, min(pieces, (part + 1) * per), s0, s1);
+  total(s0, s1);
+  if (a.ks > 1) {  // the parts of a unit meet in shared memory, added in part order
+    __syncthreads();
+    if (lane == 0) { red[2 * warp] = s0; red[2 * warp + 1] = s1; }
+    __syncthreads();
+    if (part == 0 && lane == 0) {
+      s0 = s1 = 0.f;
+      for (int i = 0; i < a.ks; ++i) { s0 += red[2 * (warp + i)]; s1 += red[2 * (warp + i) + 1]; }
     }
   }
+  if (rest < a.units && part == 0 && lane == 0) store(rest, s0, s1);
 }
 
 // ---- F32 weights, many rows: 64 output rows x 64 activation rows per CTA, 4 x 4 per thread
@@ -341,16 +389,12 @@ int fb200_dense_gemv(fb200_device* dev, const fb200_dense_job& j) {
   const size_t smem = (size_t)j.w->k * (a.ff_norm_w ? 8 : 4);
   const int per_sm = smem <= 100 * 1024 ? 2 : 1;
   const int ctas = dev->sm_count * per_sm;
-  // warps per unit: the split of K that leaves the fewest warps idle in the last round (ties: the smaller split)
-  double best = 1e30;
-  for (int ks = 1; ks <= GV_WARPS; ks *= 2) {
-    if (ks > 1 && a.k / e < ks * 32) break;
-    const int teams = ctas * (GV_WARPS / ks);
-    const double cost = (double)((a.units + teams - 1) / teams) / ks * (1.0 + 0.01 * ks);
-    if (cost < best) { best = cost; a.ks = ks; }
-  }
-  const int teams = GV_WARPS / a.ks;
-  const int grid = std::min(ctas, (a.units + teams - 1) / teams);
+  // whole rounds, and for the units that are left the split of K that one round has warps for
+  a.whole = a.units / (ctas * GV_WARPS);
+  const int left = a.units - a.whole * ctas * GV_WARPS;
+  a.ks = 1;
+  while (a.ks < GV_WARPS && left * a.ks * 2 <= ctas * GV_WARPS && a.k / e >= a.ks * 2 * 32) a.ks *= 2;
+  const int grid = a.whole ? ctas : (left * a.ks + GV_WARPS - 1) / GV_WARPS;
   static bool configured[64] = {false};
   if (!configured[dev->ordinal & 63]) {
     FB_CUDA(dev, cudaFuncSetAttribute(dense_gemv_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));

@@ -14,7 +14,7 @@
 
 namespace {
 
-constexpr int GA_WARPS = 4, GA_THREADS = GA_WARPS * 32, GA_MIN_KEYS = 64, GA_MAX_SPLITS = 32;
+constexpr int GA_WARPS = 4, GA_THREADS = GA_WARPS * 32, GA_MIN_KEYS = 32, GA_MAX_SPLITS = 32;
 
 __device__ __forceinline__ float ga_warp_sum(float v) {
 #pragma unroll
@@ -34,16 +34,25 @@ __device__ __forceinline__ void ga_store(__nv_bfloat16* p, float v) { *p = __flo
 __device__ __forceinline__ void ga_store(float* p, float v) { *p = v; }
 
 // A warp writes one head of n elements: normalised under w (null: not), its first r dimensions rotated (cs, sn: this
-// position's row of the tables), x mul; zeros up to np.
+// position's row of the tables), x mul; zeros up to np. `raw`: shared memory for the head, or null where x is read again.
 template <typename T>
 __device__ __forceinline__ void ga_head(const float* x, int n, int np, const float* w, float eps, const float* cs, const float* sn, int r,
-                                        float mul, T* dst) {
+                                        float mul, T* dst, float* raw = nullptr) {
   const int lane = threadIdx.x & 31, half = r >> 1;
   float rms = 1.f;
-  if (w) {
+  if (w || raw) {
     float ss = 0.f;
-    for (int i = lane; i < n; i += 32) ss = fmaf(x[i], x[i], ss);
-    rms = sqrtf(ga_warp_sum(ss) / (float)n + eps);
+#pragma unroll 4
+    for (int i = lane; i < n; i += 32) {
+      const float v = x[i];
+      ss = fmaf(v, v, ss);
+      if (raw) raw[i] = v;
+    }
+    if (w) rms = sqrtf(ga_warp_sum(ss) / (float)n + eps);
+    if (raw) {
+      __syncwarp();
+      x = raw;
+    }
   }
   auto value = [&](int i) { return w ? (x[i] / rms) * w[i] : x[i]; };
   for (int i = lane; i < half; i += 32) {
@@ -82,7 +91,9 @@ template <typename T, int NP, int NQ>
 __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_args a, int nsplit) {
   constexpr int E = 16 / (int)sizeof(T), LPK = 64 / E, KS = 32 / LPK, U = 2;  // U: keys per lane group in flight
   constexpr int STEP = GA_WARPS * KS * U;
-  extern __shared__ __align__(16) float gsm[];  // queries [NQ][dp], later outputs [GA_WARPS][NQ][vp]
+  // queries [NQ][dp], later outputs [GA_WARPS][NQ][vp]; in a step of one position also raw heads [GA_WARPS][max(dp, vp)], q_norm,
+  // k_norm [dp], cos, sin [r / 2]
+  extern __shared__ __align__(16) float gsm[];
   __shared__ float wm[GA_WARPS][NQ], wl[GA_WARPS][NQ], wt[NQ][GA_MAX_SPLITS], tot[NQ];
   __shared__ int last;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, slot = lane / LPK, p = lane % LPK;
@@ -96,25 +107,43 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
   const int k0 = lo + split * per, k1 = min(pos + 1, k0 + per);
   T* cache = reinterpret_cast<T*>(a.cache) + (size_t)b * a.cap * a.ldc;
   const T *kc = cache + kvh * a.dp, *vc = cache + a.g * a.dp + kvh * a.vp;
-  if (a.s == 1) {  // cached rows do not depend on the kernel in front: request the first ones
-    const int k = k0 + warp * KS * U + slot;
+  uint4 kr[U][NP], vr[U][NP];
+  auto fetch = [&](int key, int u) {
 #pragma unroll
-    for (int u = 0; u < U; ++u)
-      if (k + u * KS < min(k1, pos)) {
-        if (p * 128 < a.dp * (int)sizeof(T)) asm volatile("prefetch.global.L2 [%0];" ::"l"(kc + (size_t)(k + u * KS) * a.ldc + p * (128 / (int)sizeof(T))));
-        if (p * 128 < a.vp * (int)sizeof(T)) asm volatile("prefetch.global.L2 [%0];" ::"l"(vc + (size_t)(k + u * KS) * a.ldc + p * (128 / (int)sizeof(T))));
-      }
+    for (int i = 0; i < NP; ++i) {
+      const int at = (i * LPK + p) * E;
+      kr[u][i] = at < a.dp ? *reinterpret_cast<const uint4*>(kc + (size_t)key * a.ldc + at) : make_uint4(0u, 0u, 0u, 0u);
+      vr[u][i] = at < a.vp ? *reinterpret_cast<const uint4*>(vc + (size_t)key * a.ldc + at) : make_uint4(0u, 0u, 0u, 0u);
+    }
+  };
+  const int first = k0 + warp * KS * U;  // this warp's first keys
+  const int half = a.r >> 1;
+  float* raw = gsm + max(NQ * a.dp, GA_WARPS * NQ * a.vp);
+  float *qw = raw + GA_WARPS * max(a.dp, a.vp), *kw = qw + a.dp, *cs = kw + a.dp, *sn = cs + half;
+  if (a.s == 1) {
+    // cached rows, norms and rotation do not depend on the kernel in front: requested ahead of it
+    if (first < k1)
+#pragma unroll
+      for (int u = 0; u < U; ++u) fetch(min(first + u * KS + slot, k1 - 1), u);
+    for (int i = tid; i < a.d; i += GA_THREADS) {
+      if (a.q_norm) qw[i] = a.q_norm[i];
+      if (a.k_norm) kw[i] = a.k_norm[i];
+    }
+    for (int i = tid; i < half; i += GA_THREADS) {
+      cs[i] = a.rope_cos[(size_t)pos * half + i];
+      sn[i] = a.rope_sin[(size_t)pos * half + i];
+    }
+    __syncthreads();
   }
   pdl_wait();
   pdl_launch_dependents();
   if (a.s == 1) {  // this position's queries, and its key and value where this split holds it
     const float* y = a.y + row * a.ldy;
-    const int half = a.r >> 1;
-    const float *cs = a.rope_cos + (size_t)pos * half, *sn = a.rope_sin + (size_t)pos * half;
+    float* mine = raw + warp * max(a.dp, a.vp);
     for (int job = warp; job < nq + (k1 == pos + 1 ? 2 : 0); job += GA_WARPS) {
       T* dst = cache + (size_t)pos * a.ldc;
-      if (job < nq) ga_head(y + (size_t)(h0 + job) * a.d, a.d, a.dp, a.q_norm, a.eps, cs, sn, a.r, a.scale, gsm + job * a.dp);
-      else if (job == nq) ga_head(y + a.off_k + (size_t)kvh * a.d, a.d, a.dp, a.k_norm, a.eps, cs, sn, a.r, 1.f, dst + kvh * a.dp);
+      if (job < nq) ga_head(y + (size_t)(h0 + job) * a.d, a.d, a.dp, a.q_norm ? qw : nullptr, a.eps, cs, sn, a.r, a.scale, gsm + job * a.dp, mine);
+      else if (job == nq) ga_head(y + a.off_k + (size_t)kvh * a.d, a.d, a.dp, a.k_norm ? kw : nullptr, a.eps, cs, sn, a.r, 1.f, dst + kvh * a.dp, mine);
       else ga_head(y + a.off_v + (size_t)kvh * a.v, a.v, a.vp, nullptr, 0.f, cs, sn, 0, 1.f, dst + a.g * a.dp + kvh * a.vp);
     }
   } else {
@@ -137,17 +166,11 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
       }
   }
   __syncthreads();  // the outputs take the queries' place
-  for (int kt = k0 + warp * KS * U; kt < k1; kt += STEP) {
-    uint4 kr[U][NP], vr[U][NP];
+  for (int kt = first; kt < k1; kt += STEP) {
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      const size_t key = min(kt + u * KS + slot, k1 - 1);
-#pragma unroll
-      for (int i = 0; i < NP; ++i) {
-        const int at = (i * LPK + p) * E;
-        kr[u][i] = at < a.dp ? *reinterpret_cast<const uint4*>(kc + key * a.ldc + at) : make_uint4(0u, 0u, 0u, 0u);
-        vr[u][i] = at < a.vp ? *reinterpret_cast<const uint4*>(vc + key * a.ldc + at) : make_uint4(0u, 0u, 0u, 0u);
-      }
+      const int key = min(kt + u * KS + slot, k1 - 1);
+      if (a.s > 1 || kt != first || key == pos) fetch(key, u);  // (the new position was written after the first request)
     }
     float s[U][NQ];
 #pragma unroll
@@ -294,7 +317,7 @@ int launch_rows(fb200_device* dev, const fb200_attn_args& a) {
   // enough CTAs for two per SM; fb200_attn_part_floats counts on rows gy nsplit <= 2 SMs where nsplit > 1
   int ns = (int)std::min<size_t>(GA_MAX_SPLITS, 2 * (size_t)dev->sm_count / (rows * gy));
   ns = std::max(1, std::min(ns, (keys + GA_MIN_KEYS - 1) / GA_MIN_KEYS));
-  const size_t smem = (size_t)std::max(NQ * a.dp, GA_WARPS * NQ * a.vp) * 4;
+  const size_t smem = ((size_t)std::max(NQ * a.dp, GA_WARPS * NQ * a.vp) + (a.s == 1 ? GA_WARPS * std::max(a.dp, a.vp) + 2 * a.dp + a.r : 0)) * 4;
   return fb200_launch(dev, attn_rows_kernel<T, NP, NQ>, dim3((unsigned)(rows * ns), (unsigned)gy), dim3(GA_THREADS), smem, true, a, ns);
 }
 
