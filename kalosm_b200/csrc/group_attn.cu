@@ -33,6 +33,12 @@ __device__ __forceinline__ void ga_unpack(const uint4& u, float (&f)[4], float) 
 __device__ __forceinline__ void ga_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ void ga_store(float* p, float v) { *p = v; }
 
+// exponentials and tanh in the precision of the cache: the bf16 form of tanh(z) is 1 - 2 / (1 + exp(2 z))
+__device__ __forceinline__ float ga_exp(float x, __nv_bfloat16) { return __expf(x); }
+__device__ __forceinline__ float ga_exp(float x, float) { return expf(x); }
+__device__ __forceinline__ float ga_tanh(float z, __nv_bfloat16) { return 1.0f - __fdividef(2.0f, 1.0f + __expf(fminf(2.0f * z, 80.0f))); }
+__device__ __forceinline__ float ga_tanh(float z, float) { return tanhf(z); }
+
 // A warp writes one head of n elements: normalised under w (null: not), its first r dimensions rotated (cs, sn: this
 // position's row of the tables), x mul; zeros up to np. `raw`: shared memory for the head, or null where x is read again.
 template <typename T>
@@ -90,11 +96,11 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const fb200_attn_args a)
 template <typename T, int NP, int NQ>
 __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_args a, int nsplit) {
   constexpr int E = 16 / (int)sizeof(T), LPK = 64 / E, KS = 32 / LPK, U = 2;  // U: keys per lane group in flight
-  constexpr int STEP = GA_WARPS * KS * U;
-  // queries [NQ][dp], later outputs [GA_WARPS][NQ][vp]; in a step of one position also raw heads [GA_WARPS][max(dp, vp)], q_norm,
+  constexpr int STEP = GA_WARPS * KS * U, SETS = GA_WARPS * KS, COLS = 64 * NP;  // SETS: lane groups of the CTA
+  // queries [NQ][COLS], later outputs [SETS][NQ][COLS]; in a step of one position also raw heads [GA_WARPS][max(dp, vp)], q_norm,
   // k_norm [dp], cos, sin [r / 2]
   extern __shared__ __align__(16) float gsm[];
-  __shared__ float wm[GA_WARPS][NQ], wl[GA_WARPS][NQ], wt[NQ][GA_MAX_SPLITS], tot[NQ];
+  __shared__ float wm[SETS][NQ], wl[SETS][NQ], wt[NQ][32], top[NQ], tot[NQ];
   __shared__ int last;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, slot = lane / LPK, p = lane % LPK;
   const int split = (int)(blockIdx.x % nsplit), gq = a.h / a.g, hgroups = (gq + NQ - 1) / NQ, kvh = blockIdx.y / hgroups;
@@ -118,7 +124,8 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
   };
   const int first = k0 + warp * KS * U;  // this warp's first keys
   const int half = a.r >> 1;
-  float* raw = gsm + max(NQ * a.dp, GA_WARPS * NQ * a.vp);
+  const float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
+  float* raw = gsm + SETS * NQ * COLS;
   float *qw = raw + GA_WARPS * max(a.dp, a.vp), *kw = qw + a.dp, *cs = kw + a.dp, *sn = cs + half;
   if (a.s == 1) {
     // cached rows, norms and rotation do not depend on the kernel in front: requested ahead of it
@@ -142,14 +149,16 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
     float* mine = raw + warp * max(a.dp, a.vp);
     for (int job = warp; job < nq + (k1 == pos + 1 ? 2 : 0); job += GA_WARPS) {
       T* dst = cache + (size_t)pos * a.ldc;
-      if (job < nq) ga_head(y + (size_t)(h0 + job) * a.d, a.d, a.dp, a.q_norm ? qw : nullptr, a.eps, cs, sn, a.r, a.scale, gsm + job * a.dp, mine);
+      if (job < nq) ga_head(y + (size_t)(h0 + job) * a.d, a.d, a.dp, a.q_norm ? qw : nullptr, a.eps, cs, sn, a.r, a.scale, gsm + job * COLS, mine);
       else if (job == nq) ga_head(y + a.off_k + (size_t)kvh * a.d, a.d, a.dp, a.k_norm ? kw : nullptr, a.eps, cs, sn, a.r, 1.f, dst + kvh * a.dp, mine);
       else ga_head(y + a.off_v + (size_t)kvh * a.v, a.v, a.vp, nullptr, 0.f, cs, sn, 0, 1.f, dst + a.g * a.dp + kvh * a.vp);
     }
   } else {
     const float* q = reinterpret_cast<const float*>(a.qn) + (row * a.h + h0) * a.dp;
-    for (int i = tid; i < nq * a.dp; i += GA_THREADS) gsm[i] = q[i] * a.scale;
+    for (int i = tid; i < nq * a.dp; i += GA_THREADS) gsm[i / a.dp * COLS + i % a.dp] = q[i] * a.scale;
   }
+  for (int i = tid; i < NQ * COLS; i += GA_THREADS)
+    if (i / COLS >= nq || i % COLS >= a.dp) gsm[i] = 0.f;
   __syncthreads();
   float q[NQ][NP * E], acc[NQ][NP * E], m[NQ], l[NQ];
 #pragma unroll
@@ -159,10 +168,9 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
 #pragma unroll
     for (int i = 0; i < NP; ++i)
 #pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const int at = (i * LPK + p) * E + e;
-        q[n][i * E + e] = n < nq && at < a.dp ? gsm[n * a.dp + at] : 0.f;
-        acc[n][i * E + e] = 0.f;
+      for (int e = 0; e < E; e += 4) {
+        *reinterpret_cast<float4*>(&q[n][i * E + e]) = *reinterpret_cast<const float4*>(gsm + n * COLS + (i * LPK + p) * E + e);
+        *reinterpret_cast<float4*>(&acc[n][i * E + e]) = make_float4(0.f, 0.f, 0.f, 0.f);
       }
   }
   __syncthreads();  // the outputs take the queries' place
@@ -190,7 +198,7 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
       for (int n = 0; n < NQ; ++n) {
 #pragma unroll
         for (int o = LPK / 2; o > 0; o >>= 1) s[u][n] += __shfl_xor_sync(0xFFFFFFFFu, s[u][n], o);
-        if (a.softcap > 0.f) s[u][n] = a.softcap * tanhf(s[u][n] / a.softcap);
+        if (a.softcap > 0.f) s[u][n] = a.softcap * ga_tanh(s[u][n] * inv_cap, T());
         if (kt + u * KS + slot >= k1) s[u][n] = -INFINITY;
       }
     }
@@ -200,14 +208,14 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
       float mx = m[n];
 #pragma unroll
       for (int u = 0; u < U; ++u) mx = fmaxf(mx, s[u][n]);
-      const float base = mx == -INFINITY ? 0.f : mx, alpha = expf(m[n] - base);
+      const float base = mx == -INFINITY ? 0.f : mx, alpha = ga_exp(m[n] - base, T());
       m[n] = mx;
       l[n] *= alpha;
 #pragma unroll
       for (int i = 0; i < NP * E; ++i) acc[n][i] *= alpha;
 #pragma unroll
       for (int u = 0; u < U; ++u) {
-        pr[u][n] = expf(s[u][n] - base);
+        pr[u][n] = ga_exp(s[u][n] - base, T());
         l[n] += pr[u][n];
       }
     }
@@ -223,27 +231,27 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
           for (int e = 0; e < E; ++e) acc[n][i * E + e] = fmaf(pr[u][n], f[e], acc[n][i * E + e]);
       }
   }
-  // ---- over the lane groups of a warp, then over the warps
+  // ---- the lane groups' outputs meet in shared memory
+  const int set = warp * KS + slot;
 #pragma unroll
   for (int n = 0; n < NQ; ++n) {
-    float mx = m[n];
-#pragma unroll
-    for (int o = LPK; o < 32; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, o));
-    const float w = m[n] == -INFINITY ? 0.f : expf(m[n] - mx);
-    float lt = l[n] * w;
-#pragma unroll
-    for (int o = LPK; o < 32; o <<= 1) lt += __shfl_xor_sync(0xFFFFFFFFu, lt, o);
-    if (lane == 0) { wm[warp][n] = mx; wl[warp][n] = lt; }
+    if (p == 0) { wm[set][n] = m[n]; wl[set][n] = l[n]; }
 #pragma unroll
     for (int i = 0; i < NP; ++i)
 #pragma unroll
-      for (int e = 0; e < E; ++e) {
-        float v = acc[n][i * E + e] * w;
+      for (int e = 0; e < E; e += 4)
+        *reinterpret_cast<float4*>(gsm + (set * NQ + n) * COLS + (i * LPK + p) * E + e) = *reinterpret_cast<const float4*>(&acc[n][i * E + e]);
+  }
+  __syncthreads();
+  if (warp < NQ) {
+    const float ms = lane < SETS ? wm[lane % SETS][warp] : -INFINITY;
+    float mx = ms;
 #pragma unroll
-        for (int o = LPK; o < 32; o <<= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
-        const int at = (i * LPK + p) * E + e;
-        if (slot == 0 && at < a.vp) gsm[(warp * NQ + n) * a.vp + at] = v;
-      }
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, o));
+    const float w = ms == -INFINITY ? 0.f : ga_exp(ms - mx, T());
+    const float lt = ga_warp_sum(w != 0.f ? wl[lane % SETS][warp] * w : 0.f);
+    wt[warp][lane] = w;
+    if (lane == 0) { top[warp] = mx; tot[warp] = lt; }
   }
   __syncthreads();
   const float* y = a.y + row * a.ldy;
@@ -257,15 +265,10 @@ __global__ void __launch_bounds__(GA_THREADS) attn_rows_kernel(const fb200_attn_
   float* part = a.part + ((row * a.h + h0) * (size_t)nsplit) * (a.v + 2);  // [head][split][v + 2]
   for (int i = tid; i < nq * a.v; i += GA_THREADS) {
     const int n = i / a.v, c = i % a.v;
-    float mx = -INFINITY, v = 0.f, lt = 0.f;
-#pragma unroll
-    for (int w = 0; w < GA_WARPS; ++w) mx = fmaxf(mx, wm[w][n]);
-#pragma unroll
-    for (int w = 0; w < GA_WARPS; ++w) {
-      const float f = wm[w][n] == -INFINITY ? 0.f : expf(wm[w][n] - mx);
-      v = fmaf(gsm[(w * NQ + n) * a.vp + c], f, v);
-      lt = fmaf(wl[w][n], f, lt);
-    }
+    const float mx = top[n];
+    float v = 0.f, lt = tot[n];
+#pragma unroll 4
+    for (int j = 0; j < SETS; ++j) v = fmaf(gsm[(j * NQ + n) * COLS + c], wt[n][j], v);
     if (active == 1) {
       if (a.sink) lt += expf(a.sink[h0 + n] - mx);
       put(n, c, v / lt);
@@ -317,7 +320,8 @@ int launch_rows(fb200_device* dev, const fb200_attn_args& a) {
   // enough CTAs for two per SM; fb200_attn_part_floats counts on rows gy nsplit <= 2 SMs where nsplit > 1
   int ns = (int)std::min<size_t>(GA_MAX_SPLITS, 2 * (size_t)dev->sm_count / (rows * gy));
   ns = std::max(1, std::min(ns, (keys + GA_MIN_KEYS - 1) / GA_MIN_KEYS));
-  const size_t smem = ((size_t)std::max(NQ * a.dp, GA_WARPS * NQ * a.vp) + (a.s == 1 ? GA_WARPS * std::max(a.dp, a.vp) + 2 * a.dp + a.r : 0)) * 4;
+  constexpr int SETS = GA_WARPS * 32 * 16 / (int)sizeof(T) / 64;
+  const size_t smem = ((size_t)SETS * NQ * 64 * NP + (a.s == 1 ? GA_WARPS * std::max(a.dp, a.vp) + 2 * a.dp + a.r : 0)) * 4;
   return fb200_launch(dev, attn_rows_kernel<T, NP, NQ>, dim3((unsigned)(rows * ns), (unsigned)gy), dim3(GA_THREADS), smem, true, a, ns);
 }
 
