@@ -54,13 +54,13 @@ __device__ __forceinline__ void ga_head(const float* x, int n, int np, const flo
       ss = fmaf(v, v, ss);
       if (raw) raw[i] = v;
     }
-    if (w) rms = sqrtf(ga_warp_sum(ss) / (float)n + eps);
+    if (w) rms = 1.0f / sqrtf(ga_warp_sum(ss) / (float)n + eps);
     if (raw) {
       __syncwarp();
       x = raw;
     }
   }
-  auto value = [&](int i) { return w ? (x[i] / rms) * w[i] : x[i]; };
+  auto value = [&](int i) { return w ? (x[i] * rms) * w[i] : x[i]; };
   for (int i = lane; i < half; i += 32) {
     const float u = value(i), v = value(i + half);
     ga_store(dst + i, (u * cs[i] - v * sn[i]) * mul);
@@ -69,20 +69,78 @@ __device__ __forceinline__ void ga_head(const float* x, int n, int np, const flo
   for (int i = r + lane; i < np; i += 32) ga_store(dst + i, i < n ? value(i) * mul : 0.f);
 }
 
+__device__ __forceinline__ void ga_store2(__nv_bfloat16* p, float x, float y) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(x, y); }
+__device__ __forceinline__ void ga_store2(float* p, float x, float y) { *reinterpret_cast<float2*>(p) = make_float2(x, y); }
+
+// ga_head for n and r multiples of 4, rows and heads 8-byte aligned: two elements per access, read once. J: pairs per lane.
+template <int J, typename T>
+__device__ __forceinline__ void ga_head_pairs(const float* x, int n, int np, const float* w, float eps, const float* cs, const float* sn, int r, T* dst) {
+  const int lane = threadIdx.x & 31, hp = r >> 2, rp = r >> 1, pairs = n >> 1;  // pairs of the half, of the rotated part, of the head
+  const float2 *x2 = reinterpret_cast<const float2*>(x), *w2 = reinterpret_cast<const float2*>(w);
+  // lane's pair j: the first half of the rotated part (its partner hp pairs behind), then what does not rotate
+  float2 u[J], v[J];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < J; ++j) {
+    const int i = lane + 32 * j, at = i < hp ? i : i + hp;
+    u[j] = at < pairs ? x2[at] : make_float2(0.f, 0.f);
+    v[j] = i < hp ? x2[i + hp] : make_float2(0.f, 0.f);
+    ss = fmaf(u[j].x, u[j].x, fmaf(u[j].y, u[j].y, fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, ss))));
+  }
+  const float inv = w ? 1.0f / sqrtf(ga_warp_sum(ss) / (float)n + eps) : 1.f;
+#pragma unroll
+  for (int j = 0; j < J; ++j) {
+    const int i = lane + 32 * j, at = i < hp ? i : i + hp;
+    if (at >= (np >> 1)) continue;
+    if (w && at < pairs) {
+      const float2 f = w2[at];
+      u[j] = make_float2(u[j].x * inv * f.x, u[j].y * inv * f.y);
+    }
+    if (i < hp) {
+      if (w) {
+        const float2 f = w2[i + hp];
+        v[j] = make_float2(v[j].x * inv * f.x, v[j].y * inv * f.y);
+      }
+      const float2 c = reinterpret_cast<const float2*>(cs)[i], s = reinterpret_cast<const float2*>(sn)[i];
+      ga_store2(dst + 2 * i, u[j].x * c.x - v[j].x * s.x, u[j].y * c.y - v[j].y * s.y);
+      ga_store2(dst + 2 * i + rp, v[j].x * c.x + u[j].x * s.x, v[j].y * c.y + u[j].y * s.y);
+    } else {
+      ga_store2(dst + 2 * at, u[j].x, u[j].y);
+    }
+  }
+}
+
 template <typename T, typename QT>
 __global__ void __launch_bounds__(256) attn_prep_kernel(const fb200_attn_args a) {
   const int slots = a.h + 2 * a.g;
-  const size_t id = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5), total = (size_t)a.b * a.s * slots;
+  const uint32_t id = blockIdx.x * 8 + (threadIdx.x >> 5), total = (uint32_t)(a.b * a.s) * slots;
   pdl_wait();
   pdl_launch_dependents();
   if (id >= total) return;
-  const size_t row = id / slots;
+  const uint32_t row = id / slots;
   const int slot = (int)(id % slots), b = (int)(row / a.s), pos = *a.pos_dev + (int)(row % a.s), half = a.r >> 1;
-  const float* y = a.y + row * a.ldy;
+  const float* y = a.y + (size_t)row * a.ldy;
   const float *cs = a.rope_cos + (size_t)pos * half, *sn = a.rope_sin + (size_t)pos * half;
   T* cache = reinterpret_cast<T*>(a.cache) + ((size_t)b * a.cap + pos) * a.ldc;
-  if (slot < a.h) {
-    ga_head(y + (size_t)slot * a.d, a.d, a.dp, a.q_norm, a.eps, cs, sn, a.r, 1.f, reinterpret_cast<QT*>(a.qn) + (row * a.h + slot) * a.dp);
+  const bool pairs = ((a.d | a.v | a.r | a.off_k | a.off_v | (int)a.ldy) & 3) == 0 && a.d <= 256 && a.v <= 256 &&
+                     (reinterpret_cast<uintptr_t>(a.y) & 7u) == 0;
+  if (pairs) {  // heads are multiples of 4: the padding to dp and vp is at most two pairs
+    const bool is_v = slot >= a.h + a.g;
+    const int k = is_v ? slot - a.h - a.g : slot - a.h, n = is_v ? a.v : a.d;
+    const float* x = slot < a.h ? y + (size_t)slot * a.d : is_v ? y + a.off_v + (size_t)k * a.v : y + a.off_k + (size_t)k * a.d;
+    const float* w = slot < a.h ? a.q_norm : is_v ? nullptr : a.k_norm;
+    const int r = is_v ? 0 : a.r;
+    if (slot < a.h) {
+      QT* dst = reinterpret_cast<QT*>(a.qn) + ((size_t)row * a.h + slot) * a.dp;
+      if (n <= 128) ga_head_pairs<2>(x, n, a.dp, w, a.eps, cs, sn, r, dst);
+      else ga_head_pairs<4>(x, n, a.dp, w, a.eps, cs, sn, r, dst);
+    } else {
+      T* dst = cache + (is_v ? a.g * a.dp + k * a.vp : k * a.dp);
+      if (n <= 128) ga_head_pairs<2>(x, n, is_v ? a.vp : a.dp, w, a.eps, cs, sn, r, dst);
+      else ga_head_pairs<4>(x, n, is_v ? a.vp : a.dp, w, a.eps, cs, sn, r, dst);
+    }
+  } else if (slot < a.h) {
+    ga_head(y + (size_t)slot * a.d, a.d, a.dp, a.q_norm, a.eps, cs, sn, a.r, 1.f, reinterpret_cast<QT*>(a.qn) + ((size_t)row * a.h + slot) * a.dp);
   } else if (slot < a.h + a.g) {
     const int k = slot - a.h;
     ga_head(y + a.off_k + (size_t)k * a.d, a.d, a.dp, a.k_norm, a.eps, cs, sn, a.r, 1.f, cache + k * a.dp);
@@ -351,6 +409,7 @@ size_t fb200_attn_part_floats(const fb200_device* dev, int v) { return (size_t)2
 
 int fb200_attn_prepare(fb200_device* dev, const fb200_attn_args& a, bool q_bf16) {
   const size_t warps = (size_t)a.b * a.s * (a.h + 2 * a.g);
+  if (warps >= (1ull << 32)) return fb200_fail(dev, FB200_ERR_CAPACITY, "grouped attention: %d x %d rows of %d heads in one pass", a.b, a.s, a.h);
   const dim3 grid((unsigned)((warps + 7) / 8)), block(256);
   if (a.cache_f32) return fb200_launch(dev, attn_prep_kernel<float, float>, grid, block, 0, true, a);
   if (q_bf16) return fb200_launch(dev, attn_prep_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, 0, true, a);

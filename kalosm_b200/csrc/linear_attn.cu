@@ -38,9 +38,25 @@ __device__ __forceinline__ void linear_finish_row(const fb200_linear_args& a, si
   __syncthreads();
   ss = 0.f;
   for (int i = 0; i < LS_THREADS / 32; ++i) ss += red[i];
-  const float rms = sqrtf(ss / (float)n + a.eps);
+  const float inv = 1.0f / sqrtf(ss / (float)n + a.eps);
+  if ((n & 3) == 0 && (reinterpret_cast<uintptr_t>(g) & 15u) == 0 && (a.ldz & 3) == 0 && (reinterpret_cast<uintptr_t>(a.z) & 15u) == 0) {
+    for (int i = 4 * tid; i < n; i += 4 * LS_THREADS) {
+      const float4 x = __ldcg(reinterpret_cast<const float4*>(o + i)), w = *reinterpret_cast<const float4*>(a.out_norm + i);
+      const float4 y = *reinterpret_cast<const float4*>(g + i);
+      const float v0 = x.x * inv * w.x * dr_sigmoid(y.x) * a.out_scale, v1 = x.y * inv * w.y * dr_sigmoid(y.y) * a.out_scale;
+      const float v2 = x.z * inv * w.z * dr_sigmoid(y.z) * a.out_scale, v3 = x.w * inv * w.w * dr_sigmoid(y.w) * a.out_scale;
+      if (a.z_bf16) {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v0, v1), hi = __floats2bfloat162_rn(v2, v3);
+        *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.z) + row * a.ldz + i) =
+            make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+      } else {
+        *reinterpret_cast<float4*>(reinterpret_cast<float*>(a.z) + row * a.ldz + i) = make_float4(v0, v1, v2, v3);
+      }
+    }
+    return;
+  }
   for (int i = tid; i < n; i += LS_THREADS) {
-    const float x = (__ldcg(o + i) / rms) * a.out_norm[i] * dr_sigmoid(g[i]) * a.out_scale;
+    const float x = __ldcg(o + i) * inv * a.out_norm[i] * dr_sigmoid(g[i]) * a.out_scale;
     if (a.z_bf16) reinterpret_cast<__nv_bfloat16*>(a.z)[row * a.ldz + i] = __float2bfloat16(x);
     else reinterpret_cast<float*>(a.z)[row * a.ldz + i] = x;
   }

@@ -35,7 +35,7 @@ def check(dev, cfg, w, tokens, dtype, sizes, **kw):
 
 # ---- products with dense weights --------------------------------------------------------------------------
 
-@pytest.mark.parametrize("m,n,k", [(1, 130, 72), (1, 4099, 1024), (2, 65, 40), (5, 300, 264), (33, 129, 64), (64, 1000, 520),
+@pytest.mark.parametrize("m,n,k", [(1, 130, 72), (1, 4099, 1024), (1, 20001, 264), (1, 9472, 64), (2, 65, 40), (5, 300, 264), (33, 129, 64), (64, 1000, 520),
                                    (130, 257, 2048), (257, 4000, 128), (700, 260, 1032)])
 @pytest.mark.parametrize("ty", ["bf16", "f32"])
 def test_dense_products(dev, m, n, k, ty):

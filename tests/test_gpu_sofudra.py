@@ -87,6 +87,15 @@ def test_right_side_alone(dev, dtype, shape):
     check(dev, cfg, w, toks(cfg, 210), dtype, [[210], [70, 3, 65, 2, 17, 1], [64, 64, 64, 18], [16, 48, 128, 18]])
 
 
+@pytest.mark.parametrize("dim,vdim", [(128, 100), (40, 64)])
+def test_linear_attention_in_segments(dev, dim, vdim):
+    # prompts long enough to be cut into segments that run side by side, also behind earlier tokens
+    cfg = alone([V.parallel(b=V.right(2, dim, vdim, [0.9995, 0.9]), mlp=0)])
+    ident = U.identity_head(cfg)
+    w = V.weights(cfg, 62, lambda n, a: np.zeros_like(a) if n.endswith("left.o") else ident(n, a))
+    check(dev, cfg, w, toks(cfg, 1700), "bfloat16", [[1700], [37, 1100, 513, 50]], max_seq_len=1704)
+
+
 @pytest.mark.parametrize("window,sizes", [(1, [700]), (70, [700]), (200, [650, 50]), (64, [300, 400]), (5000, [257, 443])], ids=str)
 @pytest.mark.parametrize("vdim", [64, 128])
 def test_attention_many_rows(dev, window, sizes, vdim):
